@@ -36,7 +36,7 @@ class NormSpec:
 class PositionSpec:
     """A position encoding applied to query and key head vectors."""
 
-    kind: str  # "rope_neox"; "rope_scaled" (params: factor, low, high, original)
+    kind: str  # "rope_neox"; "rope_linear" (params: factor); "rope_scaled" (params: factor, low, high, original)
     head_dim: int
     rotary_dim: int
     theta: float
@@ -65,7 +65,8 @@ class MixerSpec:
     # temp_coef, temp_every, sink and distance_slopes; "rglru" reads width, blocks,
     # taps and decay_scale; "pair" reads left and right (two `MixerSpec`s) and eps;
     # "gqa_attention" reads values_are_keys, output_gate and keep_first; "selective_scan"
-    # reads inner, state, dt_rank and taps
+    # reads inner, state, dt_rank and taps; "capped_attention" reads bias, unit_eps, softcap and
+    # value_mix; "gated_delta" reads taps, unit_eps and eps
     params: Tuple[Tuple[str, Any], ...] = ()
     # size of a head's value vector when it differs from `head_dim`; 0: the same
     v_head_dim: int = 0
@@ -80,7 +81,7 @@ class MixerSpec:
 
 @dataclass(frozen=True)
 class FeedForwardSpec:
-    kind: str  # "swiglu"; "relu2"; "glu_clamped" (params: alpha, limit); "moe" (params: experts, top, activation,
+    kind: str  # "swiglu"; "geglu"; "relu2"; "glu_clamped" (params: alpha, limit); "moe" (params: experts, top, activation,
     # router_bias, scores, weight_input, alpha, limit, shared_ff, shared_limit)
     hidden_size: int
     intermediate_size: int
@@ -185,6 +186,10 @@ class ModelSpec:
     # None: the model has none
     pass_vectors_name: Optional[str] = None
     pass_vectors: int = 0
+    # a norm on the token embedding (after its scale, before the embedding terms): the
+    # residual stream starts normed; None: it starts as it is
+    embedding_norm: Optional[NormSpec] = None
+    embedding_norm_name: Optional[str] = None
 
     def __post_init__(self) -> None:
         if not self.run_order:

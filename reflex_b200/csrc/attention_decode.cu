@@ -78,7 +78,8 @@ constexpr int MAX_RANKS = 16;  // 8 is the portable cluster size; 16 where the d
 
 // TMA: the page tiles come by tensor-map loads (D a multiple of 64) and lie
 // swizzled, [D / 64][PAGE][64]; else by 16-byte copies into padded rows.
-template <int D, bool TMA, bool PEN>
+// MODE: 0 the scores as they are, 1 with a distance bias (`slopes`), 2 capped (`softcap`).
+template <int D, bool TMA, int MODE>
 __global__ void __launch_bounds__(DEC_THREADS + 32)
 attention_decode_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_constant__ CUtensorMap map_v,
                         const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __restrict__ k_pages,
@@ -86,7 +87,7 @@ attention_decode_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_
                         const int* __restrict__ row_pos, const int* __restrict__ row_slot,
                         __nv_bfloat16* __restrict__ out, float* __restrict__ partial, int nq,
                         int n_htiles, int n_splits, int window, int keep_first, float scale_log2,
-                        const float* __restrict__ sink, const float* __restrict__ slopes,
+                        const float* __restrict__ sink, const float* __restrict__ slopes, float softcap,
                         int cluster_merge, int trace_id, int* __restrict__ err) {
     constexpr int LD = D + 8;
     constexpr int TILE = TMA ? PAGE * D : PAGE * LD;  // elements of a page's key (or value) tile
@@ -169,7 +170,11 @@ attention_decode_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_
     // a distance bias: slope * (query position - key position) off every score; the
     // slopes are weights (no kernel writes them), times log2(e) like the scale
     float pen[2] = {0.0f, 0.0f};
-    if (PEN && slopes) {
+    if (MODE == 2) {  // the pair that `capped_log2` takes
+        pen[0] = 2.0f * scale_log2 / softcap;
+        pen[1] = softcap * LOG2E;
+    }
+    if (MODE == 1 && slopes) {
 #pragma unroll
         for (int j = 0; j < 2; ++j)
             if (2 * (lane & 3) + j < nh) pen[j] = slopes[h0 + 2 * (lane & 3) + j] * LOG2E;
@@ -221,7 +226,7 @@ attention_decode_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_
         // that the four warps are done with it; nothing else orders them page by page.
         if (warp < 4) {
             auto nothing = [&](int) { return false; };
-            attend_keys16<D, true, PEN>(qf, kbuf + (DEC_STAGES - 1) * TILE, vbuf + (DEC_STAGES - 1) * TILE, warp * 16,
+            attend_keys16<D, true, MODE>(qf, kbuf + (DEC_STAGES - 1) * TILE, vbuf + (DEC_STAGES - 1) * TILE, warp * 16,
                                    scale_log2, nothing, pen, 0, m, l, acc);
             reset();
             // the dry pass is this buffer's first use: done with it
@@ -288,7 +293,7 @@ attention_decode_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_
                 auto visible = [&](int key) {
                     return (base + key >= lo || base + key < keep_first) && base + key <= pos;
                 };
-                attend_keys16<D, true, PEN>(qf, kbuf + buf * TILE, vbuf + buf * TILE, warp * 16, scale_log2, visible,
+                attend_keys16<D, true, MODE>(qf, kbuf + buf * TILE, vbuf + buf * TILE, warp * 16, scale_log2, visible,
                                        pen, pos - base, m, l, acc);
                 __syncwarp();
                 if (lane == 0) sm100::mbar_arrive(&empty_bar[buf]);
@@ -321,7 +326,7 @@ attention_decode_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_
             auto visible = [&](int key) {
                 return (base + key >= lo_eff || base + key < keep_eff) && base + key <= pos;
             };
-            attend_keys16<D, false, PEN>(qf, kbuf + buf * TILE, vbuf + buf * TILE, warp * 16, scale_log2, visible,
+            attend_keys16<D, false, MODE>(qf, kbuf + buf * TILE, vbuf + buf * TILE, warp * 16, scale_log2, visible,
                                     pen, pos - base, m, l, acc);
             if (tracing && !dry) attending += clock64() - c2;
             if (dry) {
@@ -540,11 +545,11 @@ const CUtensorMap* store_map(const void* base, long long rows, int D) {
     return &cache.emplace(key, m).first->second;
 }
 
-template <int D, bool TMA, bool PEN>
+template <int D, bool TMA, int MODE>
 int launch_decode(const void* q, const void* k_pages, const void* v_pages, long long pool_pages,
                   const PagedKV& cache, const int* row_pos, const int* row_slot, void* out, float* partial,
                   int R, int nq, int n_splits, int window, int keep_first, float scale, const float* sink,
-                  const float* slopes, int cluster_merge, int* err, cudaStream_t s) {
+                  const float* slopes, float softcap, int cluster_merge, int* err, cudaStream_t s) {
     constexpr int LD = D + 8;
     const int g = nq / cache.n_kv_heads;
     const int n_htiles = (g + 7) / 8;
@@ -563,7 +568,7 @@ int launch_decode(const void* q, const void* k_pages, const void* v_pages, long 
         mv = store_map(v_pages, rows, D);
         if (!mk || !mv) return RFX_ERR_UNSUPPORTED;
     }
-    auto kernel = attention_decode_kernel<D, TMA, PEN>;
+    auto kernel = attention_decode_kernel<D, TMA, MODE>;
     cudaError_t e = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     if (e != cudaSuccess) return (int)e;
     dim3 grid(R, cache.n_kv_heads * n_htiles, n_splits);
@@ -596,7 +601,7 @@ int launch_decode(const void* q, const void* k_pages, const void* v_pages, long 
                     cluster_merge ? n_splits : 1, *mk, *mv,
                     (const __nv_bfloat16*)q, (const __nv_bfloat16*)k_pages, (const __nv_bfloat16*)v_pages,
                     cache, row_pos, row_slot, (__nv_bfloat16*)out, partial, nq, n_htiles, n_splits, window,
-                    keep_first, scale * LOG2E, sink, slopes, cluster_merge, g_dtrace_next++, err);
+                    keep_first, scale * LOG2E, sink, slopes, softcap, cluster_merge, g_dtrace_next++, err);
     if (e != cudaSuccess) return (int)e;
     if (n_splits > 1 && !cluster_merge)
         RFX_LAUNCH(attention_combine_kernel, R * nq, D <= 128 ? 64 : 128, 0, s, (const float*)partial,
@@ -607,10 +612,11 @@ int launch_decode(const void* q, const void* k_pages, const void* v_pages, long 
 int decode_entry(const void* q, const void* k_pages, const void* v_pages, const int* page_table,
                  int max_pages, int page_size, const int* row_pos, const int* row_slot, void* out,
                  float* partial, int R, int nq, int nkv, int head_dim, int n_splits, int window,
-                 int keep_first, float scale, const float* sink, const float* slopes, int cluster_merge,
+                 int keep_first, float scale, const float* sink, const float* slopes, float softcap, int cluster_merge,
                  long long pool_pages, int* err, void* stream) {
     if (R <= 0) return 0;
     if (page_size != PAGE || nkv <= 0 || nq % nkv != 0 || n_splits < 1) return RFX_ERR_BAD_ARG;
+    if (softcap < 0.0f || (softcap > 0.0f && slopes)) return RFX_ERR_UNSUPPORTED;  // one or the other
     if (n_splits > 1 && !partial && !cluster_merge) return RFX_ERR_BAD_ARG;
     if (cluster_merge && n_splits != 2 && n_splits != 4 && n_splits != 8 && n_splits != 16) return RFX_ERR_UNSUPPORTED;
     if (n_splits > MAX_SPLITS) return RFX_ERR_UNSUPPORTED;
@@ -626,12 +632,11 @@ int decode_entry(const void* q, const void* k_pages, const void* v_pages, const 
     const bool tma = tma_on && pool_pages > 0 && head_dim % 64 == 0 &&
                      ((reinterpret_cast<uintptr_t>(k_pages) | reinterpret_cast<uintptr_t>(v_pages)) & 15) == 0 &&
                      pool_pages * nkv * PAGE < 2147483647LL;
-    // with slopes: the kernel's form that takes the distance term off the scores
-#define RFX_GO(DD, T)                                                                                              \
-    (slopes ? launch_decode<DD, T, true>(q, k_pages, v_pages, pool_pages, cache, row_pos, row_slot, out, partial, \
-                                         R, nq, n_splits, window, keep_first, scale, sink, slopes, cluster_merge, err, s)     \
-            : launch_decode<DD, T, false>(q, k_pages, v_pages, pool_pages, cache, row_pos, row_slot, out, partial, \
-                                          R, nq, n_splits, window, keep_first, scale, sink, slopes, cluster_merge, err, s))
+    // with slopes or a cap: the kernel's form that has that term
+#define RFX_FORM(DD, T, M)                                                                                  \
+    launch_decode<DD, T, M>(q, k_pages, v_pages, pool_pages, cache, row_pos, row_slot, out, partial, R, nq, \
+                            n_splits, window, keep_first, scale, sink, slopes, softcap, cluster_merge, err, s)
+#define RFX_GO(DD, T) (slopes ? RFX_FORM(DD, T, 1) : softcap > 0.0f ? RFX_FORM(DD, T, 2) : RFX_FORM(DD, T, 0))
 #define RFX_CASE(DD)                                        \
     case DD:                                                \
         if (DD % 64 == 0 && tma) {                          \
@@ -648,6 +653,7 @@ int decode_entry(const void* q, const void* k_pages, const void* v_pages, const 
     }
 #undef RFX_CASE
 #undef RFX_GO
+#undef RFX_FORM
 }
 
 }  // namespace
@@ -668,23 +674,24 @@ extern "C" int rfx_attention_decode(const void* q, const void* k_pages, const vo
                                     int n_splits, int window, float scale, const float* sink,
                                     const float* slopes, long long pool_pages, int* err, void* stream) {
     return decode_entry(q, k_pages, v_pages, page_table, max_pages, page_size, row_pos, row_slot, out,
-                        partial, R, nq, nkv, head_dim, n_splits, window, 0, scale, sink, slopes, 0, pool_pages,
+                        partial, R, nq, nkv, head_dim, n_splits, window, 0, scale, sink, slopes, 0.0f, 0, pool_pages,
                         err, stream);
 }
 
-// The same with `keep_first`: the first so many positions of a sequence stay
-// visible beyond the window.
+// The same with `keep_first` (the first so many positions of a sequence stay
+// visible beyond the window) and `softcap` (> 0: a score s becomes softcap * tanh(s / softcap)
+// before the softmax; not together with slopes).
 extern "C" int rfx_attention_decode_kf(const void* q, const void* k_pages, const void* v_pages,
                                        const int* page_table, int max_pages, int page_size,
                                        const int* row_pos, const int* row_slot, void* out,
                                        float* partial, int R, int nq, int nkv, int head_dim,
                                        int n_splits, int window, int keep_first, float scale, const float* sink,
-                                       const float* slopes, long long pool_pages, int cluster, int* err,
-                                       void* stream) {
+                                       const float* slopes, float softcap, long long pool_pages, int cluster,
+                                       int* err, void* stream) {
     if (keep_first < 0) return RFX_ERR_BAD_ARG;
     return decode_entry(q, k_pages, v_pages, page_table, max_pages, page_size, row_pos, row_slot, out,
                         cluster ? nullptr : partial, R, nq, nkv, head_dim, n_splits, window, keep_first, scale,
-                        sink, slopes, cluster ? 1 : 0, pool_pages, err, stream);
+                        sink, slopes, softcap, cluster ? 1 : 0, pool_pages, err, stream);
 }
 
 // The same with 2, 4, 8 or (where the device places such a cluster) 16 splits that
@@ -701,7 +708,7 @@ extern "C" int rfx_attention_decode_cluster(const void* q, const void* k_pages, 
                                             float scale, const float* sink, const float* slopes,
                                             long long pool_pages, int* err, void* stream) {
     return decode_entry(q, k_pages, v_pages, page_table, max_pages, page_size, row_pos, row_slot, out,
-                        nullptr, R, nq, nkv, head_dim, n_splits, window, 0, scale, sink, slopes, 1, pool_pages,
+                        nullptr, R, nq, nkv, head_dim, n_splits, window, 0, scale, sink, slopes, 0.0f, 1, pool_pages,
                         err, stream);
 }
 

@@ -10,7 +10,7 @@
 // however far back they lie;  s_j = (q . K_j) * scale;  online softmax
 // m' = max(m, s), l = l e^(m-m') + e^(s-m'), acc = acc e^(m-m') + e^(s-m') V_j;
 // With `slopes` (one per query head) s_j loses slope * (p - j), a linear
-// distance bias.  out = acc / l   (src/kernels_cuda/attention_online.cuh:64-102; the window
+// distance bias; with `softcap` > 0 it becomes softcap * tanh(s_j / softcap).  out = acc / l   (src/kernels_cuda/attention_online.cuh:64-102; the window
 // rule is src/model/config.rs:1184-1185: i - j < window).
 //
 // Orders, which a host mirror repeats bit for bit: the dot product as a fused
@@ -26,15 +26,14 @@ namespace {
 
 using namespace rfx;
 
-constexpr int MAX_PER_LANE = 16;  // head_dim <= 512
-
-template <typename T>
+// MAX_PER_LANE: 16 (head_dim <= 512) or 32 (<= 1024)
+template <typename T, int MAX_PER_LANE>
 __global__ void __launch_bounds__(128)
 attention_plain_kernel(const T* __restrict__ q, const T* __restrict__ k_pages,
                        const T* __restrict__ v_pages, PagedKV cache,
                        const int* __restrict__ row_pos, const int* __restrict__ row_slot,
                        T* __restrict__ out, int nq, int window, int keep_first, float scale,
-                       const float* __restrict__ sink, const float* __restrict__ slopes) {
+                       const float* __restrict__ sink, const float* __restrict__ slopes, float softcap) {
     pdl_prologue();
     const int d = cache.head_dim;
     const int r = blockIdx.x;
@@ -72,6 +71,7 @@ attention_plain_kernel(const T* __restrict__ q, const T* __restrict__ k_pages,
         float s = warp_sum(dot) * scale;
         // a distance bias: slope * (query position - key position) off the score
         if (slopes) s = fmaf(-slope, (float)(pos - j), s);
+        if (softcap > 0.0f) s = softcap * tanhf(s / softcap);
         const float m_new = fmaxf(m, s);
         const float corr = exact_expf(m - m_new);  // 0 at the first key (m = -inf)
         const float p = exact_expf(s - m_new);
@@ -107,23 +107,28 @@ extern "C" int rfx_attention_plain(const void* q, const void* k_pages, const voi
                                    const int* page_table, int max_pages, int page_size,
                                    const int* row_pos, const int* row_slot, void* out, int R,
                                    int nq, int nkv, int head_dim, int window, int keep_first, float scale,
-                                   const float* sink, const float* slopes, void* stream) {
+                                   const float* sink, const float* slopes, float softcap, void* stream) {
     if (R <= 0) return 0;
-    if (head_dim <= 0 || head_dim > 32 * MAX_PER_LANE) return RFX_ERR_UNSUPPORTED;
+    if (head_dim <= 0 || head_dim > 1024) return RFX_ERR_UNSUPPORTED;
+    if (softcap < 0.0f) return RFX_ERR_BAD_ARG;
     if (nkv <= 0 || nq % nkv != 0) return RFX_ERR_BAD_ARG;
     PagedKV cache{page_table, max_pages, page_size, nkv, head_dim};
     dim3 grid(R, (nq + 3) / 4);
     if (grid.y > 65535) return RFX_ERR_UNSUPPORTED;
     cudaStream_t s = (cudaStream_t)stream;
-    if (dt == RFX_DT_F32)
-        RFX_LAUNCH(attention_plain_kernel<float>, grid, 128, 0, s, (const float*)q,
-                   (const float*)k_pages, (const float*)v_pages, cache, row_pos, row_slot,
-                   (float*)out, nq, window, keep_first, scale, sink, slopes);
-    else if (dt == RFX_DT_BF16)
-        RFX_LAUNCH(attention_plain_kernel<__nv_bfloat16>, grid, 128, 0, s, (const __nv_bfloat16*)q,
-                   (const __nv_bfloat16*)k_pages, (const __nv_bfloat16*)v_pages, cache, row_pos,
-                   row_slot, (__nv_bfloat16*)out, nq, window, keep_first, scale, sink, slopes);
-    else
+#define RFX_GO(T, N)                                                                                       \
+    RFX_LAUNCH((attention_plain_kernel<T, N>), grid, 128, 0, s, (const T*)q, (const T*)k_pages,            \
+               (const T*)v_pages, cache, row_pos, row_slot, (T*)out, nq, window, keep_first, scale, sink, \
+               slopes, softcap)
+    if (dt == RFX_DT_F32) {
+        if (head_dim <= 512) RFX_GO(float, 16);
+        else RFX_GO(float, 32);
+    } else if (dt == RFX_DT_BF16) {
+        if (head_dim <= 512) RFX_GO(__nv_bfloat16, 16);
+        else RFX_GO(__nv_bfloat16, 32);
+    } else {
         return RFX_ERR_BAD_ARG;
+    }
+#undef RFX_GO
     return 0;
 }

@@ -31,7 +31,7 @@ attention_prefill_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat1
                          const int* __restrict__ seq_new, const int* __restrict__ seq_row0,
                          __nv_bfloat16* __restrict__ out, int nq, int bq, int window, int keep_first,
                          float scale_log2, const float* __restrict__ sink,
-                         const float* __restrict__ slopes) {
+                         const float* __restrict__ slopes, float softcap) {
     constexpr int LD = D + 8;
     extern __shared__ __align__(16) uint8_t smem_raw[];
     __nv_bfloat16* qs = reinterpret_cast<__nv_bfloat16*>(smem_raw);  // [128][LD]
@@ -127,13 +127,20 @@ attention_prefill_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat1
             };
             if (slopes) {
                 // a distance bias: slope * (query position - key position) off the score
-                auto penalty = [&](int key, int h) { return row_pen[h] * (float)(row_pos[h] - (base + key)); };
-                attend_tile<D, 8>(qs + warp_row0 * LD, kbuf + buf * PAGE * LD, vbuf + buf * PAGE * LD, 0,
-                                  scale_log2, visible, penalty, m, l, acc);
-            } else {  // the tile code as it is without the term (x - 0 folds away)
-                auto none = [](int, int) { return 0.0f; };
-                attend_tile<D, 8>(qs + warp_row0 * LD, kbuf + buf * PAGE * LD, vbuf + buf * PAGE * LD, 0,
-                                  scale_log2, visible, none, m, l, acc);
+                auto biased = [&](float s, int key, int h) {
+                    return s * scale_log2 - row_pen[h] * (float)(row_pos[h] - (base + key));
+                };
+                attend_tile<D, 8>(qs + warp_row0 * LD, kbuf + buf * PAGE * LD, vbuf + buf * PAGE * LD, 0, visible,
+                                  biased, m, l, acc);
+            } else if (softcap > 0.0f) {
+                const float in2 = 2.0f * scale_log2 / softcap, out2 = softcap * 1.4426950408889634f;
+                auto capped = [&](float s, int, int) { return capped_log2(s, in2, out2); };
+                attend_tile<D, 8>(qs + warp_row0 * LD, kbuf + buf * PAGE * LD, vbuf + buf * PAGE * LD, 0, visible,
+                                  capped, m, l, acc);
+            } else {
+                auto scaled = [&](float s, int, int) { return s * scale_log2; };
+                attend_tile<D, 8>(qs + warp_row0 * LD, kbuf + buf * PAGE * LD, vbuf + buf * PAGE * LD, 0, visible,
+                                  scaled, m, l, acc);
             }
         }
         __syncthreads();
@@ -159,7 +166,7 @@ template <int D>
 int launch_prefill(const void* q, const void* k_pages, const void* v_pages, const PagedKV& cache,
                    const int* seq_slot, const int* seq_start, const int* seq_new,
                    const int* seq_row0, void* out, int S, int max_new, int nq, int window, int keep_first,
-                   float scale, const float* sink, const float* slopes, cudaStream_t s) {
+                   float scale, const float* sink, const float* slopes, float softcap, cudaStream_t s) {
     constexpr int LD = D + 8;
     const int g = nq / cache.n_kv_heads;
     if (g > PF_ROWS) return RFX_ERR_UNSUPPORTED;
@@ -172,7 +179,8 @@ int launch_prefill(const void* q, const void* k_pages, const void* v_pages, cons
     if (grid.y > 65535 || grid.z > 65535) return RFX_ERR_UNSUPPORTED;
     RFX_LAUNCH(kernel, grid, PF_THREADS, smem, s, (const __nv_bfloat16*)q,
                (const __nv_bfloat16*)k_pages, (const __nv_bfloat16*)v_pages, cache, seq_slot, seq_start,
-               seq_new, seq_row0, (__nv_bfloat16*)out, nq, bq, window, keep_first, scale * 1.4426950408889634f, sink, slopes);
+               seq_new, seq_row0, (__nv_bfloat16*)out, nq, bq, window, keep_first, scale * 1.4426950408889634f, sink, slopes,
+               softcap);
     return 0;
 }
 
@@ -186,22 +194,22 @@ int launch_prefill(const void* q, const void* k_pages, const void* v_pages, cons
 // off every score.
 // head_dim: multiples of 16 up to 256; group size nq / nkv up to 128; page 64.
 // `keep_first`: with a window, the first so many positions of a sequence stay visible
-// beyond it.
+// beyond it.  `softcap` > 0: a score s becomes softcap * tanh(s / softcap) (not with slopes).
 extern "C" int rfx_attention_prefill_kf(const void* q, const void* k_pages, const void* v_pages,
                                         const int* page_table, int max_pages, int page_size,
                                         const int* seq_slot, const int* seq_start, const int* seq_new,
                                         const int* seq_row0, void* out, int S, int max_new, int nq,
                                         int nkv, int head_dim, int window, int keep_first, float scale,
-                                        const float* sink, const float* slopes, void* stream) {
+                                        const float* sink, const float* slopes, float softcap, void* stream) {
     if (S <= 0 || max_new <= 0) return 0;
-    if (keep_first < 0) return RFX_ERR_BAD_ARG;
+    if (keep_first < 0 || softcap < 0.0f || (softcap > 0.0f && slopes)) return RFX_ERR_BAD_ARG;
     if (page_size != PAGE || nkv <= 0 || nq % nkv != 0) return RFX_ERR_BAD_ARG;
     PagedKV cache{page_table, max_pages, page_size, nkv, head_dim};
     cudaStream_t s = (cudaStream_t)stream;
 #define RFX_CASE(DD)                                                                              \
     case DD:                                                                                      \
         return launch_prefill<DD>(q, k_pages, v_pages, cache, seq_slot, seq_start, seq_new,       \
-                                  seq_row0, out, S, max_new, nq, window, keep_first, scale, sink, slopes, s);
+                                  seq_row0, out, S, max_new, nq, window, keep_first, scale, sink, slopes, softcap, s);
     switch (head_dim) {
         RFX_CASE(16) RFX_CASE(32) RFX_CASE(48) RFX_CASE(64) RFX_CASE(80) RFX_CASE(96)
         RFX_CASE(112) RFX_CASE(128) RFX_CASE(144) RFX_CASE(160) RFX_CASE(176) RFX_CASE(192)
@@ -220,5 +228,5 @@ extern "C" int rfx_attention_prefill(const void* q, const void* k_pages, const v
                                      const float* slopes, void* stream) {
     return rfx_attention_prefill_kf(q, k_pages, v_pages, page_table, max_pages, page_size, seq_slot, seq_start,
                                     seq_new, seq_row0, out, S, max_new, nq, nkv, head_dim, window, 0, scale, sink,
-                                    slopes, stream);
+                                    slopes, 0.0f, stream);
 }

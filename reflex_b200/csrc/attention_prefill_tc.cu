@@ -25,6 +25,7 @@
 #include <mutex>
 #include <tuple>
 
+#include "attn_mma.cuh"
 #include "common.cuh"
 #include "paged.cuh"
 #include "sm100.cuh"
@@ -109,7 +110,11 @@ struct Smem {
 // every score of head h; taken off the raw score as (slope / scale) * distance,
 // so that the scale's multiply-add in the exponent covers it.  Without it the
 // kernel's instructions are what they were.
-template <int D, bool SLOPES>
+// MODE 1: slopes.  MODE 2, 3: capped scores, cap * tanh(s scale / cap): the tanh of s * `in_scale`
+// takes the raw score's place and `scale_log2` is cap * log2(e), so the rest of the page's code
+// is the same.  MODE 2 takes any argument; MODE 3 the polynomial for |s in_scale| <= 1/2, which
+// leaves the special-function unit to the softmax's exponentials.
+template <int D, int MODE>
 __global__ void __launch_bounds__(THREADS)
 attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q,
                             const __grid_constant__ CUtensorMap map_k,
@@ -117,8 +122,9 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q,
                             const int* __restrict__ seq_slot, const int* __restrict__ seq_start,
                             const int* __restrict__ seq_new, const int* __restrict__ seq_row0,
                             __nv_bfloat16* __restrict__ out, int nq, int bq, int window, int keep_first,
-                            float scale_log2, const float* __restrict__ sink,
+                            float scale_log2, float in_scale, const float* __restrict__ sink,
                             const float* __restrict__ slopes, int* __restrict__ err) {
+    constexpr bool SLOPES = MODE == 1;
     static_assert(D == 64 || D == 128, "head sizes 64 and 128");
     constexpr int KB = D / 64;                 // 64-column blocks of a row
     constexpr int KV_BYTES = PAGE * D * 2;
@@ -318,6 +324,17 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q,
                 for (int c = 0; c < PAGE; ++c)
                     sr[c] = __float_as_uint(fmaf(-slope_raw, d0 - (float)c, __uint_as_float(sr[c])));
             }
+            if constexpr (MODE == 2) {
+#pragma unroll
+                for (int c = 0; c < PAGE; ++c)
+                    sr[c] = __float_as_uint(
+                        attn::capped_log2(__uint_as_float(sr[c]), 2.0f * 1.4426950408889634f * in_scale, 1.0f));
+            }
+            if constexpr (MODE == 3) {
+#pragma unroll
+                for (int c = 0; c < PAGE; ++c)
+                    sr[c] = __float_as_uint(attn::tanh_small(__uint_as_float(sr[c]) * in_scale));
+            }
             if (all_visible) {
 #pragma unroll
                 for (int c = 0; c < PAGE; ++c) s[c] = __uint_as_float(sr[c]);
@@ -454,11 +471,11 @@ bool make_map_q(CUtensorMap* map, const void* base, int R, int nq, int D, int g,
               CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE) == CUDA_SUCCESS;
 }
 
-template <int D, bool SLOPES>
+template <int D, int MODE>
 int launch_tc(const void* q, const void* k_pages, const void* v_pages, long long n_pages_total,
               const PagedKV& cache, const int* seq_slot, const int* seq_start, const int* seq_new,
               const int* seq_row0, void* out, int S, int max_new, int R, int nq, int window, int keep_first,
-              float scale, const float* sink, const float* slopes, int* err, cudaStream_t s) {
+              float scale, const float* sink, const float* slopes, float softcap, int* err, cudaStream_t s) {
     const int g = nq / cache.n_kv_heads;
     if (g > ROWS) return RFX_ERR_UNSUPPORTED;
     const int bq = ROWS / g;
@@ -468,14 +485,15 @@ int launch_tc(const void* q, const void* k_pages, const void* v_pages, long long
         !rfx::tma::make_map_rows64(&mv, v_pages, kv_rows, D, PAGE))
         return RFX_ERR_UNSUPPORTED;
     const size_t smem = Smem::total(D);
-    auto kernel = attention_prefill_tc_kernel<D, SLOPES>;
+    auto kernel = attention_prefill_tc_kernel<D, MODE>;
     cudaError_t e = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     if (e != cudaSuccess) return (int)e;
     if ((max_new + bq - 1) / bq > 65535 || S > 65535) return RFX_ERR_UNSUPPORTED;
     dim3 grid(cache.n_kv_heads, S, (max_new + bq - 1) / bq);
     if (grid.y > 65535 || grid.z > 65535) return RFX_ERR_UNSUPPORTED;
     RFX_LAUNCH(kernel, grid, THREADS, smem, s, mq, mk, mv, cache, seq_slot, seq_start, seq_new, seq_row0,
-               (__nv_bfloat16*)out, nq, bq, window, keep_first, scale * 1.4426950408889634f, sink, slopes, err);
+               (__nv_bfloat16*)out, nq, bq, window, keep_first,
+               (MODE >= 2 ? softcap : scale) * 1.4426950408889634f, MODE >= 2 ? scale / softcap : 1.0f, sink, slopes, err);
     return 0;
 }
 
@@ -496,28 +514,39 @@ extern "C" int rfx_attention_prefill_tc_trace(void* buffer, int ctas) {
 }
 
 // `keep_first`: with a window, the first so many positions of a sequence stay visible
-// beyond it.
+// beyond it.  `softcap` > 0: a score s becomes softcap * tanh(s / softcap) (not with slopes);
+// `score_bound` > 0: the caller's word that no |s| is larger.
 extern "C" int rfx_attention_prefill_tc_kf(const void* q, const void* k_pages, const void* v_pages,
                                            long long n_pages_total, const int* page_table, int max_pages,
                                            int page_size, const int* seq_slot, const int* seq_start,
                                            const int* seq_new, const int* seq_row0, void* out, int S,
                                            int max_new, int R, int nq, int nkv, int head_dim, int window,
                                            int keep_first, float scale, const float* sink, const float* slopes,
-                                           int* err, void* stream) {
+                                           float softcap, float score_bound, int* err, void* stream) {
     if (S <= 0 || max_new <= 0 || R <= 0) return 0;
     if (keep_first < 0 || !(scale > 0.0f)) return RFX_ERR_UNSUPPORTED;  // the maximum is taken before the scale
     if (page_size != PAGE || nkv <= 0 || nq % nkv != 0) return RFX_ERR_BAD_ARG;
+    if (softcap < 0.0f || (softcap > 0.0f && slopes)) return RFX_ERR_UNSUPPORTED;
     if (slopes && !(scale > 0.0f)) return RFX_ERR_UNSUPPORTED;  // the slopes ride on the scale's multiply-add
     if ((reinterpret_cast<uintptr_t>(q) | reinterpret_cast<uintptr_t>(k_pages) |
          reinterpret_cast<uintptr_t>(v_pages)) & 15)
         return RFX_ERR_BAD_ARG;
     PagedKV cache{page_table, max_pages, page_size, nkv, head_dim};
     cudaStream_t s = (cudaStream_t)stream;
-#define RFX_GO(DD, SL)                                                                                  \
-    launch_tc<DD, SL>(q, k_pages, v_pages, n_pages_total, cache, seq_slot, seq_start, seq_new, seq_row0, \
-                      out, S, max_new, R, nq, window, keep_first, scale, sink, slopes, err, s)
-    if (head_dim == 64) return slopes ? RFX_GO(64, true) : RFX_GO(64, false);
-    if (head_dim == 128) return slopes ? RFX_GO(128, true) : RFX_GO(128, false);
+#define RFX_GO(DD, M)                                                                                   \
+    launch_tc<DD, M>(q, k_pages, v_pages, n_pages_total, cache, seq_slot, seq_start, seq_new, seq_row0, \
+                      out, S, max_new, R, nq, window, keep_first, scale, sink, slopes, softcap, err, s)
+    const int mode = slopes ? 1 : !(softcap > 0.0f) ? 0 : (score_bound > 0.0f && score_bound <= attn::TANH_SMALL * softcap) ? 3 : 2;
+#define RFX_D(DD)                             \
+    if (head_dim == DD) {                     \
+        if (mode == 0) return RFX_GO(DD, 0);  \
+        if (mode == 1) return RFX_GO(DD, 1);  \
+        if (mode == 2) return RFX_GO(DD, 2);  \
+        return RFX_GO(DD, 3);                 \
+    }
+    RFX_D(64)
+    RFX_D(128)
+#undef RFX_D
 #undef RFX_GO
     return RFX_ERR_UNSUPPORTED;
 }
@@ -531,5 +560,5 @@ extern "C" int rfx_attention_prefill_tc(const void* q, const void* k_pages, cons
                                         void* stream) {
     return rfx_attention_prefill_tc_kf(q, k_pages, v_pages, n_pages_total, page_table, max_pages, page_size,
                                        seq_slot, seq_start, seq_new, seq_row0, out, S, max_new, R, nq, nkv,
-                                       head_dim, window, 0, scale, sink, slopes, err, stream);
+                                       head_dim, window, 0, scale, sink, slopes, 0.0f, 0.0f, err, stream);
 }

@@ -67,6 +67,26 @@ __device__ __forceinline__ uint32_t pack_bf16(float lo, float hi) {
     return *reinterpret_cast<uint32_t*>(&v);
 }
 
+// A capped score, cap * tanh(s scale / cap) times log2(e), for any argument: tanh(y) =
+// 1 - 2 / (1 + e^2y) with the hardware's base-2 exponential and reciprocal.
+// `in2` = 2 log2(e) scale / cap, `out2` = cap log2(e).  The result is off by about 1e-7 of the cap.
+__device__ __forceinline__ float capped_log2(float s, float in2, float out2) {
+    float e, r;
+    asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(e) : "f"(s * in2));
+    asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(r) : "f"(1.0f + e));
+    return fmaf(-2.0f * out2, r, out2);
+}
+// tanh(y) / y as a polynomial in y^2, |y| <= 1/2 (least squares in a Chebyshev basis, relative
+// error 2e-8): tanh without the special-function unit, where the caller knows the bound.
+constexpr float TANH_SMALL = 0.5f;
+__device__ __forceinline__ float tanh_small(float y) {
+    const float z = y * y;
+    float p = fmaf(0.01714132f, z, -0.05298924f);
+    p = fmaf(p, z, 0.13324829f);
+    p = fmaf(p, z, -0.33333072f);
+    return fmaf(p * z, y, y);
+}
+
 // Copy `rows_valid` rows of a contiguous [rows][D] global tile into a padded
 // shared tile; rows beyond are zero-filled.  All `nthreads` threads take part.
 template <int D>
@@ -85,13 +105,13 @@ __device__ __forceinline__ void load_tile_async(__nv_bfloat16* smem, const __nv_
 //   qs: [16][D + 8] query rows (already in shared memory)
 //   kvalid(j): whether tile key j (0-based in the tile) is visible to row half
 //   hrow (0: row lane/4, 1: row lane/4 + 8)
-// scale_log2 = scale * log2(e); probabilities are 2^(s * scale_log2 - m).
-//   penalty(j, hrow): what is taken off a visible key's scaled score (a distance
-//   bias, already times log2(e)); 0.0f leaves the score's bits as they are
-template <int D, int NT, typename Visible, typename Penalty>
+// Probabilities are 2^(score - m):
+//   score(s, j, hrow): a visible key's score times log2(e), from the raw product s
+//   (its scale, a distance bias, a cap)
+template <int D, int NT, typename Visible, typename Score>
 __device__ __forceinline__ void attend_tile(const __nv_bfloat16* qs, const __nv_bfloat16* ks,
-                                            const __nv_bfloat16* vs, int key0, float scale_log2,
-                                            Visible visible, Penalty penalty, float (&m)[2], float (&l)[2],
+                                            const __nv_bfloat16* vs, int key0, Visible visible, Score score,
+                                            float (&m)[2], float (&l)[2],
                                             float (&acc)[D / 8][4]) {
     static_assert(NT % 2 == 0, "keys come in pairs of 8-key tiles");
     const int lane = threadIdx.x & 31;
@@ -124,7 +144,7 @@ __device__ __forceinline__ void attend_tile(const __nv_bfloat16* qs, const __nv_
         for (int i = 0; i < 4; ++i) {
             const int key = key0 + t * 8 + 2 * (lane & 3) + (i & 1);
             const int h = i >> 1;
-            const float v = visible(key, h) ? s[t][i] * scale_log2 - penalty(key, h) : -INFINITY;
+            const float v = visible(key, h) ? score(s[t][i], key, h) : -INFINITY;
             s[t][i] = v;
             mx[h] = fmaxf(mx[h], v);
         }
@@ -216,11 +236,12 @@ __device__ __forceinline__ const __nv_bfloat16* tile_at(const __nv_bfloat16* til
     return tile + row * (D + 8) + col;
 }
 
-//   pen[2], dist0: a distance bias on the scores.  Tile key j lies dist0 - j
-//   positions before the query, and pen[i] * (dist0 - j) is taken off its scaled
-//   score for the thread's i-th head (slope times log2(e)).  PEN false: no such
-//   term, and the instructions are what they were without it
-template <int D, bool SWZ = false, bool PEN = false, typename Visible>
+//   MODE 0: the scores as they are (the instructions of no other mode are in the way).
+//   MODE 1: a distance bias.  Tile key j lies dist0 - j positions before the query, and
+//   pen[i] * (dist0 - j) is taken off its scaled score for the thread's i-th head
+//   (slope times log2(e)).
+//   MODE 2: capped scores (`capped_log2`), pen[0] its `in2`, pen[1] its `out2`
+template <int D, bool SWZ = false, int MODE = 0, typename Visible>
 __device__ __forceinline__ void attend_keys16(const uint32_t (&qf)[D / 16][2], const __nv_bfloat16* ks,
                                               const __nv_bfloat16* vs, int key0, float scale_log2,
                                               Visible visible, const float (&pen)[2], int dist0,
@@ -237,7 +258,12 @@ __device__ __forceinline__ void attend_keys16(const uint32_t (&qf)[D / 16][2], c
     const int ka = key0 + (lane >> 2), kb = ka + 8;
     const bool va = visible(ka), vb = visible(kb);
     float v[4];
-    if constexpr (PEN) {
+    if constexpr (MODE == 2) {
+        v[0] = va ? capped_log2(s[0], pen[0], pen[1]) : -INFINITY;
+        v[1] = va ? capped_log2(s[1], pen[0], pen[1]) : -INFINITY;
+        v[2] = vb ? capped_log2(s[2], pen[0], pen[1]) : -INFINITY;
+        v[3] = vb ? capped_log2(s[3], pen[0], pen[1]) : -INFINITY;
+    } else if constexpr (MODE == 1) {
         const float da = (float)(dist0 - ka), db = (float)(dist0 - kb);
         v[0] = va ? s[0] * scale_log2 - pen[0] * da : -INFINITY;
         v[1] = va ? s[1] * scale_log2 - pen[1] * da : -INFINITY;

@@ -144,6 +144,22 @@ __device__ __forceinline__ float silu_mul_for(float g, float u) {
     else return silu_mul(g, u);
 }
 
+// gelu(g) * u with the tanh form of gelu, 0.5 g (1 + tanh(sqrt(2 / pi) (g + 0.044715 g^3))); for a
+// result that is rounded to bfloat16 as g / (1 + e^(-2 y)), the same function, with the fast
+// exponential and division.
+template <typename TO>
+__device__ __forceinline__ float gelu_tanh_mul_for(float g, float u) {
+    const float y = 0.7978845608028654f * fmaf(0.044715f * g * g, g, g);
+    if constexpr (sizeof(TO) == 2) return __fdividef(g, 1.0f + __expf(-2.0f * y)) * u;
+    else return (0.5f * g * (1.0f + tanhf(y))) * u;
+}
+// The gated activations by number: 0 silu, 1 the tanh form of gelu.
+template <typename TO, int ACT>
+__device__ __forceinline__ float gated_mul_for(float g, float u) {
+    if constexpr (ACT == 1) return gelu_tanh_mul_for<TO>(g, u);
+    else return silu_mul_for<TO>(g, u);
+}
+
 // Sum over the 32 lanes in a fixed butterfly order; every lane gets the total.
 __device__ __forceinline__ float warp_sum(float v) {
 #pragma unroll

@@ -94,10 +94,10 @@ __global__ void rmsnorm_kernel(const float* x, const TD* __restrict__ delta,
     }
 }
 
-// out[r, i] = silu(gate_i) * up_i,  silu(g) = g / (1 + exp(-g))
+// out[r, i] = act(gate_i) * up_i, act silu, g / (1 + exp(-g)), or (ACT 1) the tanh form of gelu
 // (src/kernels_cuda/silu_and_mul.cu:7-23).  A row of `gu` holds the gates in its
 // first half and the ups in its second, or (alternating) gate_i at 2i, up_i at 2i+1.
-template <typename T>
+template <typename T, int ACT>
 __global__ void swiglu_kernel(const T* __restrict__ gu, T* __restrict__ out, int R, int I,
                               int alternating) {
     pdl_prologue();
@@ -107,7 +107,7 @@ __global__ void swiglu_kernel(const T* __restrict__ gu, T* __restrict__ out, int
         const size_t r = i / I, c = i % I;
         const float g = ld<T>(gu, r * 2 * I + (alternating ? 2 * c : c));
         const float u = ld<T>(gu, r * 2 * I + (alternating ? 2 * c + 1 : I + c));
-        st<T>(out, i, silu_mul_for<T>(g, u));
+        st<T>(out, i, gated_mul_for<T, ACT>(g, u));
     }
 }
 
@@ -115,6 +115,7 @@ __global__ void swiglu_kernel(const T* __restrict__ gu, T* __restrict__ out, int
 // stores, two steps' loads in flight.  With alternating pairs a row's 2I inputs
 // and I outputs are contiguous and rows follow one another, so output pack i
 // comes from input elements [16 i, 16 i + 16).
+template <int ACT>
 __device__ __forceinline__ uint4 swiglu8(const uint4 a, const uint4 b, bool alternating) {
     const __nv_bfloat162* pa = reinterpret_cast<const __nv_bfloat162*>(&a);
     const __nv_bfloat162* pb = reinterpret_cast<const __nv_bfloat162*>(&b);
@@ -125,22 +126,23 @@ __device__ __forceinline__ uint4 swiglu8(const uint4 a, const uint4 b, bool alte
         for (int j = 0; j < 2; ++j) {
             const float2 p0 = __bfloat1622float2(pa[2 * j]), p1 = __bfloat1622float2(pa[2 * j + 1]);
             const float2 q0 = __bfloat1622float2(pb[2 * j]), q1 = __bfloat1622float2(pb[2 * j + 1]);
-            po[j] = __floats2bfloat162_rn(silu_mul_for<__nv_bfloat16>(p0.x, p0.y),
-                                          silu_mul_for<__nv_bfloat16>(p1.x, p1.y));
-            po[2 + j] = __floats2bfloat162_rn(silu_mul_for<__nv_bfloat16>(q0.x, q0.y),
-                                              silu_mul_for<__nv_bfloat16>(q1.x, q1.y));
+            po[j] = __floats2bfloat162_rn(gated_mul_for<__nv_bfloat16, ACT>(p0.x, p0.y),
+                                          gated_mul_for<__nv_bfloat16, ACT>(p1.x, p1.y));
+            po[2 + j] = __floats2bfloat162_rn(gated_mul_for<__nv_bfloat16, ACT>(q0.x, q0.y),
+                                              gated_mul_for<__nv_bfloat16, ACT>(q1.x, q1.y));
         }
     } else {  // a = eight gates, b = their ups
 #pragma unroll
         for (int j = 0; j < 4; ++j) {
             const float2 g = __bfloat1622float2(pa[j]), up = __bfloat1622float2(pb[j]);
-            po[j] = __floats2bfloat162_rn(silu_mul_for<__nv_bfloat16>(g.x, up.x),
-                                          silu_mul_for<__nv_bfloat16>(g.y, up.y));
+            po[j] = __floats2bfloat162_rn(gated_mul_for<__nv_bfloat16, ACT>(g.x, up.x),
+                                          gated_mul_for<__nv_bfloat16, ACT>(g.y, up.y));
         }
     }
     return o;
 }
 
+template <int ACT>
 __global__ void __launch_bounds__(256)
 swiglu_bf16x8_kernel(const __nv_bfloat16* __restrict__ gu, __nv_bfloat16* __restrict__ out, int R, int I,
                      int alternating) {
@@ -164,13 +166,13 @@ swiglu_bf16x8_kernel(const __nv_bfloat16* __restrict__ gu, __nv_bfloat16* __rest
         sources(i, a0, b0);
         sources(i + step, a1, b1);
         const uint4 va0 = *a0, vb0 = *b0, va1 = *a1, vb1 = *b1;
-        *reinterpret_cast<uint4*>(out + 8 * i) = swiglu8(va0, vb0, alternating);
-        *reinterpret_cast<uint4*>(out + 8 * (i + step)) = swiglu8(va1, vb1, alternating);
+        *reinterpret_cast<uint4*>(out + 8 * i) = swiglu8<ACT>(va0, vb0, alternating);
+        *reinterpret_cast<uint4*>(out + 8 * (i + step)) = swiglu8<ACT>(va1, vb1, alternating);
     }
     if (i < n8) {
         const uint4 *a0, *b0;
         sources(i, a0, b0);
-        *reinterpret_cast<uint4*>(out + 8 * i) = swiglu8(*a0, *b0, alternating);
+        *reinterpret_cast<uint4*>(out + 8 * i) = swiglu8<ACT>(*a0, *b0, alternating);
     }
 }
 
@@ -243,28 +245,45 @@ extern "C" int rfx_rmsnorm(const float* x, const void* delta, int delta_dt, floa
     return 0;
 }
 
-extern "C" int rfx_swiglu(const void* gate_up, void* out, int dt, int R, int I, int alternating,
-                          void* stream) {
+// `act`: 0 silu, 1 the tanh form of gelu.
+extern "C" int rfx_gated_act(const void* gate_up, void* out, int dt, int R, int I, int alternating, int act,
+                             void* stream) {
     if (R <= 0 || I <= 0) return 0;
+    if (act != 0 && act != 1) return RFX_ERR_BAD_ARG;
     cudaStream_t s = (cudaStream_t)stream;
     const size_t n = (size_t)R * I;
     int blocks = (int)((n + 255) / 256);
     if (blocks > sm_count() * 16) blocks = sm_count() * 16;
-    if (dt == RFX_DT_F32)
-        RFX_LAUNCH(swiglu_kernel<float>, blocks, 256, 0, s, (const float*)gate_up, (float*)out, R, I,
-                   alternating);
-    else if (dt == RFX_DT_BF16 && I % 8 == 0 &&
-             ((reinterpret_cast<uintptr_t>(gate_up) | reinterpret_cast<uintptr_t>(out)) & 15) == 0) {
+#define RFX_GO(T)                                                                                                \
+    do {                                                                                                         \
+        if (act == 0)                                                                                            \
+            RFX_LAUNCH((swiglu_kernel<T, 0>), blocks, 256, 0, s, (const T*)gate_up, (T*)out, R, I, alternating); \
+        else                                                                                                     \
+            RFX_LAUNCH((swiglu_kernel<T, 1>), blocks, 256, 0, s, (const T*)gate_up, (T*)out, R, I, alternating); \
+    } while (0)
+    if (dt == RFX_DT_F32) {
+        RFX_GO(float);
+    } else if (dt == RFX_DT_BF16 && I % 8 == 0 &&
+               ((reinterpret_cast<uintptr_t>(gate_up) | reinterpret_cast<uintptr_t>(out)) & 15) == 0) {
         int b8 = (int)((n / 8 + 255) / 256);
         if (b8 > sm_count() * 8) b8 = sm_count() * 8;
-        RFX_LAUNCH(swiglu_bf16x8_kernel, b8, 256, 0, s, (const __nv_bfloat16*)gate_up,
-                   (__nv_bfloat16*)out, R, I, alternating);
-    } else if (dt == RFX_DT_BF16)
-        RFX_LAUNCH(swiglu_kernel<__nv_bfloat16>, blocks, 256, 0, s, (const __nv_bfloat16*)gate_up,
-                   (__nv_bfloat16*)out, R, I, alternating);
-    else
+        if (act == 0)
+            RFX_LAUNCH(swiglu_bf16x8_kernel<0>, b8, 256, 0, s, (const __nv_bfloat16*)gate_up, (__nv_bfloat16*)out, R,
+                       I, alternating);
+        else
+            RFX_LAUNCH(swiglu_bf16x8_kernel<1>, b8, 256, 0, s, (const __nv_bfloat16*)gate_up, (__nv_bfloat16*)out, R,
+                       I, alternating);
+    } else if (dt == RFX_DT_BF16) {
+        RFX_GO(__nv_bfloat16);
+    } else {
         return RFX_ERR_BAD_ARG;
+    }
+#undef RFX_GO
     return 0;
+}
+
+extern "C" int rfx_swiglu(const void* gate_up, void* out, int dt, int R, int I, int alternating, void* stream) {
+    return rfx_gated_act(gate_up, out, dt, R, I, alternating, 0, stream);
 }
 
 extern "C" int rfx_add(float* a, const void* b, int b_dt, long long n, void* stream) {

@@ -103,9 +103,10 @@ struct Fuse {
 
 // The gated activation of EPI 1 (results rounded to bfloat16 take the fast exponential
 // and division, as `silu_mul_for` does).
-template <typename TO, bool CLAMPED>
+template <typename TO, int EPI>
 __device__ __forceinline__ float gated_act(float g, float u, const Fuse& f) {
-    if constexpr (CLAMPED) {
+    if constexpr (EPI == 7) return rfx::gelu_tanh_mul_for<TO>(g, u);
+    if constexpr (EPI == 4) {
         g = fminf(g, f.act_limit);
         u = fminf(fmaxf(u, -f.act_limit), f.act_limit);
         if constexpr (sizeof(TO) == 2) return __fdividef(g, 1.0f + __expf(-f.act_alpha * g)) * (u + 1.0f);
@@ -144,7 +145,8 @@ __device__ __forceinline__ float plain_out(float a, const Fuse& f) {
 // launch and no round trip of the [R, 2I] intermediate
 // (src/kernels_cuda/silu_and_mul.cu:7-23 is the reference's separate kernel).
 // EPI 4: the same with the clamped gated activation (`gated_act`), a template
-// instance of its own, so that EPI 1's instructions are what they were.
+// instance of its own, so that EPI 1's instructions are what they were.  EPI 7: the
+// same with the tanh form of gelu.
 using rfx::silu_mul;
 using rfx::silu_mul_for;
 
@@ -337,7 +339,7 @@ gemm_wt_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constant_
     const int kb0 = z * per;
     const int nkb = max(0, min(num_kb, kb0 + per) - kb0);
     // rows of the tile that each rank of a K-split cluster finishes
-    constexpr bool GATED = EPI == 1 || EPI == 4;  // rows alternate gate, up; the epilogue writes their activation
+    constexpr bool GATED = EPI == 1 || EPI == 4 || EPI == 7;  // rows alternate gate, up; the epilogue writes their activation
     constexpr bool PLAIN = EPI == 0 || EPI == 5 || EPI == 6;  // y = x W^T, EPI 5: y = max(x W^T, 0)^2, EPI 6: xielu of it
     const int mw = GATED ? ((((bm + ksplit - 1) / ksplit) + 1) & ~1) : (bm + ksplit - 1) / ksplit;
 
@@ -597,7 +599,7 @@ gemm_wt_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constant_
                             const float f = rstd_s[rr];
                             acc.x *= f, acc.y *= f, acc.z *= f, acc.w *= f;
                         }
-                        const float o0 = gated_act<TO, EPI == 4>(acc.x, acc.y, fuse), o1 = gated_act<TO, EPI == 4>(acc.z, acc.w, fuse);
+                        const float o0 = gated_act<TO, EPI>(acc.x, acc.y, fuse), o1 = gated_act<TO, EPI>(acc.z, acc.w, fuse);
                         if (!dry) store2(y + (size_t)r * (N / 2) + n / 2, o0, o1);
                     }
                 } else if (quads && EPI == 2 && BN <= 64) {
@@ -679,7 +681,7 @@ gemm_wt_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constant_
                         }
                         const int r = r0 + rr;
                         if (r < R && n0 + mm + 1 < N && !dry)
-                            rfx::st<TO>(y, (size_t)r * (N / 2) + (n0 + mm) / 2, gated_act<TO, EPI == 4>(g, u, fuse));
+                            rfx::st<TO>(y, (size_t)r * (N / 2) + (n0 + mm) / 2, gated_act<TO, EPI>(g, u, fuse));
                     }
                 } else {
                     for (int e = et; e < BN * mw; e += ET) {
@@ -741,7 +743,7 @@ gemm_wt_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constant_
                             const float got = __shfl_xor_sync(0xffffffffu, even ? a1 : a0, 1);
                             const float gate = even ? a0 : got, up = even ? got : a1;
                             const int r = r0 + c * 16 + j + (even ? 0 : 1);
-                            const float o = gated_act<TO, EPI == 4>(gate, up, fuse);
+                            const float o = gated_act<TO, EPI>(gate, up, fuse);
                             if (pair_ok && r < R) rfx::st<TO>(y, (size_t)r * (N / 2) + n / 2, o);
                         }
                     } else {
@@ -909,7 +911,7 @@ int launch(const void* x, const void* W, void* y, int R, int N, int K, int kspli
     const int num_kb = (K + BK - 1) / BK;
     Cut cut = choose_cut(N, r_tiles, num_kb, ksplit_req, EPI == 3, BN);
     if (EPI == 3 && (r_tiles != 1 || BN % cut.ks)) return RFX_ERR_UNSUPPORTED;
-    if ((EPI == 1 || EPI == 4) && (cut.bm & 1)) {  // pairs must not straddle tiles
+    if ((EPI == 1 || EPI == 4 || EPI == 7) && (cut.bm & 1)) {  // pairs must not straddle tiles
         cut.bm += 1;
         if (cut.bm > BM) return RFX_ERR_UNSUPPORTED;
         cut.tiles = (N + cut.bm - 1) / cut.bm;
@@ -1023,6 +1025,20 @@ extern "C" int rfx_gemm_bf16_tc_glu_clamped(const void* x, const void* W, void* 
     f.act_alpha = alpha;
     f.act_limit = limit;
     if (y_dt == RFX_DT_BF16) return dispatch<__nv_bfloat16, 4, false>(x, W, y, R, N, K, ksplit, f, nullptr, err, s);
+    return RFX_ERR_UNSUPPORTED;
+}
+
+// y [R, N / 2] = gelu(x W_gate^T) * (x W_up^T), gelu's tanh form, for W whose rows alternate gate_j,
+// up_j, as the product's epilogue, for a decode-sized batch (R <= 64).
+extern "C" int rfx_gemm_bf16_tc_geglu(const void* x, const void* W, void* y, int y_dt, int R, int N, int K,
+                                      int ksplit, int* err, void* stream) {
+    if (R <= 0 || N <= 0) return 0;
+    if (int c = check_common(x, W, R, N, K)) return c;
+    if (N & 1) return RFX_ERR_BAD_ARG;
+    if (R > 64) return RFX_ERR_UNSUPPORTED;
+    Fuse f{};
+    if (y_dt == RFX_DT_BF16)
+        return dispatch<__nv_bfloat16, 7, false>(x, W, y, R, N, K, ksplit, f, nullptr, err, (cudaStream_t)stream);
     return RFX_ERR_UNSUPPORTED;
 }
 

@@ -57,19 +57,20 @@ latent_post_kernel(const TI* __restrict__ proj, int stride, const float* __restr
 
 constexpr int TM = 64, TN = 64, TK = 16;
 
-// x [R, heads, K] (row stride ldx), W [heads, N, K], y [R, heads, N] (row stride ldy);
+// x [R, heads, K] (row stride ldx, head stride xh), W [heads, N, K], y [R, heads, N] (row
+// stride ldy, head stride yh);
 // scale [R, heads] or null.
 template <typename T, typename TO>
 __global__ void __launch_bounds__(256)
-heads_linear_kernel(const T* __restrict__ x, int ldx, const T* __restrict__ W, TO* __restrict__ y,
-                    int ldy, const float* __restrict__ scale, int R, int N, int K, int heads) {
+heads_linear_kernel(const T* __restrict__ x, int ldx, int xh, const T* __restrict__ W, TO* __restrict__ y,
+                    int ldy, int yh, const float* __restrict__ scale, int R, int N, int K, int heads) {
     __shared__ float xs[TK][TM + 1];
     __shared__ float ws[TK][TN + 1];
     pdl_prologue();
     const int b = blockIdx.z;
     const int r0 = blockIdx.y * TM, n0 = blockIdx.x * TN;
     const int tx = threadIdx.x % 16, ty = threadIdx.x / 16;
-    const T* xb = x + (size_t)b * K;
+    const T* xb = x + (size_t)b * xh;
     const T* wb = W + (size_t)b * N * K;
     float acc[4][4];
 #pragma unroll
@@ -108,7 +109,7 @@ heads_linear_kernel(const T* __restrict__ x, int ldx, const T* __restrict__ W, T
 #pragma unroll
         for (int j = 0; j < 4; ++j) {
             const int n = n0 + tx * 4 + j;
-            if (n < N) st<TO>(y + (size_t)r * ldy + (size_t)b * N, n, acc[i][j] * f);
+            if (n < N) st<TO>(y + (size_t)r * ldy + (size_t)b * yh, n, acc[i][j] * f);
         }
     }
 }
@@ -121,13 +122,13 @@ constexpr int GV_ROWS = 16;
 
 template <typename T, typename TO>
 __global__ void __launch_bounds__(256)
-heads_gemv_kernel(const T* __restrict__ x, int ldx, const T* __restrict__ W, TO* __restrict__ y, int ldy,
-                  const float* __restrict__ scale, int R, int N, int K, int heads) {
+heads_gemv_kernel(const T* __restrict__ x, int ldx, int xh, const T* __restrict__ W, TO* __restrict__ y, int ldy,
+                  int yh, const float* __restrict__ scale, int R, int N, int K, int heads) {
     extern __shared__ __align__(16) float xs[];  // [R][K]
     pdl_prologue();
     const int b = blockIdx.x;
     for (int e = threadIdx.x; e < R * K; e += blockDim.x)
-        xs[e] = ld<T>(x, (size_t)(e / K) * ldx + (size_t)b * K + e % K);
+        xs[e] = ld<T>(x, (size_t)(e / K) * ldx + (size_t)b * xh + e % K);
     __syncthreads();
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, nwarps = blockDim.x >> 5;
     const T* wb = W + (size_t)b * N * K;
@@ -168,7 +169,7 @@ heads_gemv_kernel(const T* __restrict__ x, int ldx, const T* __restrict__ W, TO*
         for (int r = 0; r < GV_ROWS; ++r) {
             if (r >= R) break;
             const float v = warp_sum(acc[r]);
-            if (lane == 0) st<TO>(y + (size_t)r * ldy + (size_t)b * N, n, v * (scale ? scale[(size_t)r * heads + b] : 1.0f));
+            if (lane == 0) st<TO>(y + (size_t)r * ldy + (size_t)b * yh, n, v * (scale ? scale[(size_t)r * heads + b] : 1.0f));
         }
     }
 }
@@ -205,10 +206,10 @@ extern "C" int rfx_latent_post(const void* proj, int in_dt, int ld, const float*
     return 0;
 }
 
-extern "C" int rfx_heads_linear(const void* x, int ldx, const void* W, void* y, int ldy, int dt,
+extern "C" int rfx_heads_linear(const void* x, int ldx, int xh, const void* W, void* y, int ldy, int yh, int dt,
                                 const float* scale, int R, int N, int K, int heads, void* stream) {
     if (R <= 0 || N <= 0 || heads <= 0) return 0;
-    if (K <= 0) return RFX_ERR_BAD_ARG;
+    if (K <= 0 || xh < K || yh < N) return RFX_ERR_BAD_ARG;
     cudaStream_t s = (cudaStream_t)stream;
     if (R <= GV_ROWS && (size_t)R * K * sizeof(float) <= 48 * 1024) {
         // a few rows: every weight is read once and meets all rows
@@ -217,11 +218,11 @@ extern "C" int rfx_heads_linear(const void* x, int ldx, const void* W, void* y, 
         dim3 g(heads, gy);
         const size_t smem = (size_t)R * K * sizeof(float);
         if (dt == RFX_DT_F32)
-            RFX_LAUNCH((heads_gemv_kernel<float, float>), g, 256, smem, s, (const float*)x, ldx, (const float*)W,
-                       (float*)y, ldy, scale, R, N, K, heads);
+            RFX_LAUNCH((heads_gemv_kernel<float, float>), g, 256, smem, s, (const float*)x, ldx, xh, (const float*)W,
+                       (float*)y, ldy, yh, scale, R, N, K, heads);
         else if (dt == RFX_DT_BF16)
             RFX_LAUNCH((heads_gemv_kernel<__nv_bfloat16, __nv_bfloat16>), g, 256, smem, s,
-                       (const __nv_bfloat16*)x, ldx, (const __nv_bfloat16*)W, (__nv_bfloat16*)y, ldy, scale, R, N,
+                       (const __nv_bfloat16*)x, ldx, xh, (const __nv_bfloat16*)W, (__nv_bfloat16*)y, ldy, yh, scale, R, N,
                        K, heads);
         else
             return RFX_ERR_BAD_ARG;
@@ -230,11 +231,11 @@ extern "C" int rfx_heads_linear(const void* x, int ldx, const void* W, void* y, 
     dim3 grid((N + TN - 1) / TN, (R + TM - 1) / TM, heads);
     if (grid.y > 65535 || grid.z > 65535) return RFX_ERR_UNSUPPORTED;
     if (dt == RFX_DT_F32)
-        RFX_LAUNCH((heads_linear_kernel<float, float>), grid, 256, 0, s, (const float*)x, ldx,
-                   (const float*)W, (float*)y, ldy, scale, R, N, K, heads);
+        RFX_LAUNCH((heads_linear_kernel<float, float>), grid, 256, 0, s, (const float*)x, ldx, xh,
+                   (const float*)W, (float*)y, ldy, yh, scale, R, N, K, heads);
     else if (dt == RFX_DT_BF16)
         RFX_LAUNCH((heads_linear_kernel<__nv_bfloat16, __nv_bfloat16>), grid, 256, 0, s,
-                   (const __nv_bfloat16*)x, ldx, (const __nv_bfloat16*)W, (__nv_bfloat16*)y, ldy, scale, R,
+                   (const __nv_bfloat16*)x, ldx, xh, (const __nv_bfloat16*)W, (__nv_bfloat16*)y, ldy, yh, scale, R,
                    N, K, heads);
     else
         return RFX_ERR_BAD_ARG;

@@ -6,11 +6,15 @@
 //     x <- x + mult * y * rsqrt(mean(y^2) + eps) * w_post
 //     out = x * rsqrt(mean(x^2) + eps) * w_next        (when w_next is given)
 // so the norm after one sublayer and the norm before the next are one pass over
-// the row.  A block a row; the row lives in shared memory between the sums of
+// the row.  Weights stored around zero come with an offset (w_post and w_next are taken
+// as offset + w).  Without w_next `out`, where given, is the new x itself in the product's
+// type (layers that norm only what a sublayer gives); with `fresh` x <- mult * norm(y) alone
+// (a normed embedding; y may be x).  A block a row; the row lives in shared memory between the sums of
 // squares and the outputs.
 //
 // group_norm_gate: x [R, C] 32-bit in `groups` equal parts, each over its own
-// root mean square, times w[c], times sigmoid(z[r, col + c]) when a gate is given.
+// root mean square, times w[c] (or a weight the parts share, `shared`), times
+// sigmoid(z[r, col + c]) or silu of it (`act` 1) when a gate is given.
 //
 // xielu: z > 0: ap z^2 + z / 2; else an (e^z - 1 - z) + z / 2, with ap and an given
 // (the softplus of the stored numbers is taken once, when the weights are bound).
@@ -26,9 +30,9 @@ using namespace rfx;
 
 template <typename TO>
 __global__ void __launch_bounds__(256)
-sandwich_norm_kernel(const float* __restrict__ y, float* __restrict__ x, const float* __restrict__ w_post,
-                     float mult, float eps, const float* __restrict__ w_next, float eps_next,
-                     TO* __restrict__ out, int H) {
+sandwich_norm_kernel(const float* y, float* x, const float* __restrict__ w_post,
+                     float post_offset, float mult, float eps, const float* __restrict__ w_next,
+                     float next_offset, float eps_next, TO* __restrict__ out, int fresh, int H) {
     extern __shared__ __align__(16) float row[];  // [H]
     __shared__ float scratch[32];
     pdl_prologue();
@@ -42,23 +46,24 @@ sandwich_norm_kernel(const float* __restrict__ y, float* __restrict__ x, const f
     const float r1 = 1.0f / sqrtf(block_sum(ss, scratch) / (float)H + eps);
     ss = 0.0f;
     for (int c = threadIdx.x; c < H; c += blockDim.x) {
-        const float v = fmaf(mult, (row[c] * r1) * w_post[c], x[base + c]);
+        const float v = fmaf(mult, (row[c] * r1) * (post_offset + w_post[c]), fresh ? 0.0f : x[base + c]);
         x[base + c] = v;
         row[c] = v;
         ss = fmaf(v, v, ss);
+        if (w_next == nullptr && out) st<TO>(out, base + c, v);
     }
     if (w_next == nullptr) return;
     const float r2 = 1.0f / sqrtf(block_sum(ss, scratch) / (float)H + eps_next);
-    for (int c = threadIdx.x; c < H; c += blockDim.x) st<TO>(out, base + c, (row[c] * r2) * w_next[c]);
+    for (int c = threadIdx.x; c < H; c += blockDim.x) st<TO>(out, base + c, (row[c] * r2) * (next_offset + w_next[c]));
 }
 
 // The same with 16-byte accesses, for widths that are a multiple of four: the row stays in
 // registers (up to V groups of four a thread) between the sums of squares and the outputs.
 template <typename TO, int V>
 __global__ void __launch_bounds__(512)
-sandwich_norm4_kernel(const float* __restrict__ y, float* __restrict__ x, const float* __restrict__ w_post,
-                      float mult, float eps, const float* __restrict__ w_next, float eps_next,
-                      TO* __restrict__ out, int H) {
+sandwich_norm4_kernel(const float* y, float* x, const float* __restrict__ w_post,
+                      float post_offset, float mult, float eps, const float* __restrict__ w_next,
+                      float next_offset, float eps_next, TO* __restrict__ out, int fresh, int H) {
     __shared__ float scratch[32];
     pdl_prologue();
     const size_t base = (size_t)blockIdx.x * H;
@@ -73,7 +78,7 @@ sandwich_norm4_kernel(const float* __restrict__ y, float* __restrict__ x, const 
         const int c = threadIdx.x + i * blockDim.x;
         if (c < H4) {
             v[i] = y4[c];
-            xv[i] = x4[c];
+            xv[i] = fresh ? make_float4(0.0f, 0.0f, 0.0f, 0.0f) : x4[c];
             wp[i] = wp4[c];
             ss = fmaf(v[i].x, v[i].x, fmaf(v[i].y, v[i].y, fmaf(v[i].z, v[i].z, fmaf(v[i].w, v[i].w, ss))));
         }
@@ -84,11 +89,12 @@ sandwich_norm4_kernel(const float* __restrict__ y, float* __restrict__ x, const 
     for (int i = 0; i < V; ++i) {
         const int c = threadIdx.x + i * blockDim.x;
         if (c < H4) {
-            v[i].x = fmaf(mult, (v[i].x * r1) * wp[i].x, xv[i].x);
-            v[i].y = fmaf(mult, (v[i].y * r1) * wp[i].y, xv[i].y);
-            v[i].z = fmaf(mult, (v[i].z * r1) * wp[i].z, xv[i].z);
-            v[i].w = fmaf(mult, (v[i].w * r1) * wp[i].w, xv[i].w);
+            v[i].x = fmaf(mult, (v[i].x * r1) * (post_offset + wp[i].x), xv[i].x);
+            v[i].y = fmaf(mult, (v[i].y * r1) * (post_offset + wp[i].y), xv[i].y);
+            v[i].z = fmaf(mult, (v[i].z * r1) * (post_offset + wp[i].z), xv[i].z);
+            v[i].w = fmaf(mult, (v[i].w * r1) * (post_offset + wp[i].w), xv[i].w);
             x4[c] = v[i];
+            if (w_next == nullptr && out) store4(out + base + 4 * (size_t)c, v[i]);
             ss = fmaf(v[i].x, v[i].x, fmaf(v[i].y, v[i].y, fmaf(v[i].z, v[i].z, fmaf(v[i].w, v[i].w, ss))));
         }
     }
@@ -100,10 +106,17 @@ sandwich_norm4_kernel(const float* __restrict__ y, float* __restrict__ x, const 
         const int c = threadIdx.x + i * blockDim.x;
         if (c < H4) {
             const float4 wn = wn4[c];
-            store4(out + base + 4 * (size_t)c, make_float4((v[i].x * r2) * wn.x, (v[i].y * r2) * wn.y,
-                                                           (v[i].z * r2) * wn.z, (v[i].w * r2) * wn.w));
+            store4(out + base + 4 * (size_t)c,
+                   make_float4((v[i].x * r2) * (next_offset + wn.x), (v[i].y * r2) * (next_offset + wn.y),
+                               (v[i].z * r2) * (next_offset + wn.z), (v[i].w * r2) * (next_offset + wn.w)));
         }
     }
+}
+
+// sigmoid(t), or (act 1) silu(t)
+__device__ __forceinline__ float gate_of(float t, int act) {
+    const float s = 1.0f / (1.0f + exact_expf(-t));
+    return act ? t * s : s;
 }
 
 // One block a (row, part), 16 bytes an access: parts of many elements (a norm in a few equal
@@ -111,13 +124,14 @@ sandwich_norm4_kernel(const float* __restrict__ y, float* __restrict__ x, const 
 template <typename TO>
 __global__ void __launch_bounds__(256)
 group_norm_gate_wide_kernel(const float* __restrict__ x, const float* __restrict__ w, float eps,
-                            const float* __restrict__ z, int ldz, int zcol, TO* __restrict__ out, int C, int gs) {
+                            const float* __restrict__ z, int ldz, int zcol, int act, int shared,
+                            TO* __restrict__ out, int C, int gs) {
     __shared__ float scratch[32];
     pdl_prologue();
     const int r = blockIdx.x, g = blockIdx.y;
     const size_t base = (size_t)r * C + (size_t)g * gs;
     const float4* x4 = reinterpret_cast<const float4*>(x + base);
-    const float4* w4 = reinterpret_cast<const float4*>(w + (size_t)g * gs);
+    const float4* w4 = reinterpret_cast<const float4*>(shared ? w : w + (size_t)g * gs);
     float ss = 0.0f;
     for (int c = threadIdx.x; c < gs / 4; c += blockDim.x) {
         const float4 v = x4[c];
@@ -129,10 +143,10 @@ group_norm_gate_wide_kernel(const float* __restrict__ x, const float* __restrict
         float4 o = make_float4((v.x * rs) * wv.x, (v.y * rs) * wv.y, (v.z * rs) * wv.z, (v.w * rs) * wv.w);
         if (z) {
             const float* zp = z + (size_t)r * ldz + zcol + (size_t)g * gs + 4 * c;
-            o.x *= 1.0f / (1.0f + exact_expf(-zp[0]));
-            o.y *= 1.0f / (1.0f + exact_expf(-zp[1]));
-            o.z *= 1.0f / (1.0f + exact_expf(-zp[2]));
-            o.w *= 1.0f / (1.0f + exact_expf(-zp[3]));
+            o.x *= gate_of(zp[0], act);
+            o.y *= gate_of(zp[1], act);
+            o.z *= gate_of(zp[2], act);
+            o.w *= gate_of(zp[3], act);
         }
         store4(out + base + 4 * (size_t)c, o);
     }
@@ -141,7 +155,8 @@ group_norm_gate_wide_kernel(const float* __restrict__ x, const float* __restrict
 template <typename TO>
 __global__ void __launch_bounds__(256)
 group_norm_gate_kernel(const float* __restrict__ x, const float* __restrict__ w, float eps,
-                       const float* __restrict__ z, int ldz, int zcol, TO* __restrict__ out, int C, int groups) {
+                       const float* __restrict__ z, int ldz, int zcol, int act, int shared, TO* __restrict__ out,
+                       int C, int groups) {
     pdl_prologue();
     const int r = blockIdx.x;
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, nwarps = blockDim.x >> 5;
@@ -153,10 +168,10 @@ group_norm_gate_kernel(const float* __restrict__ x, const float* __restrict__ w,
         for (int c = lane; c < gs; c += 32) ss = fmaf(xr[c], xr[c], ss);
         const float rs = 1.0f / sqrtf(warp_sum(ss) / (float)gs + eps);
         for (int c = lane; c < gs; c += 32) {
-            float v = (xr[c] * rs) * w[g * gs + c];
+            float v = (xr[c] * rs) * w[shared ? c : g * gs + c];
             if (z) {
                 const float t = z[(size_t)r * ldz + zcol + g * gs + c];
-                v *= 1.0f / (1.0f + exact_expf(-t));
+                v *= gate_of(t, act);
             }
             st<TO>(out, (size_t)r * C + (size_t)g * gs + c, v);
         }
@@ -207,9 +222,9 @@ inline int blocks_for(size_t n, int threads) {
 
 }  // namespace
 
-extern "C" int rfx_sandwich_norm(const float* y, float* x, const float* w_post, float mult, float eps,
-                                 const float* w_next, float eps_next, void* out, int out_dt, int R, int H,
-                                 void* stream) {
+extern "C" int rfx_sandwich_norm(const float* y, float* x, const float* w_post, float post_offset, float mult,
+                                 float eps, const float* w_next, float next_offset, float eps_next, void* out,
+                                 int out_dt, int fresh, int R, int H, void* stream) {
     if (R <= 0) return 0;
     const size_t smem = (size_t)H * sizeof(float);
     if (smem > 200 * 1024) return RFX_ERR_UNSUPPORTED;
@@ -221,8 +236,8 @@ extern "C" int rfx_sandwich_norm(const float* y, float* x, const float* w_post, 
         const int H4 = H / 4;
         const int threads = H4 <= 128 ? 128 : H4 <= 256 ? 256 : 512;
 #define RFX_V(TO, V)                                                                                           \
-    RFX_LAUNCH((sandwich_norm4_kernel<TO, V>), R, threads, 0, s, y, x, w_post, mult, eps, w_next, eps_next,   \
-               (TO*)out, H)
+    RFX_LAUNCH((sandwich_norm4_kernel<TO, V>), R, threads, 0, s, y, x, w_post, post_offset, mult, eps, w_next, \
+               next_offset, eps_next, (TO*)out, fresh, H)
 #define RFX_PICK(TO)                                      \
     do {                                                  \
         if (H4 <= threads) RFX_V(TO, 1);                  \
@@ -243,8 +258,8 @@ extern "C" int rfx_sandwich_norm(const float* y, float* x, const float* w_post, 
                                                  cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);   \
             if (e != cudaSuccess) return (int)e;                                                            \
         }                                                                                                   \
-        RFX_LAUNCH(sandwich_norm_kernel<TO>, R, 256, smem, s, y, x, w_post, mult, eps, w_next, eps_next,    \
-                   (TO*)out, H);                                                                            \
+        RFX_LAUNCH(sandwich_norm_kernel<TO>, R, 256, smem, s, y, x, w_post, post_offset, mult, eps, w_next, \
+                   next_offset, eps_next, (TO*)out, fresh, H);                                                                           \
     } while (0)
     if (out_dt == RFX_DT_F32) RFX_GO(float);
     else if (out_dt == RFX_DT_BF16) RFX_GO(__nv_bfloat16);
@@ -254,7 +269,8 @@ extern "C" int rfx_sandwich_norm(const float* y, float* x, const float* w_post, 
 }
 
 extern "C" int rfx_group_norm_gate(const float* x, const float* w, float eps, const float* z, int ldz, int zcol,
-                                   void* out, int out_dt, int R, int C, int groups, void* stream) {
+                                   int act, int shared, void* out, int out_dt, int R, int C, int groups,
+                                   void* stream) {
     if (R <= 0) return 0;
     if (groups <= 0 || C % groups) return RFX_ERR_BAD_ARG;
     cudaStream_t s = (cudaStream_t)stream;
@@ -263,9 +279,10 @@ extern "C" int rfx_group_norm_gate(const float* x, const float* w, float eps, co
     if (gs >= 512 && gs % 4 == 0 && C % 4 == 0 && al && groups <= 65535) {
         dim3 grid(R, groups);
         if (out_dt == RFX_DT_F32)
-            RFX_LAUNCH(group_norm_gate_wide_kernel<float>, grid, 256, 0, s, x, w, eps, z, ldz, zcol, (float*)out, C, gs);
+            RFX_LAUNCH(group_norm_gate_wide_kernel<float>, grid, 256, 0, s, x, w, eps, z, ldz, zcol, act, shared,
+                       (float*)out, C, gs);
         else if (out_dt == RFX_DT_BF16)
-            RFX_LAUNCH(group_norm_gate_wide_kernel<__nv_bfloat16>, grid, 256, 0, s, x, w, eps, z, ldz, zcol,
+            RFX_LAUNCH(group_norm_gate_wide_kernel<__nv_bfloat16>, grid, 256, 0, s, x, w, eps, z, ldz, zcol, act, shared,
                        (__nv_bfloat16*)out, C, gs);
         else return RFX_ERR_BAD_ARG;
         return 0;
@@ -275,9 +292,10 @@ extern "C" int rfx_group_norm_gate(const float* x, const float* w, float eps, co
     if (gy > 65535) gy = 65535;
     dim3 grid(R, gy);
     if (out_dt == RFX_DT_F32)
-        RFX_LAUNCH(group_norm_gate_kernel<float>, grid, threads, 0, s, x, w, eps, z, ldz, zcol, (float*)out, C, groups);
+        RFX_LAUNCH(group_norm_gate_kernel<float>, grid, threads, 0, s, x, w, eps, z, ldz, zcol, act, shared,
+                   (float*)out, C, groups);
     else if (out_dt == RFX_DT_BF16)
-        RFX_LAUNCH(group_norm_gate_kernel<__nv_bfloat16>, grid, threads, 0, s, x, w, eps, z, ldz, zcol,
+        RFX_LAUNCH(group_norm_gate_kernel<__nv_bfloat16>, grid, threads, 0, s, x, w, eps, z, ldz, zcol, act, shared,
                    (__nv_bfloat16*)out, C, groups);
     else return RFX_ERR_BAD_ARG;
     return 0;

@@ -17,6 +17,7 @@ from .. import ops
 from ..cache.specs import KVSpec, StateSpec
 from ..config.spec import ModelSpec, RunEntry
 from ..config.spec import names_dict
+from ..parts.block import PostNormBlock, ReadyRows
 from ..parts.registry import BLOCKS, EMBEDDING_TERMS, NORMS, TensorInfo
 
 
@@ -29,6 +30,9 @@ class RunContext:
     kv: Any = None             # KVView of this run's cache entry, if it has one
     state: Any = None          # [slots, *shape] tensor of this run's state, if any
     entry: int = -1
+    # what runs of one step leave for later runs of it (a layer's values that later layers
+    # mix into theirs): rows that live as long as the step
+    shared: Any = None
     # a mixer whose `cache_spec()` is a tuple: its views, in the tuple's order
     # (`kv` and `state` are then the first of each kind)
     parts: Any = None
@@ -38,6 +42,9 @@ def expected_tensors(spec: ModelSpec) -> Dict[str, Tuple[Tuple[str, ...], Tensor
     """tensor name -> (where it goes, TensorInfo) for the whole model."""
     out: Dict[str, Tuple[Tuple[str, ...], TensorInfo]] = {}
     out[spec.embedding_name] = (("embedding",), TensorInfo((spec.vocab_size, spec.hidden_size), "table"))
+    if spec.embedding_norm is not None:
+        out[spec.embedding_norm_name] = (("embedding_norm",), NORMS.get(spec.embedding_norm.kind).tensor_specs(
+            spec.embedding_norm)["weight"])
     for ti, term in enumerate(spec.embedding_terms):
         names = names_dict(term.names)
         for role, info in EMBEDDING_TERMS.get(term.kind).tensor_specs(term).items():
@@ -64,6 +71,11 @@ class CausalLM:
         self.device = torch.device(device)
         self.layers = [BLOCKS.get(l.block)(l, dtype, self.device) for l in spec.layers]
         self.final_norm = NORMS.get(spec.final_norm.kind)(spec.final_norm, dtype, self.device)
+        self.embedding_norm = None
+        if spec.embedding_norm is not None:
+            if spec.embedding_norm.kind != "rmsnorm":
+                raise ValueError("the embedding's norm must be an RMS norm")
+            self.embedding_norm = NORMS.get(spec.embedding_norm.kind)(spec.embedding_norm, dtype, self.device)
         self.embedding_terms = [EMBEDDING_TERMS.get(t.kind)(t, dtype, self.device) for t in spec.embedding_terms]
         self.embedding: Optional[torch.Tensor] = None
         self.head: Optional[torch.Tensor] = None
@@ -102,6 +114,8 @@ class CausalLM:
                 self.embedding = t.to(device=self.device, dtype=self.dtype).contiguous()
             elif where[0] == "head":
                 self.head = t.to(device=self.device, dtype=self.dtype).contiguous()
+            elif where[0] == "embedding_norm":
+                self.embedding_norm.bind({"weight": t})
             elif where[0] == "final_norm":
                 self.final_norm.bind({"weight": t})
             elif where[0] == "stream_mix":
@@ -150,6 +164,13 @@ class CausalLM:
         # gives a zero row and sets the device's error word, which `check_errors` reads
         h = ops.embed(self.embedding, batch.tokens, self.spec.embedding_scale,
                       ops.device_error_word(self.device))
+        pending = None
+        if self.embedding_norm is not None:
+            # the stream starts normed; a first block that reads the stream itself gets its rows too
+            n, first = self.embedding_norm, self.layers[self.spec.run_order[0].layer]
+            reads = isinstance(first, PostNormBlock) and not self.embedding_terms
+            x = ops.post_norm(h, h, n.weight, n.spec.weight_offset, n.spec.eps, self.dtype if reads else None, fresh=True)
+            pending = ReadyRows(x) if x is not None else None
         for ti, term in enumerate(self.embedding_terms):
             entry = self.term_entry(ti)
             term.add(h, batch, cache.state(entry) if cache.has(entry) == "state" else None)
@@ -157,7 +178,7 @@ class CausalLM:
             # the residual as several parallel copies: the embedding output into each
             h = ops.hyper_expand(h, self.spec.residual_streams)
         ops.prof_mark("embed")
-        pending = None
+        shared: Dict[str, Any] = {}
         order = self.spec.run_order
         # the embedding output, for the runs that start from a mix of it and the stream
         x0 = ops.keep_copy(h) if any(r.mixes_input or r.adds_input for r in order) else None
@@ -188,7 +209,7 @@ class CausalLM:
                 pending = None
                 ops.loop_input_(h, x0 if run.adds_input else None, self.pass_vectors[run.pass_vector])
                 ops.prof_mark("stream_mix")
-            ctx = RunContext(batch=batch, writes_cache=run.writes_cache, entry=run.cache)
+            ctx = RunContext(batch=batch, writes_cache=run.writes_cache, entry=run.cache, shared=shared)
             kind = cache.has(run.cache)
             if kind == "kv":
                 ctx.kv = cache.kv(run.cache)

@@ -95,16 +95,19 @@ def add_(a: torch.Tensor, b: torch.Tensor) -> torch.Tensor:
     return a
 
 
-def swiglu(gate_up: torch.Tensor, alternating: bool = False) -> torch.Tensor:
-    """[R, 2I] -> silu(gate) * up, [R, I].  A row holds the gates in its first
+GATED_ACTIVATIONS = {"silu": 0, "gelu_tanh": 1}
+
+
+def swiglu(gate_up: torch.Tensor, alternating: bool = False, activation: str = "silu") -> torch.Tensor:
+    """[R, 2I] -> act(gate) * up, [R, I], act silu or the tanh form of gelu.  A row holds the gates in its first
     half and the ups in its second, or (`alternating`) gate_i at 2i and up_i at
     2i + 1."""
     R, two_i = gate_up.shape
     I = two_i // 2
     out = _new((R, I), gate_up.dtype, gate_up.device)
-    st = native.lib().rfx_swiglu(_chk(gate_up, "gate_up"), out.data_ptr(), dt_code(gate_up.dtype),
-                                 R, I, 1 if alternating else 0, _stream())
-    native.check(st, "swiglu")
+    st = native.lib().rfx_gated_act(_chk(gate_up, "gate_up"), out.data_ptr(), dt_code(gate_up.dtype),
+                                    R, I, 1 if alternating else 0, GATED_ACTIVATIONS[activation], _stream())
+    native.check(st, f"gated_act ({activation})")
     return out
 
 
@@ -373,6 +376,26 @@ def linear_swiglu(x: torch.Tensor, weight_pairs: torch.Tensor) -> torch.Tensor:
     return swiglu(linear(x, weight_pairs), alternating=True)
 
 
+def linear_geglu(x: torch.Tensor, weight_pairs: torch.Tensor) -> torch.Tensor:
+    """gelu(x @ gate.T) * (x @ up.T), gelu's tanh form, for a weight whose rows
+    alternate gate_j, up_j; [R, I] in x's dtype.  For a few bfloat16 rows the
+    activation is the product kernel's epilogue; otherwise product, then the
+    activation kernel."""
+    R, K = x.shape
+    if (x.dtype == torch.bfloat16 and R <= GEMV_MAX_ROWS and K % 8 == 0 and FUSE_GLU
+            and (x.data_ptr() | weight_pairs.data_ptr()) % 16 == 0):
+        N = weight_pairs.shape[0]
+        _chk(x, "x", torch.bfloat16)
+        _chk(weight_pairs, "weight", torch.bfloat16)
+        y = _new((R, N // 2), torch.bfloat16, x.device)
+        st = native.lib().rfx_gemm_bf16_tc_geglu(
+            x.data_ptr(), weight_pairs.data_ptr(), y.data_ptr(), BF16, R, N, K, 0,
+            device_error_word(x.device).data_ptr(), _stream())
+        native.check(st, f"gemm_bf16_tc_geglu (R={R}, N={N}, K={K})")
+        return y
+    return swiglu(linear(x, weight_pairs), alternating=True, activation="gelu_tanh")
+
+
 # ----------------------------------------------------------------- attention
 def qkv_post(qkv: torch.Tensor, q_weight, k_weight, eps: float, weight_offset: float,
              rotation, row_pos: torch.Tensor, row_slot: torch.Tensor,
@@ -479,8 +502,9 @@ def attention_plain(q: torch.Tensor, k_pages: torch.Tensor, v_pages: torch.Tenso
                     row_slot: torch.Tensor, nq: int, nkv: int, head_dim: int,
                     window: Optional[int], scale: float,
                     sink: Optional[torch.Tensor] = None,
-                    slopes: Optional[torch.Tensor] = None, keep_first: int = 0) -> torch.Tensor:
-    """`keep_first`: with a window, the first so many positions of a sequence
+                    slopes: Optional[torch.Tensor] = None, keep_first: int = 0,
+                    softcap: float = 0.0) -> torch.Tensor:
+    """`softcap` > 0: a score s becomes softcap * tanh(s / softcap).  `keep_first`: with a window, the first so many positions of a sequence
     stay visible beyond it.  `sink` (float32, one per query head): exp(sink) joins the softmax's
     denominator once, with no key and no value.  `slopes` (float32, one per
     query head): slope * (query position - key position) is taken off every
@@ -492,7 +516,7 @@ def attention_plain(q: torch.Tensor, k_pages: torch.Tensor, v_pages: torch.Tenso
         dt_code(q.dtype), _chk(page_table, "page_table", torch.int32), page_table.shape[1],
         page_size, _chk(row_pos, "row_pos", torch.int32), _chk(row_slot, "row_slot", torch.int32),
         out.data_ptr(), R, nq, nkv, head_dim, int(window or 0), int(keep_first if window else 0), float(scale),
-        _chk(sink, "sink", torch.float32), _chk(slopes, "slopes", torch.float32), _stream())
+        _chk(sink, "sink", torch.float32), _chk(slopes, "slopes", torch.float32), float(softcap), _stream())
     native.check(st, f"attention_plain (head_dim={head_dim})")
     return out
 
@@ -563,7 +587,8 @@ def decode_splits(n_rows: int, nq: int, nkv: int, max_pages: int = 64) -> int:
 def attention_decode(q, k_pages, v_pages, page_table, page_size, row_pos, row_slot, nq, nkv,
                      head_dim, window, scale, n_splits: Optional[int] = None,
                      sink: Optional[torch.Tensor] = None,
-                     slopes: Optional[torch.Tensor] = None, keep_first: int = 0) -> torch.Tensor:
+                     slopes: Optional[torch.Tensor] = None, keep_first: int = 0,
+                     softcap: float = 0.0) -> torch.Tensor:
     """bfloat16 tensor-core attention for rows that are each one query
     position (decode), split over the keys."""
     keep_first = int(keep_first) if window else 0
@@ -583,7 +608,7 @@ def attention_decode(q, k_pages, v_pages, page_table, page_size, row_pos, row_sl
             _chk(page_table, "page_table", torch.int32), page_table.shape[1], page_size,
             _chk(row_pos, "row_pos", torch.int32), _chk(row_slot, "row_slot", torch.int32), out.data_ptr(), 0,
             R, nq, nkv, head_dim, n_splits, int(window or 0), keep_first, float(scale),
-            _chk(sink, "sink", torch.float32), _chk(slopes, "slopes", torch.float32), pool_pages, 1,
+            _chk(sink, "sink", torch.float32), _chk(slopes, "slopes", torch.float32), float(softcap), pool_pages, 1,
             device_error_word(q.device).data_ptr(), _stream())
         if st != native.ERR_UNSUPPORTED:
             native.check(st, f"attention_decode_cluster (head_dim={head_dim}, splits={n_splits})")
@@ -595,7 +620,7 @@ def attention_decode(q, k_pages, v_pages, page_table, page_size, row_pos, row_sl
         _chk(row_pos, "row_pos", torch.int32), _chk(row_slot, "row_slot", torch.int32), out.data_ptr(),
         partial.data_ptr() if partial is not None else 0, R, nq, nkv, head_dim, n_splits,
         int(window or 0), keep_first, float(scale), _chk(sink, "sink", torch.float32),
-        _chk(slopes, "slopes", torch.float32), pool_pages, 0, device_error_word(q.device).data_ptr(), _stream())
+        _chk(slopes, "slopes", torch.float32), float(softcap), pool_pages, 0, device_error_word(q.device).data_ptr(), _stream())
     native.check(st, f"attention_decode (head_dim={head_dim}, splits={n_splits})")
     return out
 
@@ -605,7 +630,7 @@ CLUSTER_MERGE = _env_flag("REFLEX_B200_CLUSTER_MERGE", True)
 
 def attention_prefill(q, k_pages, v_pages, page_table, page_size, seq_slot, seq_start, seq_new,
                       seq_row0, max_new: int, nq, nkv, head_dim, window, scale, sink=None,
-                      slopes=None, keep_first: int = 0) -> torch.Tensor:
+                      slopes=None, keep_first: int = 0, softcap: float = 0.0) -> torch.Tensor:
     """bfloat16 tensor-core attention for a packed batch of sequences that
     each bring one or more rows (prefill, chunks, mixed steps)."""
     _chk(q, "q", torch.bfloat16)
@@ -621,16 +646,19 @@ def attention_prefill(q, k_pages, v_pages, page_table, page_size, seq_slot, seq_
         _chk(seq_slot, "seq_slot", torch.int32), _chk(seq_start, "seq_start", torch.int32),
         _chk(seq_new, "seq_new", torch.int32), _chk(seq_row0, "seq_row0", torch.int32), out.data_ptr(),
         S, int(max_new), nq, nkv, head_dim, int(window or 0), int(keep_first) if window else 0, float(scale),
-        _chk(sink, "sink", torch.float32), _chk(slopes, "slopes", torch.float32), _stream())
+        _chk(sink, "sink", torch.float32), _chk(slopes, "slopes", torch.float32), float(softcap), _stream())
     native.check(st, f"attention_prefill (head_dim={head_dim})")
     return out
 
 
 def attention_prefill_tc(q, k_pages, v_pages, page_table, page_size, seq_slot, seq_start, seq_new,
                          seq_row0, max_new: int, nq, nkv, head_dim, window, scale, sink=None,
-                         slopes=None, keep_first: int = 0) -> torch.Tensor:
+                         slopes=None, keep_first: int = 0, softcap: float = 0.0,
+                         score_bound: float = 0.0) -> torch.Tensor:
     """The tcgen05/TMEM form of `attention_prefill`, for head sizes 64 and 128
-    (with `slopes` the scale must be positive)."""
+    (the scale must be positive).  `score_bound` > 0: no scaled score is larger
+    (queries and keys of known length); with a cap twice that, its tanh is a
+    polynomial."""
     _chk(q, "q", torch.bfloat16)
     if head_dim not in (64, 128):
         raise InvalidInput(f"attention_prefill_tc takes head_dim 64 or 128, got {head_dim}")
@@ -644,20 +672,22 @@ def attention_prefill_tc(q, k_pages, v_pages, page_table, page_size, seq_slot, s
         _chk(seq_new, "seq_new", torch.int32), _chk(seq_row0, "seq_row0", torch.int32), out.data_ptr(),
         seq_slot.numel(), int(max_new), q.shape[0], nq, nkv, head_dim, int(window or 0),
         int(keep_first) if window else 0, float(scale),
-        _chk(sink, "sink", torch.float32), _chk(slopes, "slopes", torch.float32),
+        _chk(sink, "sink", torch.float32), _chk(slopes, "slopes", torch.float32), float(softcap), float(score_bound),
         device_error_word(q.device).data_ptr(), _stream())
     native.check(st, f"attention_prefill_tc (head_dim={head_dim})")
     return out
 
 
 def attention(q, k_pages, v_pages, page_table, page_size, batch, nq, nkv, head_dim, window, scale,
-              sink=None, slopes=None, keep_first: int = 0):
+              sink=None, slopes=None, keep_first: int = 0, softcap: float = 0.0, score_bound: float = 0.0):
     """Attention of the step's rows over their sequences' cached keys and
     values; picks the kernel for the dtype and the kind of step.  `sink`: one
     float32 per query head whose exponential joins the softmax's denominator.
     `slopes`: one float32 per query head; slope * (query position - key
     position) is taken off every score.  `keep_first`: with a window, the first
-    so many positions of a sequence stay visible beyond it."""
+    so many positions of a sequence stay visible beyond it.  `softcap` > 0: a score
+    s becomes softcap * tanh(s / softcap) before the softmax; `score_bound` > 0: the
+    caller knows that no |s| is larger."""
     fast = q.dtype == torch.bfloat16 and head_dim % 16 == 0 and head_dim <= 256
     keep_first = int(keep_first) if window else 0
     if fast and batch.is_decode:
@@ -666,17 +696,17 @@ def attention(q, k_pages, v_pages, page_table, page_size, batch, nq, nkv, head_d
         return attention_decode(q, k_pages, v_pages, page_table, page_size, batch.row_pos,
                                 batch.row_slot, nq, nkv, head_dim, window, scale,
                                 n_splits=decode_splits(q.shape[0], nq, nkv, pages), sink=sink, slopes=slopes,
-                                keep_first=keep_first)
+                                keep_first=keep_first, softcap=softcap)
     if fast and nq // nkv <= 128 and head_dim in (64, 128) and scale > 0:
         return attention_prefill_tc(q, k_pages, v_pages, page_table, page_size, batch.seq_slot,
                                     batch.seq_start, batch.seq_new, batch.seq_row0, batch.max_new, nq,
-                                    nkv, head_dim, window, scale, sink, slopes, keep_first)
+                                    nkv, head_dim, window, scale, sink, slopes, keep_first, softcap, score_bound)
     if fast and nq // nkv <= 128:
         return attention_prefill(q, k_pages, v_pages, page_table, page_size, batch.seq_slot,
                                  batch.seq_start, batch.seq_new, batch.seq_row0, batch.max_new, nq,
-                                 nkv, head_dim, window, scale, sink, slopes, keep_first)
+                                 nkv, head_dim, window, scale, sink, slopes, keep_first, softcap)
     return attention_plain(q, k_pages, v_pages, page_table, page_size, batch.row_pos,
-                           batch.row_slot, nq, nkv, head_dim, window, scale, sink, slopes, keep_first)
+                           batch.row_slot, nq, nkv, head_dim, window, scale, sink, slopes, keep_first, softcap)
 
 
 # ------------------------------------------------- further norms and embedding terms
@@ -755,41 +785,44 @@ HEADS_LINEAR_MAX_ROWS = _env_int("REFLEX_B200_HEADS_LINEAR_MAX_ROWS", 64, 0, 1 <
 
 
 def heads_linear(x: torch.Tensor, weight: torch.Tensor, scale: Optional[torch.Tensor] = None,
-                 out_dtype: Optional[torch.dtype] = None) -> torch.Tensor:
-    """y[r, b, :] = x[r, b, :] @ weight[b].T for every head b: x [R, heads * K],
-    weight [heads, N, K], y [R, heads * N]; with `scale` (float32 [R, heads])
-    y[r, b, :] is multiplied by scale[r, b].  float32 and a few bfloat16 rows:
-    this library's kernel (32-bit accumulation in index order); more bfloat16
-    rows: the library's batched product, then the scaling kernel.  `out_dtype`
-    float32 with bfloat16 operands (many rows only): the batched product's
-    32-bit sums come out unrounded."""
+                 out_dtype: Optional[torch.dtype] = None, out: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """y[r, b, :] = x[r, b, :K] @ weight[b].T for every head b: x [R, heads * xh] with
+    xh >= K elements a head (the first K are read), weight [heads, N, K], y [R, heads
+    * N]; with `scale` (float32 [R, heads]) y[r, b, :] is multiplied by scale[r, b].
+    `out` [R, heads * yh], yh >= N: the results go into the first N elements of each of
+    its heads.  float32 and a few bfloat16 rows: this library's kernel (32-bit
+    accumulation in index order); more bfloat16 rows: the library's batched product,
+    then the scaling kernel.  `out_dtype` float32 with bfloat16 operands (many rows
+    only): the batched product's 32-bit sums come out unrounded."""
     heads, N, K = weight.shape
     R = x.shape[0]
-    if x.shape[1] != heads * K or x.dtype != weight.dtype:
-        raise InvalidInput("heads_linear: x must be [rows, heads * K] in the weight's dtype")
+    xh = x.shape[1] // heads
+    if x.shape[1] != heads * xh or xh < K or x.dtype != weight.dtype:
+        raise InvalidInput("heads_linear: x must be [rows, heads * (K or more)] in the weight's dtype")
     _chk(x, "x")
     _chk(weight, "weight")
     wide = out_dtype == torch.float32 and x.dtype == torch.bfloat16
     if wide and R <= HEADS_LINEAR_MAX_ROWS:
         raise InvalidInput("heads_linear: 32-bit results of bfloat16 operands need more rows than its own kernel takes")
-    y = _new((R, heads * N), torch.float32 if wide else x.dtype, x.device)
-    if wide:
-        torch.bmm(x.view(R, heads, K).transpose(0, 1), weight.transpose(1, 2), out_dtype=torch.float32,
-                  out=y.view(R, heads, N).transpose(0, 1))
-        if scale is not None:
-            st = native.lib().rfx_scale_heads(y.data_ptr(), dt_code(y.dtype), _chk(scale, "scale", torch.float32),
-                                              y.numel(), N, _stream())
-            native.check(st, "scale_heads")
-        return y
+    y = _new((R, heads * N), torch.float32 if wide else x.dtype, x.device) if out is None else out
+    yh = y.shape[1] // heads
+    if y.shape[0] != R or y.shape[1] != heads * yh or yh < N or (out is not None and (wide or y.dtype != x.dtype)):
+        raise InvalidInput("heads_linear: out must be [rows, heads * (N or more)] in x's dtype")
     if x.dtype == torch.bfloat16 and R > HEADS_LINEAR_MAX_ROWS:
-        torch.bmm(x.view(R, heads, K).transpose(0, 1), weight.transpose(1, 2),
-                  out=y.view(R, heads, N).transpose(0, 1))
+        if scale is not None and yh != N:
+            raise InvalidInput("heads_linear: a scale goes with heads of N elements")
+        args = (x.view(R, heads, xh)[:, :, :K].transpose(0, 1), weight.transpose(1, 2))
+        into = y.view(R, heads, yh)[:, :, :N].transpose(0, 1)
+        if wide:
+            torch.bmm(*args, out_dtype=torch.float32, out=into)
+        else:
+            torch.bmm(*args, out=into)
         if scale is not None:
             st = native.lib().rfx_scale_heads(y.data_ptr(), dt_code(y.dtype), _chk(scale, "scale", torch.float32),
                                               y.numel(), N, _stream())
             native.check(st, "scale_heads")
         return y
-    st = native.lib().rfx_heads_linear(x.data_ptr(), heads * K, weight.data_ptr(), y.data_ptr(), heads * N,
+    st = native.lib().rfx_heads_linear(x.data_ptr(), heads * xh, xh, weight.data_ptr(), y.data_ptr(), heads * yh, yh,
                                        dt_code(x.dtype), _chk(scale, "scale", torch.float32), R, N, K, heads,
                                        _stream())
     native.check(st, f"heads_linear (heads={heads}, N={N}, K={K})")
@@ -1063,6 +1096,13 @@ def stream_concat(x: torch.Tensor, delta: Optional[torch.Tensor], x0: torch.Tens
 def keep_copy(x: torch.Tensor) -> torch.Tensor:
     """A copy of `x` that lives for the whole step."""
     out = _new(tuple(x.shape), x.dtype, x.device, keep=True)
+    out.copy_(x)
+    return out
+
+
+def cast_rows(x: torch.Tensor, out_dtype: torch.dtype) -> torch.Tensor:
+    """A copy of `x` in `out_dtype`."""
+    out = _new(tuple(x.shape), out_dtype, x.device)
     out.copy_(x)
     return out
 
@@ -1348,29 +1388,53 @@ def mamba_scan(x: torch.Tensor, dtpre: torch.Tensor, dt_bias: Optional[torch.Ten
 
 # ------------------------------------------- norms around a sublayer, small companions
 def sandwich_norm(y: torch.Tensor, x: torch.Tensor, post_weight: torch.Tensor, mult: float, eps: float,
-                  next_weight: Optional[torch.Tensor], next_eps: float, out_dtype: torch.dtype):
-    """x <- x + mult * rms_norm(y) * post_weight in place (`y`, `x` float32 [R, H]);
-    with `next_weight` also returns rms_norm(x) * next_weight in `out_dtype`: the
-    norm after one sublayer and the norm before the next in one pass over the row."""
+                  next_weight: Optional[torch.Tensor], next_eps: float, out_dtype: torch.dtype,
+                  post_offset: float = 0.0, next_offset: float = 0.0):
+    """x <- x + mult * rms_norm(y) * (post_offset + post_weight) in place (`y`, `x`
+    float32 [R, H]); with `next_weight` also returns rms_norm(x) * (next_offset +
+    next_weight) in `out_dtype`: the norm after one sublayer and the norm before the
+    next in one pass over the row."""
     R, H = x.shape
     if tuple(y.shape) != (R, H):
         raise InvalidInput("sandwich_norm: y and x must have the same shape")
     out = _new((R, H), out_dtype, x.device) if next_weight is not None else None
     st = native.lib().rfx_sandwich_norm(
         _chk(y, "y", torch.float32), _chk(x, "x", torch.float32), _chk(post_weight, "post_weight", torch.float32),
-        float(mult), float(eps), _chk(next_weight, "next_weight", torch.float32), float(next_eps),
-        out.data_ptr() if out is not None else 0, dt_code(out_dtype), R, H, _stream())
+        float(post_offset), float(mult), float(eps), _chk(next_weight, "next_weight", torch.float32),
+        float(next_offset), float(next_eps), out.data_ptr() if out is not None else 0, dt_code(out_dtype), 0, R, H,
+        _stream())
     native.check(st, f"sandwich_norm (H={H})")
     return out
 
 
+def post_norm(y: torch.Tensor, x: torch.Tensor, weight: torch.Tensor, weight_offset: float, eps: float,
+              out_dtype: Optional[torch.dtype], fresh: bool = False):
+    """x <- x + rms_norm(y) * (weight_offset + weight) in place, `y`, `x` float32
+    [R, H]; `fresh`: x <- the normed y alone (`y` may be `x`).  With `out_dtype`
+    also returns the new x in that type, the next product's input."""
+    R, H = x.shape
+    if tuple(y.shape) != (R, H):
+        raise InvalidInput("post_norm: y and x must have the same shape")
+    out = _new((R, H), out_dtype, x.device) if out_dtype is not None else None
+    st = native.lib().rfx_sandwich_norm(
+        _chk(y, "y", torch.float32), _chk(x, "x", torch.float32), _chk(weight, "weight", torch.float32),
+        float(weight_offset), 1.0, float(eps), 0, 0.0, 0.0, out.data_ptr() if out is not None else 0,
+        dt_code(out_dtype) if out_dtype is not None else F32, 1 if fresh else 0, R, H, _stream())
+    native.check(st, f"post_norm (H={H})")
+    return out
+
+
 def group_norm_gate(x: torch.Tensor, weight: torch.Tensor, eps: float, groups: int, out_dtype: torch.dtype,
-                    gate: Optional[torch.Tensor] = None, gate_col: int = 0) -> torch.Tensor:
+                    gate: Optional[torch.Tensor] = None, gate_col: int = 0,
+                    activation: str = "sigmoid") -> torch.Tensor:
     """`x` float32 [R, C] in `groups` equal parts, each divided by its own root mean
-    square, times weight[c]; with `gate` (float32 rows, the gate's pre-activations
-    from column `gate_col` on) also times their sigmoid."""
+    square, times weight[c] (a weight of one part's size is shared by the parts);
+    with `gate` (float32 rows, the gate's pre-activations from column `gate_col`
+    on) also times their sigmoid or (`activation`) silu."""
     R, C = x.shape
-    if C % groups or weight.numel() != C:
+    if activation not in ("sigmoid", "silu"):
+        raise InvalidInput(f"group_norm_gate: activation must be 'sigmoid' or 'silu', got {activation!r}")
+    if C % groups or weight.numel() not in (C, C // groups):
         raise InvalidInput("group_norm_gate: the groups must divide the row and the weight match it")
     if gate is not None and gate_col + C > gate.shape[1]:
         raise InvalidInput("group_norm_gate: the gate's columns do not fit into its rows")
@@ -1378,7 +1442,8 @@ def group_norm_gate(x: torch.Tensor, weight: torch.Tensor, eps: float, groups: i
     st = native.lib().rfx_group_norm_gate(
         _chk(x, "x", torch.float32), _chk(weight, "weight", torch.float32), float(eps),
         _chk(gate, "gate", torch.float32), gate.shape[1] if gate is not None else 0, int(gate_col),
-        out.data_ptr(), dt_code(out_dtype), R, C, int(groups), _stream())
+        1 if activation == "silu" else 0, 1 if weight.numel() != C else 0, out.data_ptr(), dt_code(out_dtype), R, C,
+        int(groups), _stream())
     native.check(st, f"group_norm_gate (C={C}, groups={groups})")
     return out
 
@@ -1562,6 +1627,116 @@ def delta_rule(proj: torch.Tensor, r_off: int, k_off: int, v_off: int, a_off: in
         batch.seq_slot.numel(), out.data_ptr(), dt_code(torch.float32), heads, dim, _stream())
     native.check(st, f"delta_rule (heads={heads}, dim={dim})")
     return out
+
+
+def gated_delta_prep(proj: torch.Tensor, b_off: int, a_off: int, filters_t: torch.Tensor, state: torch.Tensor, batch,
+                     dt_bias: torch.Tensor, A: torch.Tensor, unit_eps: float, q_scale: float, heads: int,
+                     kv_heads: int, dim: int, vdim: int, update_state: bool = False):
+    """The rows of a stacked product [q | k | v | ..] (float32) through their short
+    convolutions (`filters_t` float32 [taps, channels]) and silu, q and k made unit
+    vectors per head (q also times `q_scale`): float32 [R, channels]; and from the
+    columns at `b_off` and `a_off` the write rates sigmoid(b) and the decays exp(A
+    softplus(a + dt_bias)): float32 [R, 2 heads], decays first.  `state` holds each
+    slot's last inputs at its vector's start; `update_state`: one row a sequence,
+    and the launch moves them on."""
+    if update_state and proj.shape[0] != batch.seq_slot.numel():
+        raise InvalidInput("gated_delta_prep: update_state is for steps of one row a sequence")
+    R, ld = proj.shape
+    taps, C = filters_t.shape
+    if C != 2 * kv_heads * dim + heads * vdim or max(b_off, a_off) + heads > ld or C > ld:
+        raise InvalidInput("gated_delta_prep: the columns do not fit into the rows")
+    out = _new((R, C), torch.float32, proj.device)
+    gates = _new((R, 2 * heads), torch.float32, proj.device)
+    st = native.lib().rfx_gated_delta_prep(
+        _chk(proj, "proj", torch.float32), ld, int(b_off), int(a_off), _chk(filters_t, "filters_t", torch.float32),
+        int(taps), _chk(state, "state", torch.float32), state.stride(0), _chk(batch.row_slot, "row_slot", torch.int32),
+        _chk(dt_bias, "dt_bias", torch.float32), _chk(A, "A", torch.float32), float(unit_eps), float(q_scale),
+        out.data_ptr(), gates.data_ptr(), R, heads, kv_heads, dim, vdim, 1 if update_state else 0, _stream())
+    native.check(st, f"gated_delta_prep (heads={heads}, dim={dim}, vdim={vdim}, taps={taps})")
+    return out, gates
+
+
+def gated_delta_scan(qkv: torch.Tensor, gates: torch.Tensor, state: torch.Tensor, state_off: int, batch, heads: int,
+                     kv_heads: int, dim: int, vdim: int) -> torch.Tensor:
+    """The gated delta rule over the step's rows (csrc/gated_delta.cu): `qkv` and
+    `gates` as `gated_delta_prep` makes them; the running state is `state[slot,
+    state_off : state_off + heads * vdim * (dim rounded up to 4)]`.  Returns S^T q,
+    float32 [R, heads * vdim]."""
+    R = qkv.shape[0]
+    if qkv.shape[1] != 2 * kv_heads * dim + heads * vdim or tuple(gates.shape) != (R, 2 * heads):
+        raise InvalidInput("gated_delta_scan: the rows do not match the sizes")
+    out = _new((R, heads * vdim), torch.float32, qkv.device)
+    st = native.lib().rfx_gated_delta_scan(
+        _chk(qkv, "qkv", torch.float32), _chk(gates, "gates", torch.float32), _chk(state, "state", torch.float32),
+        state.stride(0), int(state_off), _chk(batch.seq_slot, "seq_slot", torch.int32),
+        _chk(batch.seq_row0, "seq_row0", torch.int32), batch.seq_slot.numel(), out.data_ptr(), heads, kv_heads, dim,
+        vdim, int(batch.max_new), _stream())
+    native.check(st, f"gated_delta_scan (heads={heads}, dim={dim}, vdim={vdim})")
+    return out
+
+
+# --------------------------------- rotation, then the norm; latents with a rotated part
+def _plain_rotation(rotation, what: str):
+    if rotation is None:
+        return None, 0
+    if rotation.pairing != "half" or rotation.magnitude != 1.0:
+        raise InvalidInput(f"{what}: takes a plain half-split rotation")
+    return rotation.denominators, int(rotation.rotary_dim)
+
+
+def rot_qkv_post(proj: torch.Tensor, bias: Optional[torch.Tensor], rotation, unit_eps: Optional[float],
+                 mix: Optional[torch.Tensor], v_first: Optional[torch.Tensor], keep_values: bool, row_pos, row_slot,
+                 k_pages, v_pages, page_table, page_size: int, nq: int, nkv: int, dim: int, vdim: int, pad: int,
+                 writes_cache: bool, out_dtype: torch.dtype):
+    """Rows [q | k | v] plus `bias` (float32): q and k rotated (a half-split
+    `parts.Rotation` or None), then, with `unit_eps`, divided by their root mean
+    square per head; q out as [R, nq * pad], k and v into the cache, heads `pad`
+    wide (zeros beyond `dim` and `vdim`).  `v_first` (float32 [R, nkv * vdim]) and
+    `mix` (one float32 number): the values become (1 - mix) v + mix v_first first.
+    Returns (q, values): `keep_values` asks for the step's unmixed values as
+    float32 rows that live for the whole step (else None)."""
+    R = proj.shape[0]
+    if proj.shape[1] < nq * dim + (nkv * (dim + vdim) if writes_cache else 0):
+        raise InvalidInput("rot_qkv_post: the q | k | v columns do not fit into the rows")
+    if v_first is not None and (tuple(v_first.shape) != (R, nkv * vdim) or mix is None):
+        raise InvalidInput("rot_qkv_post: the first values' rows must match the values and come with a mix")
+    denom, rot = _plain_rotation(rotation, "rot_qkv_post")
+    q = _new((R, nq * pad), out_dtype, proj.device)
+    kept = _new((R, nkv * vdim), torch.float32, proj.device, keep=True) if keep_values else None
+    st = native.lib().rfx_rot_qkv_post(
+        _chk(proj, "proj"), dt_code(proj.dtype), proj.shape[1], _chk(bias, "bias", torch.float32),
+        _chk(denom, "denominators", torch.float32), rot, 0 if unit_eps is None else 1, float(unit_eps or 0.0),
+        _chk(mix, "mix", torch.float32) if v_first is not None else 0, _chk(v_first, "v_first", torch.float32),
+        kept.data_ptr() if kept is not None else 0, _chk(row_pos, "row_pos", torch.int32),
+        _chk(row_slot, "row_slot", torch.int32), q.data_ptr(), _chk(k_pages, "k_pages", out_dtype),
+        _chk(v_pages, "v_pages", out_dtype), dt_code(out_dtype), _chk(page_table, "page_table", torch.int32),
+        page_table.shape[1], page_size, R, nq, nkv, dim, vdim, pad, 1 if writes_cache else 0, _stream())
+    native.check(st, f"rot_qkv_post (dim={dim}, vdim={vdim})")
+    return q, kept
+
+
+def latent_rot_post(proj: torch.Tensor, kv_weight: torch.Tensor, eps: float, rotation, row_pos, row_slot, pages,
+                    page_table, page_size: int, heads: int, dim: int, rot_dim: int, rank: int, width: int,
+                    writes_cache: bool, out_dtype: torch.dtype):
+    """Rows [q | latent | shared key part]: returns (q_flat [R, heads * dim], the
+    unrotated parts of q; q_abs [R, heads * width], whose columns from `rank` on of
+    every head hold the rotated part and zeros, the rest still to be filled), and
+    writes [latent / rms(latent) * kv_weight | rotated key part | zeros], `width`
+    elements, into the cache at the rows' positions."""
+    R = proj.shape[0]
+    denom, rot = _plain_rotation(rotation, "latent_rot_post")
+    if rot not in (0, rot_dim):
+        raise InvalidInput("latent_rot_post: the rotation covers the whole rotated part")
+    flat = _new((R, heads * dim), out_dtype, proj.device)
+    qa = _new((R, heads * width), out_dtype, proj.device)
+    st = native.lib().rfx_latent_rot_post(
+        _chk(proj, "proj"), dt_code(proj.dtype), proj.shape[1], _chk(kv_weight, "kv_weight", torch.float32),
+        float(eps), _chk(denom, "denominators", torch.float32), _chk(row_pos, "row_pos", torch.int32),
+        _chk(row_slot, "row_slot", torch.int32), flat.data_ptr(), qa.data_ptr(), _chk(pages, "pages", out_dtype),
+        dt_code(out_dtype), _chk(page_table, "page_table", torch.int32), page_table.shape[1], page_size, R, heads,
+        dim, rot_dim, rank, width, 1 if writes_cache else 0, _stream())
+    native.check(st, f"latent_rot_post (rank={rank}, rot={rot_dim})")
+    return flat, qa
 
 
 # ------------------------------------------------------------------ sampling

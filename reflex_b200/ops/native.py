@@ -46,16 +46,17 @@ _SIGNATURES = {
                      c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_void_p],
     "rfx_attention_plain": [c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_int, c_int, c_void_p,
                             c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_void_p, c_void_p,
-                            c_void_p],
+                            c_float, c_void_p],
     "rfx_attention_decode_kf": [c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_void_p, c_void_p,
                                 c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_float,
-                                c_void_p, c_void_p, c_longlong, c_int, c_void_p, c_void_p],
+                                c_void_p, c_void_p, c_float, c_longlong, c_int, c_void_p, c_void_p],
     "rfx_attention_prefill_kf": [c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_void_p, c_void_p,
                                  c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int,
-                                 c_float, c_void_p, c_void_p, c_void_p],
+                                 c_float, c_void_p, c_void_p, c_float, c_void_p],
     "rfx_attention_prefill_tc_kf": [c_void_p, c_void_p, c_void_p, c_longlong, c_void_p, c_int, c_int, c_void_p,
                                     c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int,
-                                    c_int, c_int, c_int, c_float, c_void_p, c_void_p, c_void_p, c_void_p],
+                                    c_int, c_int, c_int, c_float, c_void_p, c_void_p, c_float, c_float, c_void_p,
+                                    c_void_p],
     "rfx_qkv_post_kv": [c_void_p, c_int, c_int, c_void_p, c_void_p, c_float, c_float, c_void_p, c_int,
                         c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_int, c_int,
                         c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_int, c_void_p],
@@ -90,8 +91,8 @@ _SIGNATURES = {
     "rfx_latent_post": [c_void_p, c_int, c_int, c_void_p, c_void_p, c_float, c_void_p, c_void_p, c_void_p,
                         c_void_p, c_int, c_void_p, c_int, c_int, c_void_p, c_int, c_int, c_int, c_int, c_int,
                         c_void_p],
-    "rfx_heads_linear": [c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_void_p, c_int, c_int, c_int,
-                         c_int, c_void_p],
+    "rfx_heads_linear": [c_void_p, c_int, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_void_p, c_int, c_int,
+                         c_int, c_int, c_void_p],
     "rfx_scale_heads": [c_void_p, c_int, c_void_p, c_longlong, c_int, c_void_p],
     "rfx_mlstm_scan": [c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_float,
                        c_float, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int,
@@ -112,10 +113,23 @@ _SIGNATURES = {
     "rfx_moe_combine": [c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_void_p],
     "rfx_moe_route_scaled": [c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_float,
                              c_void_p],
-    "rfx_sandwich_norm": [c_void_p, c_void_p, c_void_p, c_float, c_float, c_void_p, c_float, c_void_p, c_int, c_int,
-                          c_int, c_void_p],
-    "rfx_group_norm_gate": [c_void_p, c_void_p, c_float, c_void_p, c_int, c_int, c_void_p, c_int, c_int, c_int, c_int,
-                            c_void_p],
+    "rfx_sandwich_norm": [c_void_p, c_void_p, c_void_p, c_float, c_float, c_float, c_void_p, c_float, c_float,
+                          c_void_p, c_int, c_int, c_int, c_int, c_void_p],
+    "rfx_group_norm_gate": [c_void_p, c_void_p, c_float, c_void_p, c_int, c_int, c_int, c_int, c_void_p, c_int, c_int,
+                            c_int, c_int, c_void_p],
+    "rfx_gated_act": [c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_void_p],
+    "rfx_gemm_bf16_tc_geglu": [c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p],
+    "rfx_gated_delta_prep": [c_void_p, c_int, c_int, c_int, c_void_p, c_int, c_void_p, c_longlong, c_void_p, c_void_p,
+                             c_void_p, c_float, c_float, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int,
+                             c_void_p],
+    "rfx_gated_delta_scan": [c_void_p, c_void_p, c_void_p, c_longlong, c_longlong, c_void_p, c_void_p, c_int, c_void_p,
+                             c_int, c_int, c_int, c_int, c_int, c_void_p],
+    "rfx_rot_qkv_post": [c_void_p, c_int, c_int, c_void_p, c_void_p, c_int, c_int, c_float, c_void_p, c_void_p,
+                         c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_int, c_int,
+                         c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p],
+    "rfx_latent_rot_post": [c_void_p, c_int, c_int, c_void_p, c_float, c_void_p, c_void_p, c_void_p, c_void_p,
+                            c_void_p, c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int,
+                            c_int, c_int, c_void_p],
     "rfx_xielu": [c_void_p, c_int, c_longlong, c_float, c_float, c_void_p],
     "rfx_loop_input": [c_void_p, c_void_p, c_void_p, c_int, c_int, c_void_p],
     "rfx_tanh_cols": [c_void_p, c_int, c_int, c_void_p, c_int, c_int, c_int, c_void_p],

@@ -18,3 +18,4 @@ from . import norm, rope, mlp, attention, block, embedding, latent_attention, ml
 from . import conv_attention, rglru, pair  # noqa: F401,E402  (registers the parts)
 from . import hyper, selective_scan  # noqa: F401,E402
 from . import sigmoid_attention, ssd, delta_rule  # noqa: F401,E402
+from . import capped_attention, gated_delta  # noqa: F401,E402

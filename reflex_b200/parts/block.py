@@ -4,7 +4,8 @@
 (src/model/dense.rs:1441-1484).  "parallel": n = norm1(h); h += mixer(n) + ffn(n),
 one norm that both sublayers read.  "sandwich": a norm on both sides of every
 sublayer, h += m * post1(mixer(norm1(h))); h += m * post2(ffn(norm2(h))), m one
-number of the layer.  The residual stream is 32-bit; each add is
+number of the layer.  "postnorm": a norm only on what a sublayer gives,
+h += norm1(mixer(h)); h += norm2(ffn(h)).  The residual stream is 32-bit; each add is
 fused into the norm that follows it, so a block hands its last delta on as
 `pending` and the next block's (or the model's final) norm adds it
 (src/model/decode_step.rs:199-210, 293-300).
@@ -200,6 +201,14 @@ class ParallelBlock(PreNormBlock):
         return hidden, delta
 
 
+class ReadyRows:
+    """Rows the next block starts from, already made in the compute type: its first
+    norm's, or the stream's own where a block reads it unnormed."""
+
+    def __init__(self, rows):
+        self.rows = rows
+
+
 @register_block("sandwich")
 class SandwichBlock(PreNormBlock):
     """h += m * post1(mixer(norm1(h))); h += m * post2(ffn(norm2(h))): every
@@ -209,12 +218,6 @@ class SandwichBlock(PreNormBlock):
     the next one are one pass over the row (`ops.sandwich_norm`): the block hands
     the next block its first norm's rows ready (`ReadyRows`) when it is told that
     norm, and adds into the residual itself, so it never leaves a delta pending."""
-
-    class ReadyRows:
-        """Rows the next block's first norm has already produced."""
-
-        def __init__(self, rows):
-            self.rows = rows
 
     skips_final_norm_fusion = True  # the model's last norm meets the wanted rows only
 
@@ -258,7 +261,7 @@ class SandwichBlock(PreNormBlock):
     def forward(self, hidden: torch.Tensor, pending, ctx, next_norm=None):
         from .. import ops
 
-        if isinstance(pending, SandwichBlock.ReadyRows):
+        if isinstance(pending, ReadyRows):
             x = pending.rows
         else:
             if isinstance(pending, ops.NormedInput):
@@ -274,10 +277,60 @@ class SandwichBlock(PreNormBlock):
                               after.spec.eps if after is not None else 0.0, self.dtype)
         ops.prof_mark("norm")
         if not self.has_feed_forward:
-            return hidden, (SandwichBlock.ReadyRows(x) if x is not None else None)
+            return hidden, (ReadyRows(x) if x is not None else None)
         y = self.feed_forward.forward(x)
         x = ops.sandwich_norm(y, hidden, self.post_feed_forward.weight, self.mult, self.post_feed_forward.spec.eps,
                               nxt.weight if nxt is not None else None, nxt.spec.eps if nxt is not None else 0.0,
                               self.dtype)
         ops.prof_mark("norm")
-        return hidden, (SandwichBlock.ReadyRows(x) if x is not None else None)
+        return hidden, (ReadyRows(x) if x is not None else None)
+
+
+@register_block("postnorm")
+class PostNormBlock(PreNormBlock):
+    """h += norm1(mixer(h)); h += norm2(ffn(h)): the sublayers read the stream itself,
+    rounded to the compute type, and only their results are normed (`mixer_norm`,
+    `feed_forward_norm`, RMS norms with any weight offset).  Norm, add and the
+    rounded rows of the next sublayer are one pass (`ops.post_norm`); a block hands
+    the next one its input rows ready (`ReadyRows`) and never leaves a delta pending."""
+
+    skips_final_norm_fusion = True  # the model's last norm meets the wanted rows only
+    READS_STREAM = object()         # what a block of this kind wants of the one before it: the stream's rows
+
+    def __init__(self, spec: LayerSpec, dtype: torch.dtype, device):
+        super().__init__(spec, dtype, device)
+        self.dtype = dtype
+        for n in (self.mixer_norm, self.feed_forward_norm):
+            if n is not None and n.spec.kind != "rmsnorm":
+                raise ValueError("postnorm block: takes RMS norms")
+
+    @property
+    def fusable_first_norm(self):
+        return PostNormBlock.READS_STREAM
+
+    @property
+    def capturable(self) -> bool:
+        return PreNormBlock.capturable.fget(self)
+
+    def forward(self, hidden: torch.Tensor, pending, ctx, next_norm=None):
+        from .. import ops
+
+        if isinstance(pending, ReadyRows):
+            x = pending.rows
+        else:
+            if pending is not None and not isinstance(pending, ops.NormedInput):
+                ops.add_(hidden, pending)
+            x = ops.cast_rows(hidden, self.dtype)
+            ops.prof_mark("norm")
+        after = self.dtype if next_norm is PostNormBlock.READS_STREAM else None
+        y = self.mixer.forward(x, ctx)
+        n = self.mixer_norm
+        x = ops.post_norm(y, hidden, n.weight, n.spec.weight_offset, n.spec.eps,
+                          self.dtype if self.has_feed_forward else after)
+        ops.prof_mark("norm")
+        if self.has_feed_forward:
+            y = self.feed_forward.forward(x)
+            n = self.feed_forward_norm
+            x = ops.post_norm(y, hidden, n.weight, n.spec.weight_offset, n.spec.eps, after)
+            ops.prof_mark("norm")
+        return hidden, (ReadyRows(x) if x is not None else None)

@@ -8,7 +8,16 @@ With h the mixer's input [rows, hidden]:
   s_ij = (q_i . k_j) * scale  for 0 <= i - j < window
   p = exp(s) / (sum_j exp(s_ij) + exp(sink_h))     the sink has no key and no value
   out = W_o concat_h( sigmoid(W_g h)_h * sum_j p_ij v_j )
-There is no position encoding.  Since k_j = W_uk c_j, the score is
+There is no position encoding.
+
+Without `q_rank` (the other form) q = W_q h, per head `head_dim` unrotated and
+`rot_dim` rotated elements, [unrotated | rotated], and W_dkv h has `rot_dim` more
+rows: one rotated key part r_j all heads share, not normed:
+  s_ij = (q_i . k_j + rot(q_i') . rot(r_j)) * scale
+The cached row is then [c | rot(r) | zeros], and the folded query is followed by
+its rotated part.
+
+Since k_j = W_uk c_j, the score is
 (W_uk,h^T q_i) . c_j and the weighted values are W_uv,h (sum_j p_ij c_j): the
 attention runs over the cached latents themselves as one shared key/value head
 of `kv_rank` elements (keys and values are the same rows of the cache), with
@@ -25,37 +34,54 @@ import torch
 from .. import ops
 from ..cache.specs import KVSpec
 from ..config.spec import MixerSpec
-from .registry import TensorInfo, register_mixer
+from ..errors import InvalidInput
+from .registry import POSITIONS, TensorInfo, register_mixer
 
 
 @register_mixer("latent_attention")
 class LatentAttention:
     capturable = True  # positions, slots and the page table are read from device memory
-    supports_fused_residual = True
+
+    @property
+    def supports_fused_residual(self) -> bool:
+        return self.q_rank > 0
 
     def __init__(self, spec: MixerSpec, dtype: torch.dtype, device):
         self.spec = spec
         self.dtype = dtype
         self.device = device
-        self.q_rank = int(spec.param("q_rank"))
+        self.q_rank = int(spec.param("q_rank", 0) or 0)  # 0: queries straight from the input
+        self.rot_dim = int(spec.param("rot_dim", 0) or 0)
+        self.position = (POSITIONS.get(spec.position.kind)(spec.position, dtype, device)
+                         if spec.position is not None else None)
         self.kv_rank = int(spec.param("kv_rank"))
         self.eps = float(spec.param("eps"))
         self.has_sink = bool(spec.param("sink", False))
         self.has_gate = spec.param("gate") == "head"
+        if self.q_rank and (self.rot_dim or self.position is not None):
+            raise InvalidInput("latent_attention: a rotated part goes with queries straight from the input")
+        if not self.q_rank and self.has_gate:
+            raise InvalidInput("latent_attention: a gate goes with queries through a latent")
+        # elements of a cached row: the latent and the rotated part, in steps of 16 for the tensor cores
+        self.width = self.kv_rank if self.q_rank else (self.kv_rank + self.rot_dim + 15) // 16 * 16
         self.down = self.q_up = self.k_absorb = self.v_up = self.o = None
         self.q_norm = self.kv_norm = self.sink = None
 
     @classmethod
     def tensor_specs(cls, spec: MixerSpec) -> Dict[str, TensorInfo]:
         W, H, d, dv = spec.hidden_size, spec.num_heads, spec.head_dim, spec.value_dim
-        qr, kr = int(spec.param("q_rank")), int(spec.param("kv_rank"))
-        out = {
-            "q_down": TensorInfo((qr, W), "matrix"), "q_norm": TensorInfo((qr,), "norm"),
-            "q_up": TensorInfo((H * d, qr), "matrix"),
-            "kv_down": TensorInfo((kr, W), "matrix"), "kv_norm": TensorInfo((kr,), "norm"),
+        qr, kr = int(spec.param("q_rank", 0) or 0), int(spec.param("kv_rank"))
+        rot = int(spec.param("rot_dim", 0) or 0)
+        if qr:
+            out = {"q_down": TensorInfo((qr, W), "matrix"), "q_norm": TensorInfo((qr,), "norm"),
+                   "q_up": TensorInfo((H * d, qr), "matrix")}
+        else:
+            out = {"q_proj": TensorInfo((H * (d + rot), W), "matrix")}
+        out.update({
+            "kv_down": TensorInfo((kr + rot, W), "matrix"), "kv_norm": TensorInfo((kr,), "norm"),
             "k_up": TensorInfo((H * d, kr), "matrix"), "v_up": TensorInfo((H * dv, kr), "matrix"),
             "o_proj": TensorInfo((W, H * dv), "matrix"),
-        }
+        })
         if spec.param("sink", False):
             out["sink"] = TensorInfo((H,), "bias")
         if spec.param("gate") == "head":
@@ -64,7 +90,7 @@ class LatentAttention:
 
     def cache_spec(self) -> KVSpec:
         # one latent a position serves as key and as value
-        return KVSpec(1, self.kv_rank, self.spec.window, shared_kv=True)
+        return KVSpec(1, self.width, self.spec.window, shared_kv=True)
 
     def bind(self, tensors: Dict[str, torch.Tensor]) -> None:
         s = self.spec
@@ -76,22 +102,30 @@ class LatentAttention:
         def f32(t):
             return t.to(device=self.device, dtype=torch.float32).contiguous()
 
-        parts = [dev(tensors["q_down"]), dev(tensors["kv_down"])]
+        parts = [dev(tensors["q_down" if self.q_rank else "q_proj"]), dev(tensors["kv_down"])]
         if self.has_gate:
             parts.append(dev(tensors["gate"]))
+        if not self.q_rank:
+            # zero rows up to a multiple of 8: the product's rows stay 16-byte aligned
+            rows = sum(p.shape[0] for p in parts)
+            parts.append(torch.zeros((-rows % 8, s.hidden_size), dtype=self.dtype, device=self.device))
         self.down = torch.cat(parts, dim=0).contiguous()  # one product for both latents and the gates
-        self.q_up = dev(tensors["q_up"]).contiguous()
+        if self.q_rank:
+            self.q_up = dev(tensors["q_up"]).contiguous()
+            self.q_norm = f32(tensors["q_norm"])
         # W_uk per head, transposed: [H, kv_rank, dim], so that q_h -> W_uk,h^T q_h is a per-head product
         self.k_absorb = dev(tensors["k_up"]).view(H, d, self.kv_rank).transpose(1, 2).contiguous()
         self.v_up = dev(tensors["v_up"]).view(H, dv, self.kv_rank).contiguous()
         self.o = dev(tensors["o_proj"]).contiguous()
-        self.q_norm, self.kv_norm = f32(tensors["q_norm"]), f32(tensors["kv_norm"])
+        self.kv_norm = f32(tensors["kv_norm"])
         self.sink = f32(tensors["sink"]) if self.has_sink else None
 
     def forward(self, x, ctx, residual=None):
         s = self.spec
         kv, batch = ctx.kv, ctx.batch
         H = s.num_heads
+        if not self.q_rank:
+            return self._forward_direct(x, ctx)
         proj = ops.linear(x, self.down, out_dtype=torch.float32)
         ops.prof_mark("qkv_gemm")
         cq, gate = ops.latent_post(proj, self.q_norm, self.kv_norm, self.eps, batch.row_pos, batch.row_slot,
@@ -112,6 +146,28 @@ class LatentAttention:
             if fused is not None:
                 ops.prof_mark("o_proj")
                 return None if fused is ops.ADDED else fused
+        out = ops.linear(vals, self.o, out_dtype=torch.float32)
+        ops.prof_mark("o_proj")
+        return out
+
+    def _forward_direct(self, x, ctx):
+        """The form without a query latent; the delta [rows, hidden] comes back 32-bit."""
+        s, kv, batch = self.spec, ctx.kv, ctx.batch
+        H = s.num_heads
+        proj = ops.linear(x, self.down, out_dtype=torch.float32)
+        ops.prof_mark("qkv_gemm")
+        flat, qa = ops.latent_rot_post(
+            proj, self.kv_norm, self.eps, None if self.position is None else self.position.rotation(), batch.row_pos,
+            batch.row_slot, kv.k_pages, kv.page_table, kv.page_size, H, s.head_dim, self.rot_dim, self.kv_rank,
+            self.width, ctx.writes_cache, self.dtype)
+        ops.prof_mark("latent_post")
+        ops.heads_linear(flat, self.k_absorb, out=qa)
+        ops.prof_mark("q_absorb")
+        attn = ops.attention(qa, kv.k_pages, kv.k_pages, kv.page_table, kv.page_size, batch, H, 1, self.width,
+                             s.window, s.scale, sink=self.sink)
+        ops.prof_mark("attn")
+        vals = ops.heads_linear(attn, self.v_up)  # of each head the latent's elements; the rest is dropped
+        ops.prof_mark("v_up")
         out = ops.linear(vals, self.o, out_dtype=torch.float32)
         ops.prof_mark("o_proj")
         return out

@@ -67,6 +67,24 @@ class SwiGLU:
         return out
 
 
+@register_feed_forward("geglu")
+class GeGLU(SwiGLU):
+    """The gated feed-forward with the tanh form of gelu: out = W_d (gelu(W_g x) *
+    (W_u x)), gelu(z) = z / 2 (1 + tanh(sqrt(2 / pi) (z + 0.044715 z^3))).  Gate and up
+    are one woven matrix, as in `SwiGLU`, and for a few rows the activation is the
+    product's epilogue."""
+
+    accepts_normed_input = False
+    supports_fused_residual = False
+
+    def forward(self, x, residual=None):
+        act = ops.linear_geglu(x, self.gate_up)
+        ops.prof_mark("ffn_gate_up")
+        out = ops.linear(act, self.down, out_dtype=torch.float32)
+        ops.prof_mark("ffn_down")
+        return out
+
+
 @register_feed_forward("glu_clamped")
 class ClampedGLU:
     """The clamped gated feed-forward: g = min(W_g x, limit), u = clamp(W_u x,

@@ -48,6 +48,22 @@ class RotaryNeox:
         return Rotation(self.denominators, self.spec.rotary_dim, "half", 1.0)
 
 
+@register_position("rope_linear")
+class RotaryLinear(RotaryNeox):
+    """The half-split rotation with every frequency divided by the parameter `factor`:
+    the pair turns by position / (factor * theta^(2i/rd)).  Only the table of
+    denominators differs from the plain encoding."""
+
+    def __init__(self, spec: PositionSpec, dtype: torch.dtype, device):
+        super().__init__(spec, dtype, device)
+        factor = float(dict(spec.params).get("factor", 1.0))
+        if not factor > 0:
+            raise InvalidInput("rope_linear: factor must be positive")
+        denom = [factor * math.pow(float(spec.theta), 2.0 * i / float(spec.rotary_dim))
+                 for i in range(spec.rotary_dim // 2)]
+        self.denominators = torch.tensor(denom, dtype=torch.float64).to(torch.float32).to(device)
+
+
 @register_position("rope_scaled")
 class RotaryScaled(RotaryNeox):
     """The half-split rotation with wavelength-dependent frequency scaling.
