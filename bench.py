@@ -342,6 +342,29 @@ def zelinex_config(z):
             "residual_mult": 0.8, "loop": {"start": 0, "stop": z["layers"], "times": 1}, "layers": layers}
 
 
+def zivulix_config(z):
+    """Zivulix at the sizes of `z`: of four layers two are a gated delta rule (heads of
+    128 keys and values, twice the width of values, half as many query/key heads, four
+    taps), one is a capped attention (a quarter as many key/value heads, half of each head
+    rotated, the window of the models beside it, mixed values) and one a latent attention
+    (a rotated part of 64 beside the models' head size, every earlier key), every layer
+    with a feed-forward."""
+    delta = {"type": "delta", "mixer": {"heads": z["width"] // 64, "kv_heads": z["width"] // 128, "dim": 128,
+                                        "vdim": 128, "conv": 4}}
+    att = {"type": "attention",
+           "mixer": {"heads": z["heads"], "kv_heads": max(1, z["heads"] // 4), "dim": z["dim"], "vdim": z["dim"],
+                     "scale": z["dim"] ** -0.5, "softcap": 50.0, "v_mix": True,
+                     "rot": {"base": 500000.0, "dims": z["dim"] // 2, "scaling": {"factor": 4.0}},
+                     "mask": {"size": z["window"]}}}
+    lat = {"type": "latent_attention",
+           "mixer": {"heads": z["heads"], "dim": z["dim"], "rot_dim": 64, "vdim": z["dim"], "kv_rank": z["kv_rank"],
+                     "scale": (z["dim"] + 64) ** -0.5, "rot": {"base": 500000.0, "dims": 64}}}
+    pattern = [delta, att, delta, lat]
+    layers = [dict(pattern[i % 4], mlp={"kind": "dense", "ff": z["ff"]}) for i in range(z["layers"])]
+    return {"architecture": "Zivulix", "vocab": z["vocab"], "width": z["width"], "norm": {"eps": 1e-5},
+            "layers": layers}
+
+
 def qwen3_config_like(z):
     cfg = dict(QWEN3_8B)
     cfg.update({"num_hidden_layers": z["layers"], "hidden_size": z["width"], "num_attention_heads": z["heads"],
@@ -355,8 +378,9 @@ def design_comparison(args) -> int:
     """Prefill and decode throughput of a design (`--design`) beside Qwen3 at
     equal sizes (and, for Pakarax, beside Kegasun too: the model with a
     recurrence and experts; for Zelinex beside Pakarax: the model with two mixers
-    side by side, experts and a loop), with every phase's time in a prefill and in a
-    decode step."""
+    side by side, experts and a loop; for Zivulix beside Kegasun, the model with a latent
+    attention, and Zelinex, the model with a delta rule), with every phase's time in a
+    prefill and in a decode step."""
     import torch
 
     from reflex_b200 import ops
@@ -367,10 +391,11 @@ def design_comparison(args) -> int:
     torch.cuda.set_device(0)
     T, B, P, steps = PREFILL_TOKENS, args.batch, PROMPT, max(16, min(args.steps, 64))
     mine = args.design
-    beside = [("qwen3", qwen3_config_like)] + ([("kegasun", kegasun_config)] if mine == "pakarax" else []) \
-        + ([("pakarax", pakarax_config)] if mine == "zelinex" else [])
+    beside = [("qwen3", qwen3_config_like)] + {
+        "pakarax": [("kegasun", kegasun_config)], "zelinex": [("pakarax", pakarax_config)],
+        "zivulix": [("kegasun", kegasun_config), ("zelinex", zelinex_config)]}.get(mine, [])
     mine_config = {"kegasun": kegasun_config, "pakarax": pakarax_config, "purusun": purusun_config,
-                   "zelinex": zelinex_config}[mine]
+                   "zelinex": zelinex_config, "zivulix": zivulix_config}[mine]
     out = {"metric": f"prefill and decode tokens/s, {mine} beside " + " and ".join(n for n, _ in beside)
                      + " at equal sizes", "unit": "tokens/s",
            "dtype": "bf16", "data": "synthetic: seeded uniform token ids, random-init weights",
@@ -495,7 +520,7 @@ def main() -> int:
                     help="workloads beside the headline: 14b and 32b add their points (default: all)")
     ap.add_argument("--prompt", type=int, default=PROMPT, help="prompt tokens before the decode steps")
     ap.add_argument("--context", type=int, default=CONTEXT, help="cache positions per sequence")
-    ap.add_argument("--design", default="", choices=["", "kegasun", "pakarax", "purusun", "zelinex"],
+    ap.add_argument("--design", default="", choices=["", "kegasun", "pakarax", "purusun", "zelinex", "zivulix"],
                     help="instead of the headline: this design beside Qwen3 at equal sizes (prefill, decode, phases)")
     ap.add_argument("--sizes", default="w1024,w2048,w4096", help="with --design: which of the sizes " +
                     ", ".join(sorted(DESIGN_SIZES)))
