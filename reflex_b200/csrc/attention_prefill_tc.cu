@@ -99,11 +99,27 @@ __host__ __device__ constexpr uint32_t idesc_b_mn(int M, int N) {
     return umma_idesc_bf16(M, N) | (1u << 16);
 }
 
+struct Bars {
+    uint64_t q_full, k_full[KV_STAGES], k_empty[KV_STAGES], v_full[KV_STAGES], v_empty[KV_STAGES], s_full[2], p_full[2],
+        o_full;
+    uint32_t tmem_base;
+    int abort_flag;
+};
+
+// Value tiles in flight: two, or one where keys wider than values would otherwise keep a second
+// CTA off the SM.
+constexpr int v_stages(int DK, int DV) { return DK > DV ? 1 : KV_STAGES; }
+
 struct Smem {
     // all tiles 1024-byte aligned
-    static constexpr int q_bytes(int D) { return ROWS * D * 2; }
-    static constexpr int kv_bytes(int D) { return PAGE * D * 2; }
-    static constexpr int total(int D) { return q_bytes(D) + 2 * KV_STAGES * kv_bytes(D) + 1024; }
+    static constexpr int tiles(int DK, int DV) {
+        return ROWS * DK * 2 + KV_STAGES * PAGE * DK * 2 + v_stages(DK, DV) * PAGE * DV * 2;
+    }
+    // paged: slack to align the tiles (the barriers are static); contiguous: the barriers lie
+    // behind the tiles and the block's shared memory is all dynamic, so it starts aligned
+    static constexpr int total(int DK, int DV, bool contig) {
+        return tiles(DK, DV) + (contig ? (int)sizeof(Bars) : 1024);
+    }
 };
 
 // SLOPES: a linear distance bias, slope_h * (query position - key position) off
@@ -114,7 +130,11 @@ struct Smem {
 // takes the raw score's place and `scale_log2` is cap * log2(e), so the rest of the page's code
 // is the same.  MODE 2 takes any argument; MODE 3 the polynomial for |s in_scale| <= 1/2, which
 // leaves the special-function unit to the softmax's exponentials.
-template <int D, int MODE>
+// CONTIG: keys and values are not pages but the rows of one matrix (a latent's keys and
+// values made for this step): position p of sequence i is row seq_base[i] + p, head h's key its
+// columns h DK .., its value its columns v_col + h DV .. (map_k and map_v then are the same
+// matrix).  `dv` columns of a value are written out (DV without CONTIG).
+template <int DK, int DV, int MODE, bool CONTIG>
 __global__ void __launch_bounds__(THREADS)
 attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q,
                             const __grid_constant__ CUtensorMap map_k,
@@ -123,26 +143,40 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q,
                             const int* __restrict__ seq_new, const int* __restrict__ seq_row0,
                             __nv_bfloat16* __restrict__ out, int nq, int bq, int window, int keep_first,
                             float scale_log2, float in_scale, const float* __restrict__ sink,
-                            const float* __restrict__ slopes, int* __restrict__ err) {
+                            const float* __restrict__ slopes, const int* __restrict__ seq_base, int v_col, int dv,
+                            int* __restrict__ err) {
     constexpr bool SLOPES = MODE == 1;
-    static_assert(D == 64 || D == 128, "head sizes 64 and 128");
-    constexpr int KB = D / 64;                 // 64-column blocks of a row
-    constexpr int KV_BYTES = PAGE * D * 2;
+    static_assert(DK % 64 == 0 && DK <= 192 && (DV == 64 || DV == 128), "keys up to 192, values 64 or 128");
+    constexpr int KB = DK / 64, VB = DV / 64;  // 64-column blocks of a row
+    constexpr int K_BYTES = PAGE * DK * 2, V_BYTES = PAGE * DV * 2;
+    constexpr int VS = v_stages(DK, DV);
     constexpr uint32_t TMEM_COLS = 256;
     // S: 2 x 64 columns (P_b, 32 columns of packed bfloat16, overwrites the start
-    // of S_b once the row has read it), then O: D columns
+    // of S_b once the row has read it), then O: DV columns
     constexpr uint32_t S_COL = 0, O_COL = 128;
 
-    extern __shared__ uint8_t smem_raw[];
-    __shared__ __align__(8) uint64_t q_full, k_full[KV_STAGES], k_empty[KV_STAGES], v_full[KV_STAGES],
-        v_empty[KV_STAGES], s_full[2], p_full[2], o_full;
-    __shared__ uint32_t tmem_base_smem;
-    __shared__ int abort_flag;
-
+    extern __shared__ __align__(1024) uint8_t smem_raw[];
     uint8_t* base = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~(uintptr_t)1023);
+    Bars* bars;
+    if constexpr (CONTIG) {
+        if (base != smem_raw) {  // every thread alike: nothing has been set up yet
+            rfx::pdl_prologue();
+            if (threadIdx.x == 0) atomicExch(err, 26);
+            return;
+        }
+        bars = reinterpret_cast<Bars*>(base + Smem::tiles(DK, DV));
+    } else {
+        __shared__ __align__(8) Bars bars_static;
+        bars = &bars_static;
+    }
+    uint64_t &q_full = bars->q_full, &o_full = bars->o_full;
+    uint64_t *k_full = bars->k_full, *k_empty = bars->k_empty, *v_full = bars->v_full, *v_empty = bars->v_empty,
+             *s_full = bars->s_full, *p_full = bars->p_full;
+    uint32_t& tmem_base_smem = bars->tmem_base;
+    int& abort_flag = bars->abort_flag;
     uint8_t* q_tile = base;
-    uint8_t* k_ring = q_tile + ROWS * D * 2;
-    uint8_t* v_ring = k_ring + KV_STAGES * KV_BYTES;
+    uint8_t* k_ring = q_tile + ROWS * DK * 2;
+    uint8_t* v_ring = k_ring + KV_STAGES * K_BYTES;
 
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     if (threadIdx.x == 0) trace_mark(0);  // 0 entry, 1 set up, 2 first scores, 3 last page done, 4 output written, 5 exit
@@ -201,33 +235,62 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q,
             mbar_expect_tx(&q_full, (uint32_t)(bq * g * 128 * KB));
             for (int kb = 0; kb < KB; ++kb)
                 tma_load_3d(q_tile + kb * ROWS * 128, &map_q, &q_full, kb * 64, kvh * g, row0 + q0);
-            for (int j = 0; j < n_pages; ++j) {
+            // the tile's first row in the store (or in the matrix), and its first columns
+            const int row_base = CONTIG ? seq_base[seq] : 0;
+            auto y_of = [&](int j) {
+                return CONTIG ? row_base + logical(j) * PAGE : (table[logical(j)] * cache.n_kv_heads + kvh) * PAGE;
+            };
+            const int kx = CONTIG ? kvh * DK : 0, vx = CONTIG ? v_col + kvh * DV : 0;
+            auto load_k = [&](int j, int y) -> bool {
                 const int s = j % KV_STAGES;
-                const uint32_t ph = (j / KV_STAGES) & 1;
-                const int page = table[logical(j)];
-                const int y = (page * cache.n_kv_heads + kvh) * PAGE;
-                if (!mbar_wait(&k_empty[s], ph ^ 1)) { atomicExch(err, 11); abort_flag = 1; break; }
-                mbar_expect_tx(&k_full[s], KV_BYTES);
+                if (!mbar_wait(&k_empty[s], ((j / KV_STAGES) & 1) ^ 1)) { atomicExch(err, 11); return false; }
+                mbar_expect_tx(&k_full[s], K_BYTES);
                 for (int kb = 0; kb < KB; ++kb)
-                    tma_load_2d(k_ring + s * KV_BYTES + kb * PAGE * 128, &map_k, &k_full[s], kb * 64, y);
-                if (!mbar_wait(&v_empty[s], ph ^ 1)) { atomicExch(err, 12); abort_flag = 1; break; }
-                mbar_expect_tx(&v_full[s], KV_BYTES);
-                for (int kb = 0; kb < KB; ++kb)
-                    tma_load_2d(v_ring + s * KV_BYTES + kb * PAGE * 128, &map_v, &v_full[s], kb * 64, y);
+                    tma_load_2d(k_ring + s * K_BYTES + kb * PAGE * 128, &map_k, &k_full[s], kx + kb * 64, y);
+                return true;
+            };
+            auto load_v = [&](int j, int y) -> bool {
+                const int s = j % VS;
+                if (!mbar_wait(&v_empty[s], ((j / VS) & 1) ^ 1)) { atomicExch(err, 12); return false; }
+                mbar_expect_tx(&v_full[s], V_BYTES);
+                for (int kb = 0; kb < VB; ++kb)
+                    tma_load_2d(v_ring + s * V_BYTES + kb * PAGE * 128, &map_v, &v_full[s], vx + kb * 64, y);
+                return true;
+            };
+            bool ok = true;
+            if constexpr (VS == 1) {
+                // one value tile: the next page's keys are asked for before this page's values, whose
+                // tile comes free late
+                int y_next = y_of(0);
+                ok = load_k(0, y_next);
+                for (int j = 0; j < n_pages && ok; ++j) {
+                    const int y = y_next;
+                    if (j + 1 < n_pages) {
+                        y_next = y_of(j + 1);
+                        ok = load_k(j + 1, y_next);
+                    }
+                    ok = ok && load_v(j, y);
+                }
+            } else {
+                for (int j = 0; j < n_pages && ok; ++j) {
+                    const int y = y_of(j);
+                    ok = load_k(j, y) && load_v(j, y);
+                }
             }
+            if (!ok) abort_flag = 1;
         }
         __syncwarp();
     } else if (warp == 1) {
         if (elect_one()) {
             constexpr uint32_t idesc_s = umma_idesc_bf16(ROWS, PAGE);  // S: N = 64 keys
-            constexpr uint32_t idesc_o = idesc_b_mn(ROWS, D);          // O: N = D, V is MN-major
+            constexpr uint32_t idesc_o = idesc_b_mn(ROWS, DV);         // O: N = DV, V is MN-major
             const bool tracing = g_trace != nullptr;
             long long wait_k = 0, wait_p = 0, wait_v = 0, c0 = 0;
             bool ok = mbar_wait(&q_full, 0);
             if (!ok) { atomicExch(err, 13); abort_flag = 1; }
             auto pv = [&](int i) -> bool {
-                const int b = i & 1, s = i % KV_STAGES;
-                const uint32_t ph2 = (i >> 1) & 1, phs = (i / KV_STAGES) & 1;
+                const int b = i & 1, s = i % VS;
+                const uint32_t ph2 = (i >> 1) & 1, phs = (i / VS) & 1;
                 // P_i is delivered after any rescaling of O that page i asked for
                 if (tracing) c0 = clock64();
                 if (!mbar_wait(&p_full[b], ph2)) { atomicExch(err, 14); return false; }
@@ -235,7 +298,7 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q,
                 if (!mbar_wait(&v_full[s], phs)) { atomicExch(err, 15); return false; }
                 if (tracing) wait_v += clock64() - c0;
                 tc_fence_after_sync();
-                const uint32_t va = smem_u32(v_ring + s * KV_BYTES);
+                const uint32_t va = smem_u32(v_ring + s * V_BYTES);
 #pragma unroll
                 for (int k = 0; k < PAGE / 16; ++k) {  // 16 keys per MMA: 8 packed columns of P
                     const uint64_t db = umma_desc_mn_sw128(va + k * 16 * 128, PAGE * 128, 1024);
@@ -255,7 +318,7 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q,
                 if (!mbar_wait(&k_full[s], phs)) { atomicExch(err, 18); ok = false; break; }
                 if (tracing) wait_k += clock64() - c0;
                 tc_fence_after_sync();
-                const uint32_t qa = smem_u32(q_tile), ka = smem_u32(k_ring + s * KV_BYTES);
+                const uint32_t qa = smem_u32(q_tile), ka = smem_u32(k_ring + s * K_BYTES);
 #pragma unroll
                 for (int kb = 0; kb < KB; ++kb)
 #pragma unroll
@@ -379,7 +442,7 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q,
                 if (!mbar_wait(&o_full, (uint32_t)((j - 1) & 1))) { atomicExch(err, 21); ok = false; break; }
                 tc_fence_after_sync();
 #pragma unroll
-                for (int c = 0; c < D / 16; ++c) {
+                for (int c = 0; c < DV / 16; ++c) {
                     uint32_t o[16];
                     tmem_ld_16_nowait(tmem + lane_addr + O_COL + c * 16, o);
                     tmem_ld_wait();
@@ -396,14 +459,15 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q,
             tmem_st_16(tmem + lane_addr + S_COL + b * PAGE + 16, packed + 16);
             tmem_st_wait();
             // the last page may hold keys past this tile's last position whose
-            // value rows were never written: zero them, 0 * NaN would not be 0
-            const int valid_keys = pos_last + 1 - basej;
+            // value rows were never written: zero them, 0 * NaN would not be 0 (a matrix has no such
+            // rows: what lies behind a sequence is the next one's, and zeros behind the last)
+            const int valid_keys = CONTIG ? PAGE : pos_last + 1 - basej;
             if (valid_keys < PAGE) {
-                const int sidx = j % KV_STAGES;
-                if (!mbar_wait(&v_full[sidx], (j / KV_STAGES) & 1)) { atomicExch(err, 24); ok = false; break; }
-                uint8_t* vt = v_ring + sidx * KV_BYTES;
-                for (int i = t; i < (PAGE - valid_keys) * KB * 8; i += ROWS) {
-                    const int rrow = valid_keys + i / (KB * 8), rem = i % (KB * 8);
+                const int sidx = j % VS;
+                if (!mbar_wait(&v_full[sidx], (j / VS) & 1)) { atomicExch(err, 24); ok = false; break; }
+                uint8_t* vt = v_ring + sidx * V_BYTES;
+                for (int i = t; i < (PAGE - valid_keys) * VB * 8; i += ROWS) {
+                    const int rrow = valid_keys + i / (VB * 8), rem = i % (VB * 8);
                     *reinterpret_cast<uint4*>(vt + (rem / 8) * PAGE * 128 + rrow * 128 + (rem % 8) * 16) =
                         make_uint4(0, 0, 0, 0);
                 }
@@ -422,16 +486,17 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q,
             tc_fence_after_sync();
             // a sink adds exp(sink - reference) to the denominator, once, with no value
             const float inv = 1.0f / (sink ? l + ex2(fmaf(sink[kvh * g + row_h], 1.4426950408889634f, -m)) : l);
-            __nv_bfloat16* o = out + ((size_t)(row0 + q0 + row_p) * nq + kvh * g + row_h) * D;
+            const int ow = CONTIG ? dv : DV;  // columns of an output head
+            __nv_bfloat16* o = out + ((size_t)(row0 + q0 + row_p) * nq + kvh * g + row_h) * ow;
             // two loads of 16 columns in flight: the next one travels while this one is stored
             uint32_t rr[2][16];
             tmem_ld_16_nowait(tmem + lane_addr + O_COL, rr[0]);
 #pragma unroll
-            for (int c = 0; c < D / 16; ++c) {
+            for (int c = 0; c < DV / 16; ++c) {
                 tmem_ld_wait_16(rr[c & 1]);
-                if (c + 1 < D / 16) tmem_ld_16_nowait(tmem + lane_addr + O_COL + (c + 1) * 16, rr[(c + 1) & 1]);
+                if (c + 1 < DV / 16) tmem_ld_16_nowait(tmem + lane_addr + O_COL + (c + 1) * 16, rr[(c + 1) & 1]);
                 uint32_t(&r)[16] = rr[c & 1];
-                if (row_valid) {
+                if (row_valid && (!CONTIG || c * 16 < ow)) {
                     uint4 v[2];
                     __nv_bfloat162* pv2 = reinterpret_cast<__nv_bfloat162*>(v);
 #pragma unroll
@@ -484,8 +549,8 @@ int launch_tc(const void* q, const void* k_pages, const void* v_pages, long long
     if (!make_map_q(&mq, q, R, nq, D, g, bq) || !rfx::tma::make_map_rows64(&mk, k_pages, kv_rows, D, PAGE) ||
         !rfx::tma::make_map_rows64(&mv, v_pages, kv_rows, D, PAGE))
         return RFX_ERR_UNSUPPORTED;
-    const size_t smem = Smem::total(D);
-    auto kernel = attention_prefill_tc_kernel<D, MODE>;
+    const size_t smem = Smem::total(D, D, false);
+    auto kernel = attention_prefill_tc_kernel<D, D, MODE, false>;
     cudaError_t e = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     if (e != cudaSuccess) return (int)e;
     if ((max_new + bq - 1) / bq > 65535 || S > 65535) return RFX_ERR_UNSUPPORTED;
@@ -493,7 +558,42 @@ int launch_tc(const void* q, const void* k_pages, const void* v_pages, long long
     if (grid.y > 65535 || grid.z > 65535) return RFX_ERR_UNSUPPORTED;
     RFX_LAUNCH(kernel, grid, THREADS, smem, s, mq, mk, mv, cache, seq_slot, seq_start, seq_new, seq_row0,
                (__nv_bfloat16*)out, nq, bq, window, keep_first,
-               (MODE >= 2 ? softcap : scale) * 1.4426950408889634f, MODE >= 2 ? scale / softcap : 1.0f, sink, slopes, err);
+               (MODE >= 2 ? softcap : scale) * 1.4426950408889634f, MODE >= 2 ? scale / softcap : 1.0f, sink, slopes,
+               (const int*)nullptr, 0, D, err);
+    return 0;
+}
+
+// [rows, cols] bfloat16, row-major: boxes of 64 columns x 64 rows (rows beyond: zeros)
+bool make_map_matrix(CUtensorMap* map, const void* base, long long rows, long long cols) {
+    EncodeTiledFn fn = encode_fn();
+    if (!fn) return false;
+    cuuint64_t dims[2] = {(cuuint64_t)cols, (cuuint64_t)rows};
+    cuuint64_t strides[1] = {(cuuint64_t)cols * 2};
+    cuuint32_t box[2] = {64, PAGE};
+    cuuint32_t estr[2] = {1, 1};
+    return fn(map, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, const_cast<void*>(base), dims, strides, box, estr,
+              CU_TENSOR_MAP_INTERLEAVE_NONE, CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_256B,
+              CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE) == CUDA_SUCCESS;
+}
+
+template <int DK, int DV>
+int launch_contig(const void* q, const void* kv, long long kv_rows, const int* seq_base, const int* seq_slot,
+                  const int* seq_start, const int* seq_new, const int* seq_row0, void* out, int S, int max_new, int R,
+                  int heads, int dv, int window, float scale, const float* sink, int* err, cudaStream_t s) {
+    CUtensorMap mq, mkv;
+    if (!make_map_q(&mq, q, R, heads, DK, 1, ROWS) ||
+        !make_map_matrix(&mkv, kv, kv_rows, (long long)heads * (DK + DV)))
+        return RFX_ERR_UNSUPPORTED;
+    const size_t smem = Smem::total(DK, DV, true);
+    auto kernel = attention_prefill_tc_kernel<DK, DV, 0, true>;
+    cudaError_t e = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    if (e != cudaSuccess) return (int)e;
+    dim3 grid(heads, S, (max_new + ROWS - 1) / ROWS);
+    if (grid.y > 65535 || grid.z > 65535) return RFX_ERR_UNSUPPORTED;
+    PagedKV cache{nullptr, 0, PAGE, heads, DK};
+    RFX_LAUNCH(kernel, grid, THREADS, smem, s, mq, mkv, mkv, cache, seq_slot, seq_start, seq_new, seq_row0,
+               (__nv_bfloat16*)out, heads, ROWS, window, 0, scale * 1.4426950408889634f, 1.0f, sink,
+               (const float*)nullptr, seq_base, heads * DK, dv, err);
     return 0;
 }
 
@@ -561,4 +661,27 @@ extern "C" int rfx_attention_prefill_tc(const void* q, const void* k_pages, cons
     return rfx_attention_prefill_tc_kf(q, k_pages, v_pages, n_pages_total, page_table, max_pages, page_size,
                                        seq_slot, seq_start, seq_new, seq_row0, out, S, max_new, R, nq, nkv,
                                        head_dim, window, 0, scale, sink, slopes, 0.0f, 0.0f, err, stream);
+}
+
+// Attention over keys and values that lie as rows of one matrix, one key and value per head
+// and position (a latent's, made for this step): `kv` bfloat16 [kv_rows, heads * (dk + dvp)], a
+// row's keys head by head, dk elements each, then its values, dvp each (dv of them used); position
+// p of sequence i is row seq_base[i] + p.  q [R, heads, dk], out [R, heads, dv].  dk: 64, 128 or
+// 192; dvp: 64 or 128, at most dk; dv a multiple of 16; scale > 0.
+extern "C" int rfx_attention_prefill_tc_rows(const void* q, const void* kv, long long kv_rows, const int* seq_base,
+                                             const int* seq_slot, const int* seq_start, const int* seq_new,
+                                             const int* seq_row0, void* out, int S, int max_new, int R, int heads,
+                                             int dk, int dvp, int dv, int window, float scale, const float* sink,
+                                             int* err, void* stream) {
+    if (S <= 0 || max_new <= 0 || R <= 0) return 0;
+    if (!(scale > 0.0f) || dv <= 0 || dv % 16 || dv > dvp || heads <= 0 || kv_rows <= 0) return RFX_ERR_UNSUPPORTED;
+    if ((reinterpret_cast<uintptr_t>(q) | reinterpret_cast<uintptr_t>(kv) | reinterpret_cast<uintptr_t>(out)) & 15)
+        return RFX_ERR_BAD_ARG;
+#define RFX_CASE(A, B)                                                                                              \
+    if (dk == A && dvp == B)                                                                                        \
+        return launch_contig<A, B>(q, kv, kv_rows, seq_base, seq_slot, seq_start, seq_new, seq_row0, out, S,        \
+                                   max_new, R, heads, dv, window, scale, sink, err, (cudaStream_t)stream);
+    RFX_CASE(64, 64) RFX_CASE(128, 64) RFX_CASE(128, 128) RFX_CASE(192, 64) RFX_CASE(192, 128)
+#undef RFX_CASE
+    return RFX_ERR_UNSUPPORTED;
 }

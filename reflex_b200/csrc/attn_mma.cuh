@@ -241,11 +241,13 @@ __device__ __forceinline__ const __nv_bfloat16* tile_at(const __nv_bfloat16* til
 //   pen[i] * (dist0 - j) is taken off its scaled score for the thread's i-th head
 //   (slope times log2(e)).
 //   MODE 2: capped scores (`capped_log2`), pen[0] its `in2`, pen[1] its `out2`
-template <int D, bool SWZ = false, int MODE = 0, typename Visible>
+//   DV: columns of the values (the first DV of the tile's rows; `vs` may be `ks`, rows that
+//   are keys and values at once)
+template <int D, bool SWZ = false, int MODE = 0, int DV = D, typename Visible>
 __device__ __forceinline__ void attend_keys16(const uint32_t (&qf)[D / 16][2], const __nv_bfloat16* ks,
                                               const __nv_bfloat16* vs, int key0, float scale_log2,
                                               Visible visible, const float (&pen)[2], int dist0,
-                                              float (&m)[2], float (&l)[2], float (&acc)[D / 16][4]) {
+                                              float (&m)[2], float (&l)[2], float (&acc)[DV / 16][4]) {
     const int lane = threadIdx.x & 31;
     float s[4] = {0.0f, 0.0f, 0.0f, 0.0f};
 #pragma unroll
@@ -293,7 +295,7 @@ __device__ __forceinline__ void attend_keys16(const uint32_t (&qf)[D / 16][2], c
     l[0] = l[0] * corr[0] + (e[0] + e[2]);
     l[1] = l[1] * corr[1] + (e[1] + e[3]);
 #pragma unroll
-    for (int i = 0; i < D / 16; ++i) {
+    for (int i = 0; i < DV / 16; ++i) {
         acc[i][0] *= corr[0];
         acc[i][1] *= corr[1];
         acc[i][2] *= corr[0];
@@ -303,7 +305,7 @@ __device__ __forceinline__ void attend_keys16(const uint32_t (&qf)[D / 16][2], c
     const uint32_t b0 = movmatrix_trans(pack_bf16(e[0], e[1]));
     const uint32_t b1 = movmatrix_trans(pack_bf16(e[2], e[3]));
 #pragma unroll
-    for (int i = 0; i < D / 16; ++i) {
+    for (int i = 0; i < DV / 16; ++i) {
         uint32_t a[4];
         ldmatrix_x4_trans(a, tile_at<D, SWZ>(vs, key0 + (lane & 7) + 8 * (lane >> 4), i * 16 + 8 * ((lane >> 3) & 1)));
         mma_bf16(acc[i], a, b0, b1);

@@ -10,8 +10,8 @@
 //    (32-bit); with `v_first` and `lambda` they become (1 - lambda) v + lambda v_first
 //    before they are cached.
 //  * rfx_latent_rot_post: rows [q | latent | shared key part]: per head the unrotated
-//    part of q goes out on its own (the product with W_uk follows), the rotated part
-//    turns and goes into the columns behind the absorbed query; the latent, over its root
+//    part of q and the turned rotated part with zeros behind it go to places of the caller's
+//    (apart, where the product with W_uk follows; side by side as one query); the latent, over its root
 //    mean square and times a weight, and the turned key part go into the page of the
 //    row's position as one row [latent | key part | zeros].
 //
@@ -167,9 +167,9 @@ template <typename TI, typename TO, bool BY4>
 __global__ void __launch_bounds__(RP_THREADS)
 latent_rot_post_kernel(const TI* __restrict__ proj, int ldp, const float* __restrict__ kv_w, float eps,
                        const float* __restrict__ denom, const int* __restrict__ row_pos,
-                       const int* __restrict__ row_slot, TO* __restrict__ q_flat, TO* __restrict__ q_abs,
-                       TO* __restrict__ pages, PagedKV cache, int H, int d, int rot, int rank, int width,
-                       int writes_cache) {
+                       const int* __restrict__ row_slot, TO* __restrict__ q_flat, int flat_h,
+                       TO* __restrict__ q_rot, int rot_h, int rot_w, TO* __restrict__ pages, PagedKV cache, int H,
+                       int d, int rot, int rank, int width, int writes_cache) {
     extern __shared__ float cs[];
     pdl_prologue();
     const int r = blockIdx.x;
@@ -178,20 +178,20 @@ latent_rot_post_kernel(const TI* __restrict__ proj, int ldp, const float* __rest
     angles(cs, denom, half, pos);
     const int lane = threadIdx.x & 31;
     const TI* row = proj + (size_t)r * ldp;
-    auto turn_into = [&](TO* dst, const TI* x) {  // the rotated part and the zeros behind it
-        for (int e = lane; e < width - rank; e += 32)
+    auto turn_into = [&](TO* dst, const TI* x, int n) {  // the rotated part and the zeros behind it
+        for (int e = lane; e < n; e += 32)
             st<TO>(dst, e, e < rot ? turned(ld<TI>(x, e), ld<TI>(x, e < half ? e + half : e - half), e, cs, half) : 0.0f);
     };
     const int units = H + (writes_cache ? 1 : 0);
     for (int u = blockIdx.y * RP_WARPS + (threadIdx.x >> 5); u < units; u += gridDim.y * RP_WARPS) {
         if (u < H) {
             const TI* x = row + (size_t)u * (d + rot);
-            TO* flat = q_flat + ((size_t)r * H + u) * d;
+            TO* flat = q_flat + ((size_t)r * H + u) * flat_h;
             if constexpr (BY4)
                 for (int e = 4 * lane; e < d; e += 128) store4(flat + e, load4(x + e));
             else
                 for (int e = lane; e < d; e += 32) st<TO>(flat, e, ld<TI>(x, e));
-            turn_into(q_abs + ((size_t)r * H + u) * width + rank, x + d);
+            turn_into(q_rot + ((size_t)r * H + u) * rot_h, x + d, rot_w);
         } else {
             const TI* x = row + (size_t)H * (d + rot);
             TO* dst = pages + kv_offset(cache, slot, pos, 0);
@@ -216,7 +216,7 @@ latent_rot_post_kernel(const TI* __restrict__ proj, int ldp, const float* __rest
             } else {
                 for (int e = lane; e < rank; e += 32) st<TO>(dst, e, (ld<TI>(x, e) * f) * kv_w[e]);
             }
-            turn_into(dst + rank, x + rank);
+            turn_into(dst + rank, x + rank, width - rank);
         }
     }
 }
@@ -268,21 +268,23 @@ extern "C" int rfx_rot_qkv_post(const void* proj, int in_dt, int ld, const float
     return 0;
 }
 
-// `width`: elements of a cached row and of an absorbed query head (at least rank + rot; zeros
-// behind them).  q_flat [R, H d], q_abs [R, H width] (only the columns from `rank` on are written).
+// `width`: elements of a cached row (at least rank + rot; zeros behind them).  Of head h of row r
+// the unrotated d elements go to q_flat + (r H + h) flat_h, the turned ones and zeros, rot_w in all,
+// to q_rot + (r H + h) rot_h.
 extern "C" int rfx_latent_rot_post(const void* proj, int in_dt, int ld, const float* kv_w, float eps,
                                    const float* denom, const int* row_pos, const int* row_slot, void* q_flat,
-                                   void* q_abs, void* pages, int out_dt, const int* page_table, int max_pages,
+                                   int flat_h, void* q_rot, int rot_h, int rot_w, void* pages, int out_dt, const int* page_table, int max_pages,
                                    int page_size, int R, int H, int d, int rot, int rank, int width,
                                    int writes_cache, void* stream) {
     if (R <= 0) return 0;
-    if (H <= 0 || d <= 0 || rank <= 0 || rot < 0 || rot % 2 || width < rank + rot ||
+    if (H <= 0 || d <= 0 || rank <= 0 || rot < 0 || rot % 2 || width < rank + rot || flat_h < d || rot_h < rot_w ||
+        rot_w < rot ||
         ld < H * (d + rot) + (writes_cache ? rank + rot : 0))
         return RFX_ERR_BAD_ARG;
     PagedKV cache{page_table, max_pages, page_size, 1, width};
     cudaStream_t s = (cudaStream_t)stream;
     const uintptr_t in_al = in_dt == RFX_DT_F32 ? 16 : 8, out_al = out_dt == RFX_DT_F32 ? 16 : 8;
-    const bool by4 = d % 4 == 0 && rot % 4 == 0 && rank % 4 == 0 && width % 4 == 0 && ld % 4 == 0 &&
+    const bool by4 = d % 4 == 0 && rot % 4 == 0 && rank % 4 == 0 && width % 4 == 0 && ld % 4 == 0 && flat_h % 4 == 0 &&
                      aligned(proj, in_al) && aligned(kv_w, 16) && aligned(q_flat, out_al) && aligned(pages, out_al);
     dim3 grid(R, rows_blocks(R, H + 1));
     const size_t smem = (size_t)(rot > 0 ? rot : 1) * sizeof(float);
@@ -290,11 +292,11 @@ extern "C" int rfx_latent_rot_post(const void* proj, int in_dt, int ld, const fl
     do {                                                                                                            \
         if (by4)                                                                                                    \
             RFX_LAUNCH((latent_rot_post_kernel<TI, TO, true>), grid, RP_THREADS, smem, s, (const TI*)proj, ld,      \
-                       kv_w, eps, denom, row_pos, row_slot, (TO*)q_flat, (TO*)q_abs, (TO*)pages, cache, H, d, rot,  \
+                       kv_w, eps, denom, row_pos, row_slot, (TO*)q_flat, flat_h, (TO*)q_rot, rot_h, rot_w, (TO*)pages, cache, H, d, rot,  \
                        rank, width, writes_cache);                                                                  \
         else                                                                                                        \
             RFX_LAUNCH((latent_rot_post_kernel<TI, TO, false>), grid, RP_THREADS, smem, s, (const TI*)proj, ld,     \
-                       kv_w, eps, denom, row_pos, row_slot, (TO*)q_flat, (TO*)q_abs, (TO*)pages, cache, H, d, rot,  \
+                       kv_w, eps, denom, row_pos, row_slot, (TO*)q_flat, flat_h, (TO*)q_rot, rot_h, rot_w, (TO*)pages, cache, H, d, rot,  \
                        rank, width, writes_cache);                                                                  \
     } while (0)
     if (in_dt == RFX_DT_F32 && out_dt == RFX_DT_F32) RFX_GO(float, float);

@@ -1717,26 +1717,126 @@ def rot_qkv_post(proj: torch.Tensor, bias: Optional[torch.Tensor], rotation, uni
 
 def latent_rot_post(proj: torch.Tensor, kv_weight: torch.Tensor, eps: float, rotation, row_pos, row_slot, pages,
                     page_table, page_size: int, heads: int, dim: int, rot_dim: int, rank: int, width: int,
-                    writes_cache: bool, out_dtype: torch.dtype):
-    """Rows [q | latent | shared key part]: returns (q_flat [R, heads * dim], the
-    unrotated parts of q; q_abs [R, heads * width], whose columns from `rank` on of
-    every head hold the rotated part and zeros, the rest still to be filled), and
-    writes [latent / rms(latent) * kv_weight | rotated key part | zeros], `width`
-    elements, into the cache at the rows' positions."""
+                    writes_cache: bool, out_dtype: torch.dtype, query_width: int = 0):
+    """Rows [q | latent | shared key part]: writes [latent / rms(latent) * kv_weight |
+    rotated key part | zeros], `width` elements, into the cache at the rows'
+    positions, and returns the queries with their last `rot_dim` elements rotated.
+    `query_width` 0: apart, (q_flat [R, heads * dim], the unrotated parts; q_abs [R,
+    heads * width], whose columns from `rank` on of every head hold the rotated part
+    and zeros, the rest still to be filled).  Else as they are, zeros behind them:
+    [R, heads * query_width]."""
     R = proj.shape[0]
     denom, rot = _plain_rotation(rotation, "latent_rot_post")
     if rot not in (0, rot_dim):
         raise InvalidInput("latent_rot_post: the rotation covers the whole rotated part")
-    flat = _new((R, heads * dim), out_dtype, proj.device)
-    qa = _new((R, heads * width), out_dtype, proj.device)
+    esize = 4 if out_dtype == torch.float32 else 2
+    if query_width:
+        flat = _new((R, heads * query_width), out_dtype, proj.device)
+        out, flat_h, rot_h, rot_w = flat, query_width, query_width, query_width - dim
+        rot_ptr = flat.data_ptr() + esize * dim
+    else:
+        flat = _new((R, heads * dim), out_dtype, proj.device)
+        qa = _new((R, heads * width), out_dtype, proj.device)
+        out, flat_h, rot_h, rot_w = (flat, qa), dim, width, width - rank
+        rot_ptr = qa.data_ptr() + esize * rank
     st = native.lib().rfx_latent_rot_post(
         _chk(proj, "proj"), dt_code(proj.dtype), proj.shape[1], _chk(kv_weight, "kv_weight", torch.float32),
         float(eps), _chk(denom, "denominators", torch.float32), _chk(row_pos, "row_pos", torch.int32),
-        _chk(row_slot, "row_slot", torch.int32), flat.data_ptr(), qa.data_ptr(), _chk(pages, "pages", out_dtype),
-        dt_code(out_dtype), _chk(page_table, "page_table", torch.int32), page_table.shape[1], page_size, R, heads,
-        dim, rot_dim, rank, width, 1 if writes_cache else 0, _stream())
+        _chk(row_slot, "row_slot", torch.int32), flat.data_ptr(), flat_h, rot_ptr, rot_h, rot_w,
+        _chk(pages, "pages", out_dtype), dt_code(out_dtype), _chk(page_table, "page_table", torch.int32),
+        page_table.shape[1], page_size, R, heads, dim, rot_dim, rank, width, 1 if writes_cache else 0, _stream())
     native.check(st, f"latent_rot_post (rank={rank}, rot={rot_dim})")
-    return flat, qa
+    return out
+
+
+LATENT_WIDTH_STEP = 64   # cached latent rows the tensor-core kernels take: in steps of this, up to
+LATENT_MAX_WIDTH = 640
+
+
+def latent_decode(q: torch.Tensor, pages: torch.Tensor, page_table, page_size: int, row_pos, row_slot, nq: int,
+                  width: int, rank: int, window, scale: float, n_splits: int, early: bool,
+                  sink: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """bfloat16 tensor-core attention of folded queries [R, nq * width] over the cached
+    latent rows, keys and values at once, split over the keys; every row stands at one
+    position.  Returns the weighted latents, [R, nq * n] with n the width or 64
+    less, of which a head's first `rank` are what it asked for.  `early`: a row a
+    sequence (the pages before each row's own were written by earlier steps)."""
+    R = q.shape[0]
+    _chk(q, "q", torch.bfloat16)
+    dv = int(native.lib().rfx_latent_value_columns(width, rank))
+    out = _new((R, nq * dv), q.dtype, q.device)
+    pool_pages = int(pages.shape[0])
+
+    def run(partial, cluster):
+        return native.lib().rfx_latent_decode(
+            q.data_ptr(), _chk(pages, "pages", torch.bfloat16), _chk(page_table, "page_table", torch.int32),
+            page_table.shape[1], page_size, _chk(row_pos, "row_pos", torch.int32),
+            _chk(row_slot, "row_slot", torch.int32), out.data_ptr(), partial, R, nq, width, rank, n_splits,
+            int(window or 0), float(scale), _chk(sink, "sink", torch.float32), pool_pages, cluster, 1 if early else 0,
+            device_error_word(q.device).data_ptr(), _stream())
+
+    if CLUSTER_MERGE and n_splits in (2, 4, 8, 16):
+        st = run(0, 1)
+        if st != native.ERR_UNSUPPORTED:
+            native.check(st, f"latent_decode (width={width}, splits={n_splits})")
+            return out
+    partial = _new((R * nq * n_splits * (dv + 2),), torch.float32, q.device) if n_splits > 1 else None
+    native.check(run(partial.data_ptr() if partial is not None else 0, 0), f"latent_decode (width={width}, splits={n_splits})")
+    return out
+
+
+def latent_attention(q: torch.Tensor, pages: torch.Tensor, page_table, page_size: int, batch, nq: int, width: int,
+                     rank: int, window, scale: float, sink: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """Attention of folded queries over cached latent rows, [R, nq * (rank or more)];
+    picks the kernel."""
+    if q.dtype == torch.bfloat16 and width % LATENT_WIDTH_STEP == 0 and width <= LATENT_MAX_WIDTH:
+        ctx = batch.max_context
+        pages_seen = -(-min(ctx, window or ctx) // page_size) + (1 if window else 0)
+        return latent_decode(q, pages, page_table, page_size, batch.row_pos, batch.row_slot, nq, width, rank, window,
+                             scale, decode_splits(q.shape[0], nq, 1, pages_seen), batch.is_decode, sink=sink)
+    return attention(q, pages, pages, page_table, page_size, batch, nq, 1, width, window, scale, sink=sink)
+
+
+def latent_gather(pages: torch.Tensor, page_table, page_size: int, batch, width: int):
+    """The cached rows of the step's sequences, positions 0 up to each sequence's last
+    row of the step, as the rows of one matrix ([rows, width]), and each sequence's
+    first row in it (int32 [S], on the device)."""
+    n = sum(s + c for s, c in zip(batch.starts, batch.new_counts))
+    rows = _new((n, width), pages.dtype, pages.device)
+    base = _new((len(batch.starts),), torch.int32, pages.device)
+    st = native.lib().rfx_latent_gather(
+        _chk(pages, "pages", torch.bfloat16), _chk(page_table, "page_table", torch.int32), page_table.shape[1],
+        page_size, _chk(batch.seq_slot, "seq_slot", torch.int32), _chk(batch.seq_start, "seq_start", torch.int32),
+        _chk(batch.seq_new, "seq_new", torch.int32), rows.data_ptr(), base.data_ptr(), len(batch.starts),
+        max(s + c for s, c in zip(batch.starts, batch.new_counts)), width, _stream())
+    native.check(st, f"latent_gather (width={width})")
+    return rows, base
+
+
+def attention_prefill_tc_rows(q: torch.Tensor, kv: torch.Tensor, seq_base: torch.Tensor, batch, heads: int, dk: int,
+                              dvp: int, dv: int, window, scale: float, sink: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """tcgen05 attention of q [R, heads * dk] over keys and values that are the rows of
+    `kv` [rows, heads * (dk + dvp)] (all heads' keys, then all heads' values);
+    position p of sequence i is row seq_base[i] + p.  [R, heads * dv]."""
+    R = q.shape[0]
+    if kv.shape[1] != heads * (dk + dvp) or q.shape[1] != heads * dk:
+        raise InvalidInput("attention_prefill_tc_rows: q and kv do not match the heads")
+    out = _new((R, heads * dv), q.dtype, q.device)
+    st = native.lib().rfx_attention_prefill_tc_rows(
+        _chk(q, "q", torch.bfloat16), _chk(kv, "kv", torch.bfloat16), kv.shape[0], _chk(seq_base, "seq_base", torch.int32),
+        _chk(batch.seq_slot, "seq_slot", torch.int32), _chk(batch.seq_start, "seq_start", torch.int32),
+        _chk(batch.seq_new, "seq_new", torch.int32), _chk(batch.seq_row0, "seq_row0", torch.int32), out.data_ptr(),
+        batch.seq_slot.numel(), int(batch.max_new), R, heads, dk, dvp, dv, int(window or 0), float(scale),
+        _chk(sink, "sink", torch.float32), device_error_word(q.device).data_ptr(), _stream())
+    native.check(st, f"attention_prefill_tc_rows (dk={dk}, dv={dv})")
+    return out
+
+
+# From so many rows of a sequence on, a latent attention makes every head's keys and values of
+# the step's sequences (one product over the cached latents) and attends over those; fewer rows
+# fold the query through the key matrix and attend over the latents themselves.
+LATENT_EXPAND_MIN_ROWS = _env_int("REFLEX_B200_LATENT_EXPAND_MIN_ROWS", 65, 2, 1 << 30)
+LATENT_EXPAND_MAX_BYTES = 2 << 30
 
 
 # ------------------------------------------------------------------ sampling

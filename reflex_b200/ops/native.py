@@ -127,8 +127,17 @@ _SIGNATURES = {
     "rfx_rot_qkv_post": [c_void_p, c_int, c_int, c_void_p, c_void_p, c_int, c_int, c_float, c_void_p, c_void_p,
                          c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_int, c_int,
                          c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p],
-    "rfx_latent_rot_post": [c_void_p, c_int, c_int, c_void_p, c_float, c_void_p, c_void_p, c_void_p, c_void_p,
-                            c_void_p, c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int,
+    "rfx_latent_decode": [c_void_p, c_void_p, c_void_p, c_int, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_int,
+                          c_int, c_int, c_int, c_int, c_int, c_float, c_void_p, c_longlong, c_int, c_int, c_void_p,
+                          c_void_p],
+    "rfx_latent_gather": [c_void_p, c_void_p, c_int, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int,
+                          c_int, c_int, c_void_p],
+    "rfx_latent_value_columns": [c_int, c_int],
+    "rfx_attention_prefill_tc_rows": [c_void_p, c_void_p, c_longlong, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p,
+                                      c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_float,
+                                      c_void_p, c_void_p, c_void_p],
+    "rfx_latent_rot_post": [c_void_p, c_int, c_int, c_void_p, c_float, c_void_p, c_void_p, c_void_p, c_void_p, c_int,
+                            c_void_p, c_int, c_int, c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int,
                             c_int, c_int, c_void_p],
     "rfx_xielu": [c_void_p, c_int, c_longlong, c_float, c_float, c_void_p],
     "rfx_loop_input": [c_void_p, c_void_p, c_void_p, c_int, c_int, c_void_p],

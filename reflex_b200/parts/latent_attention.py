@@ -15,7 +15,10 @@ Without `q_rank` (the other form) q = W_q h, per head `head_dim` unrotated and
 rows: one rotated key part r_j all heads share, not normed:
   s_ij = (q_i . k_j + rot(q_i') . rot(r_j)) * scale
 The cached row is then [c | rot(r) | zeros], and the folded query is followed by
-its rotated part.
+its rotated part.  For a prompt's many rows the other order of the same products is
+cheaper: every head's keys [W_uk c | rot(r)] and values W_uv c of the step's
+sequences are made once from the cached rows, one product, and an ordinary
+attention runs over them.
 
 Since k_j = W_uk c_j, the score is
 (W_uk,h^T q_i) . c_j and the weighted values are W_uv,h (sum_j p_ij c_j): the
@@ -62,8 +65,15 @@ class LatentAttention:
             raise InvalidInput("latent_attention: a rotated part goes with queries straight from the input")
         if not self.q_rank and self.has_gate:
             raise InvalidInput("latent_attention: a gate goes with queries through a latent")
-        # elements of a cached row: the latent and the rotated part, in steps of 16 for the tensor cores
-        self.width = self.kv_rank if self.q_rank else (self.kv_rank + self.rot_dim + 15) // 16 * 16
+        # elements of a cached row: the latent and the rotated part, in steps the tensor-core kernels take
+        step = ops.LATENT_WIDTH_STEP if dtype == torch.bfloat16 else 16
+        self.width = self.kv_rank if self.q_rank else (self.kv_rank + self.rot_dim + step - 1) // step * step
+        # the form that makes every head's keys and values (prompts): padded key and value sizes
+        d, dv = spec.head_dim + self.rot_dim, spec.value_dim
+        self.dk, self.dvp = (d + 63) // 64 * 64, (dv + 63) // 64 * 64
+        self.expands = (not self.q_rank and dtype == torch.bfloat16 and self.dk <= 192 and self.dvp <= 128
+                        and self.dvp <= self.dk and dv % 16 == 0 and spec.scale > 0)
+        self.kv_up = None
         self.down = self.q_up = self.k_absorb = self.v_up = self.o = None
         self.q_norm = self.kv_norm = self.sink = None
 
@@ -118,6 +128,17 @@ class LatentAttention:
         self.v_up = dev(tensors["v_up"]).view(H, dv, self.kv_rank).contiguous()
         self.o = dev(tensors["o_proj"]).contiguous()
         self.kv_norm = f32(tensors["kv_norm"])
+        if self.expands:
+            # one matrix from a cached row to every head's key [W_uk c | rotated part | zeros] (the
+            # rotated part passes through) and value
+            rank, rot = self.kv_rank, self.rot_dim
+            up = torch.zeros((H * (self.dk + self.dvp), self.width), dtype=self.dtype, device=self.device)
+            keys = up[: H * self.dk].view(H, self.dk, self.width)
+            keys[:, :d, :rank] = dev(tensors["k_up"]).view(H, d, rank)
+            for j in range(rot):
+                keys[:, d + j, rank + j] = 1.0
+            up[H * self.dk:].view(H, self.dvp, self.width)[:, :dv, :rank] = dev(tensors["v_up"]).view(H, dv, rank)
+            self.kv_up = up
         self.sink = f32(tensors["sink"]) if self.has_sink else None
 
     def forward(self, x, ctx, residual=None):
@@ -156,18 +177,35 @@ class LatentAttention:
         H = s.num_heads
         proj = ops.linear(x, self.down, out_dtype=torch.float32)
         ops.prof_mark("qkv_gemm")
-        flat, qa = ops.latent_rot_post(
-            proj, self.kv_norm, self.eps, None if self.position is None else self.position.rotation(), batch.row_pos,
-            batch.row_slot, kv.k_pages, kv.page_table, kv.page_size, H, s.head_dim, self.rot_dim, self.kv_rank,
-            self.width, ctx.writes_cache, self.dtype)
-        ops.prof_mark("latent_post")
-        ops.heads_linear(flat, self.k_absorb, out=qa)
-        ops.prof_mark("q_absorb")
-        attn = ops.attention(qa, kv.k_pages, kv.k_pages, kv.page_table, kv.page_size, batch, H, 1, self.width,
-                             s.window, s.scale, sink=self.sink)
-        ops.prof_mark("attn")
-        vals = ops.heads_linear(attn, self.v_up)  # of each head the latent's elements; the rest is dropped
-        ops.prof_mark("v_up")
+        rotation = None if self.position is None else self.position.rotation()
+        post = (proj, self.kv_norm, self.eps, rotation, batch.row_pos, batch.row_slot, kv.k_pages, kv.page_table,
+                kv.page_size, H, s.head_dim, self.rot_dim, self.kv_rank, self.width, ctx.writes_cache, self.dtype)
+        if self._expand(batch):
+            q = ops.latent_rot_post(*post, query_width=self.dk)
+            ops.prof_mark("latent_post")
+            rows, base = ops.latent_gather(kv.k_pages, kv.page_table, kv.page_size, batch, self.width)
+            both = ops.linear(rows, self.kv_up)
+            ops.prof_mark("kv_up")
+            vals = ops.attention_prefill_tc_rows(q, both, base, batch, H, self.dk, self.dvp, s.value_dim, s.window,
+                                                 s.scale, sink=self.sink)
+            ops.prof_mark("attn")
+        else:
+            flat, qa = ops.latent_rot_post(*post)
+            ops.prof_mark("latent_post")
+            ops.heads_linear(flat, self.k_absorb, out=qa)
+            ops.prof_mark("q_absorb")
+            attn = ops.latent_attention(qa, kv.k_pages, kv.page_table, kv.page_size, batch, H, self.width,
+                                        self.kv_rank, s.window, s.scale, sink=self.sink)
+            ops.prof_mark("attn")
+            vals = ops.heads_linear(attn, self.v_up)  # of each head the latent's elements; the rest is dropped
+            ops.prof_mark("v_up")
         out = ops.linear(vals, self.o, out_dtype=torch.float32)
         ops.prof_mark("o_proj")
         return out
+
+    def _expand(self, batch) -> bool:
+        """Whether this step makes every head's keys and values: a prompt's rows share them."""
+        if not self.expands or batch.max_new < ops.LATENT_EXPAND_MIN_ROWS:
+            return False
+        rows = sum(a + b for a, b in zip(batch.starts, batch.new_counts))
+        return 2 * rows * self.spec.num_heads * (self.dk + self.dvp) <= ops.LATENT_EXPAND_MAX_BYTES

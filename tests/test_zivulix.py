@@ -67,7 +67,7 @@ def test_cache_needs_and_which_layers_mix_values():
 
     _typed, spec = spec_of(zm.ZIV_B)
     specs = CausalLM(spec, torch.float32, "cpu").cache_entry_specs()
-    assert specs[0] == KVSpec(1, 32, None, shared_kv=True)          # 18 + 4 in steps of 16
+    assert specs[0] == KVSpec(1, 32, None, shared_kv=True)          # 18 + 4 in steps of 16 (of 64 in bfloat16)
     assert specs[1] == StateSpec((2 * 7 * 12,), "float32")           # one tap: no filter state; 10 channels in fours
     assert specs[2] == KVSpec(1, 32, None)                           # the larger of 22 and 12 in steps of 16
     assert specs[3] == StateSpec((232 + 50 * 36,), "float32")        # 2 * 116 filter inputs, then S

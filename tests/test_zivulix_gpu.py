@@ -31,6 +31,7 @@ def batch_of(seqs, slots):
     b.is_decode = all(n == 1 for _, n in seqs)
     b.max_new = max(n for _, n in seqs)
     b.max_context = max(s + n for s, n in seqs)
+    b.starts, b.new_counts = [s for s, _ in seqs], [n for _, n in seqs]
     return b
 
 
@@ -300,7 +301,8 @@ def test_a_key_that_stands_out_far_away_and_at_the_windows_edges(kernel, window)
 
 
 @pytest.mark.parametrize("H,d,rot,dv,rank", [(3, 16, 8, 24, 40), (5, 6, 4, 10, 18), (4, 64, 16, 32, 112), (16, 32, 32, 48, 288),
-                                             (20, 24, 16, 40, 48)])
+                                             (20, 24, 16, 40, 48), (3, 128, 64, 128, 256), (2, 40, 24, 64, 512),
+                                             (2, 100, 20, 96, 600)])
 @pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
 def test_latent_attention_absorbed_equals_keys_and_values_per_head(H, d, rot, dv, rank, dtype):
     """The mixer without its output product over the framework's own cache: whole, in
@@ -325,13 +327,13 @@ def test_latent_attention_absorbed_equals_keys_and_values_per_head(H, d, rot, dv
     part.bind(dict(t))
     names = {"q_proj": "q", "kv_down": "dkv", "kv_norm": "dkv.norm", "k_up": "uk", "v_up": "uv", "o_proj": "o"}
     x = torch.randn(T, W, generator=g).to(dtype).float()
-    x[3] *= 20.0    # its rotated key part, which is not normed, is twenty times as long
+    x[3] *= 12.0    # its rotated key part, which is not normed, is twelve times as long
     x = x.to(dtype).float()
     ref = pz.latent_attention(x.double().numpy(), {names[k]: v.double().numpy() for k, v in t.items()}, m, 1e-5)
     without = x.clone()
     without[3] = x[4]
     moved = pz.latent_attention(without.double().numpy(), {names[k]: v.double().numpy() for k, v in t.items()}, m, 1e-5)
-    assert np.abs(ref[-40:] - moved[-40:]).max() > 0.1 * np.abs(ref).max()
+    assert np.abs(ref[-40:] - moved[-40:]).max() > 0.05 * np.abs(ref).max()
     cache = Cache({0: part.cache_spec()}, 1024, 1 << 20, dtype, torch.device(DEV))
 
     class Ctx:

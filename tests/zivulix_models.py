@@ -74,7 +74,7 @@ ZIV_C = model(200, 256, 1e-6, [
 ZIV_D = model(130, 128, 1e-5, [
     (latent(16, 32, 32, 48, 288, 0.25, 10000.0), 64),
     (delta(2, 2, 72, 160, 3), 64),
-    (latent(2, 8, 2, 8, 30, 1.0, 7.0), None),
+    (latent(2, 8, 2, 8, 30, 0.4, 7.0), None),
 ])
 # E: the first attention layer does not mix, the second is the first that does, two more follow;
 # long windows over several pages, values narrower than keys
