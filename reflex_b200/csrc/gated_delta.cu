@@ -21,8 +21,8 @@
 //    (g, c) holds its key channels 4 (g + KG m) .. + 3 in registers (NC groups of four); the
 //    KG partial sums of S^T k and of S^T q meet by shuffles.  The state lies
 //    [heads][value column][key channel padded to a multiple of four].  Which block and
-//    warp walks a column changes nothing of its arithmetic, and neither does the way
-//    the rows were cut into steps.
+//    warp walks a column changes nothing of its arithmetic.
+//    gated_delta_chunk.cu has the form for steps that bring a sequence many rows.
 #include "attn_mma.cuh"
 #include "common.cuh"
 #include "short_conv.cuh"

@@ -1656,16 +1656,37 @@ def gated_delta_prep(proj: torch.Tensor, b_off: int, a_off: int, filters_t: torc
     return out, gates
 
 
+# from so many rows of a sequence on, the recurrence takes them sixteen at a time as products
+GATED_DELTA_CHUNK_MIN_ROWS = _env_int("REFLEX_B200_GATED_DELTA_CHUNK_MIN_ROWS", 8, 1, 1 << 30)
+
+
 def gated_delta_scan(qkv: torch.Tensor, gates: torch.Tensor, state: torch.Tensor, state_off: int, batch, heads: int,
-                     kv_heads: int, dim: int, vdim: int) -> torch.Tensor:
+                     kv_heads: int, dim: int, vdim: int, exact: bool = False) -> torch.Tensor:
     """The gated delta rule over the step's rows (csrc/gated_delta.cu): `qkv` and
     `gates` as `gated_delta_prep` makes them; the running state is `state[slot,
     state_off : state_off + heads * vdim * (dim rounded up to 4)]`.  Returns S^T q,
-    float32 [R, heads * vdim]."""
+    float32 [R, heads * vdim].  From `GATED_DELTA_CHUNK_MIN_ROWS` rows of a sequence on
+    the kernel that takes sixteen rows at a time runs (csrc/gated_delta_chunk.cu: the
+    same function, products of 32-bit numbers split for the tensor cores); with
+    `exact`, and for fewer rows and other sizes, the row-by-row walk."""
     R = qkv.shape[0]
     if qkv.shape[1] != 2 * kv_heads * dim + heads * vdim or tuple(gates.shape) != (R, 2 * heads):
         raise InvalidInput("gated_delta_scan: the rows do not match the sizes")
     out = _new((R, heads * vdim), torch.float32, qkv.device)
+    if not exact and batch.max_new >= GATED_DELTA_CHUNK_MIN_ROWS and dim % 8 == 0 and vdim % 16 == 0 and dim <= 256:
+        S = batch.seq_slot.numel()
+        row0 = _chk(batch.seq_row0, "seq_row0", torch.int32)
+        coef = _new((int(native.lib().rfx_gated_delta_chunk_floats(R, S, heads)),), torch.float32, qkv.device)
+        st = native.lib().rfx_gated_delta_chunk_prep(
+            _chk(qkv, "qkv", torch.float32), _chk(gates, "gates", torch.float32), row0, S, coef.data_ptr(), heads,
+            kv_heads, dim, vdim, int(batch.max_new), _stream())
+        native.check(st, f"gated_delta_chunk_prep (heads={heads}, dim={dim})")
+        st = native.lib().rfx_gated_delta_chunk(
+            qkv.data_ptr(), coef.data_ptr(), _chk(state, "state", torch.float32), state.stride(0), int(state_off),
+            _chk(batch.seq_slot, "seq_slot", torch.int32), row0, S, out.data_ptr(), heads, kv_heads, dim, vdim,
+            _stream())
+        native.check(st, f"gated_delta_chunk (heads={heads}, dim={dim}, vdim={vdim})")
+        return out
     st = native.lib().rfx_gated_delta_scan(
         _chk(qkv, "qkv", torch.float32), _chk(gates, "gates", torch.float32), _chk(state, "state", torch.float32),
         state.stride(0), int(state_off), _chk(batch.seq_slot, "seq_slot", torch.int32),

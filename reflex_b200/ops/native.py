@@ -124,6 +124,10 @@ _SIGNATURES = {
                              c_void_p],
     "rfx_gated_delta_scan": [c_void_p, c_void_p, c_void_p, c_longlong, c_longlong, c_void_p, c_void_p, c_int, c_void_p,
                              c_int, c_int, c_int, c_int, c_int, c_void_p],
+    "rfx_gated_delta_chunk_prep": [c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_int, c_int,
+                                   c_void_p],
+    "rfx_gated_delta_chunk": [c_void_p, c_void_p, c_void_p, c_longlong, c_longlong, c_void_p, c_void_p, c_int, c_void_p,
+                               c_int, c_int, c_int, c_int, c_void_p],
     "rfx_rot_qkv_post": [c_void_p, c_int, c_int, c_void_p, c_void_p, c_int, c_int, c_float, c_void_p, c_void_p,
                          c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_int, c_int,
                          c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p],
@@ -206,6 +210,8 @@ def lib() -> ctypes.CDLL:
         handle.rfx_mlstm_state_floats.restype = c_int
         handle.rfx_mamba_scan_scratch.argtypes = [c_int, c_int, c_int, c_int]
         handle.rfx_mamba_scan_scratch.restype = c_longlong
+        handle.rfx_gated_delta_chunk_floats.argtypes = [c_int, c_int, c_int]
+        handle.rfx_gated_delta_chunk_floats.restype = c_longlong
         handle.rfx_sm_count.argtypes = []
         handle.rfx_sm_count.restype = c_int
         handle.rfx_sample_work_bytes.argtypes = [c_int, c_int]

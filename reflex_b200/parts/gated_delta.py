@@ -101,7 +101,8 @@ class GatedDelta:
         if not single:
             ops.conv_state_update(proj, 0, self.channels, None, self.taps, state, batch)
         ops.prof_mark("conv_post")
-        o = ops.gated_delta_scan(qkv, gates, state, self.state_off, batch, self.heads, self.kv_heads, self.dim, self.vdim)
+        o = ops.gated_delta_scan(qkv, gates, state, self.state_off, batch, self.heads, self.kv_heads, self.dim, self.vdim,
+                                 exact=self.dtype == torch.float32)
         ops.prof_mark("scan")
         o = ops.group_norm_gate(o, self.norm, self.eps, self.heads, self.dtype, gate=proj, gate_col=self.gate_col,
                                 activation="silu")

@@ -410,11 +410,12 @@ def test_gated_delta_rule_carried_through_its_state(H, G, d, dv, taps, dtype):
             assert relerr(np.concatenate(got[i]), refs[i]) < tol(dtype, 1e-4, 3e-2), (cuts, i)
 
 
-def test_a_slow_decay_keeps_a_far_write_and_a_write_rate_of_one_replaces_it():
+@pytest.mark.parametrize("exact", [True, False])
+def test_a_slow_decay_keeps_a_far_write_and_a_write_rate_of_one_replaces_it(exact):
     """One head: a value written under one key is read 400 tokens later when the decay is
     one and other tokens write under another key; it is gone after one write under the
     same key at a rate of one, and after one token with a decay of zero."""
-    d, dv, T = 8, 4, 401
+    d, dv, T = 8, 16, 401
     for what in ("kept", "replaced", "decayed"):
         q, k, v = np.zeros((T, d)), np.zeros((T, d)), np.zeros((T, dv))
         q[:, 0] = 1.0
@@ -429,9 +430,49 @@ def test_a_slow_decay_keeps_a_far_write_and_a_write_rate_of_one_replaces_it():
             decay[200] = 0.0
         state = torch.zeros(1, dv * d, device=DEV)
         o = ops().gated_delta_scan(f32(np.concatenate([q, k, v], axis=1)), f32(np.concatenate([decay, rate], axis=1)),
-                                   state, 0, batch_of([(0, T)], [0]), 1, 1, d, dv).cpu().numpy()
+                                   state, 0, batch_of([(0, T)], [0]), 1, 1, d, dv, exact=exact).cpu().numpy()
         assert abs(o[0, 2] - 7.0) < 1e-5 and abs(o[199, 2] - 7.0) < 1e-5
         assert abs(o[-1, 2] - (7.0 if what == "kept" else 0.0)) < 1e-5, what
+
+
+@pytest.mark.parametrize("H,G,d,dv", [(4, 2, 64, 64), (3, 3, 24, 16), (6, 2, 128, 128), (2, 1, 96, 48), (1, 1, 256, 32),
+                                      (2, 2, 200, 80)])
+def test_sixteen_rows_at_a_time_equal_the_row_by_row_walk(H, G, d, dv):
+    """Sequences of lengths around the chunks' edges beside one another, states that are not
+    zero at the start, strong and weak decays: both kernels against the plain recurrence,
+    and far closer to it than products of rounded operands would be."""
+    g = torch.Generator().manual_seed(H + d)
+    lens = [8, 15, 16, 17, 33, 1, 100]
+    R, n = sum(lens), len(lens)
+    q, k = torch.randn(R, G, d, generator=g), torch.randn(R, G, d, generator=g)
+    k[20:30] = k[20:21]    # the same key many times within a chunk
+    q, k = torch.nn.functional.normalize(q, dim=-1), torch.nn.functional.normalize(k, dim=-1)
+    v = torch.randn(R, H, dv, generator=g)
+    decay, rate = torch.rand(R, H, generator=g) ** 0.2, torch.rand(R, H, generator=g)
+    decay[5], decay[40] = 1e-12, 1.0
+    rate[22:26] = 1.0
+    S0 = torch.randn(n, H, dv, d, generator=g)
+    qkv = torch.cat([q.reshape(R, -1), k.reshape(R, -1), v.reshape(R, -1)], dim=1).to(DEV)
+    gates = torch.cat([decay, rate], dim=1).to(DEV)
+    refs, ends, r = [], [], 0
+    for i, m in enumerate(lens):
+        S = S0[i].double().numpy().transpose(0, 2, 1).copy()
+        for t in range(r, r + m):
+            o = np.zeros((H, dv))
+            for h in range(H):
+                kt, qt = k[t, h // (H // G)].double().numpy(), q[t, h // (H // G)].double().numpy()
+                S[h] = float(decay[t, h]) * S[h]
+                S[h] += np.outer(kt, float(rate[t, h]) * (v[t, h].double().numpy() - S[h].T @ kt))
+                o[h] = S[h].T @ qt
+            refs.append(o.reshape(-1))
+        ends.append(S.transpose(0, 2, 1))
+        r += m
+    for exact in (True, False):
+        state = torch.cat([torch.full((n, 4), 3.0), S0.reshape(n, -1)], dim=1).to(DEV).contiguous()
+        o = ops().gated_delta_scan(qkv, gates, state, 4, batch_of([(0, m) for m in lens], list(range(n))), H, G, d, dv,
+                                   exact=exact)
+        assert relerr(o, np.stack(refs)) < 5e-6, exact
+        assert relerr(state[:, 4:].reshape(n, H, dv, d), np.stack(ends)) < 5e-6 and bool((state[:, :4] == 3.0).all())
 
 
 def test_a_layer_that_mixes_values_needs_the_first_ones():
