@@ -16,16 +16,17 @@
 // (x = hi + lo exactly up to 2^-22; hi hi + hi lo + lo hi, 32-bit sums): 32-bit products up
 // to about 2^-21 of their size.  The true 32-bit path takes the row-by-row kernel instead.
 //
-// A warp owns sixteen value columns and all key channels: S^T [16 columns x d] is the
-// accumulator tile row of mma.sync m16n8k8, and, with the channels of every eight taken in the
-// order (0, 2, 4, 6, 1, 3, 5, 7), the same registers are the left operand of the next
-// chunk's products; likewise u^T.
+// S^T [16 columns x channels] of a warp is an accumulator tile row of mma.sync m16n8k8, and,
+// with the channels of every eight taken in the order (0, 2, 4, 6, 1, 3, 5, 7), the same
+// registers are the left operand of the next chunk's products; likewise u^T.
 #include "attn_mma.cuh"
 #include "common.cuh"
+#include "sm100.cuh"
 
 namespace {
 
 constexpr int CH = 16;            // rows of a chunk
+constexpr int MAX_STAGES = 4;     // chunks in flight of a block
 constexpr int TLD = 24;           // row stride of T and M: a fragment's 8-byte loads meet all banks
 // per chunk and head: T [16][TLD], M [16][TLD], c [16], r_last [16], c_last and padding
 constexpr int COEF = 2 * CH * TLD + 2 * CH + 4;
@@ -77,6 +78,14 @@ __device__ __forceinline__ void product3(float (&d)[N][4], const Left& a, const 
     for (int n = 0; n < N; ++n) mma_tf32(d[n], a.hi, x[n].lo, y[n].lo);
 #pragma unroll
     for (int n = 0; n < N; ++n) mma_tf32(d[n], a.hi, x[n].hi, y[n].hi);
+}
+
+// `bytes` (a multiple of 16, both addresses 16-byte aligned) into shared memory, counted on `bar`.
+__device__ __forceinline__ void bulk_load(void* dst, const void* src, int bytes, uint64_t* bar) {
+    asm volatile("cp.async.bulk.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1], %2, [%3];" ::"r"(
+                     sm100::smem_u32(dst)),
+                 "l"(src), "r"(bytes), "r"(sm100::smem_u32(bar))
+                 : "memory");
 }
 
 // Chunk c of sequence `seq`, whose first row of the step is row0: its place among all chunks
@@ -153,75 +162,99 @@ gated_delta_chunk_prep_kernel(const float* __restrict__ qkv, const float* __rest
     }
 }
 
-template <int NT>  // key channels in eights (channels beyond d are zeros)
-__global__ void __launch_bounds__(128)
+// Four warps own sixteen value columns, a quarter of the key channels each (NT eights; channels
+// beyond d are zeros); a block has up to four such groups and one more warp that only brings the
+// chunks: rows, values and coefficients by bulk copies, `stages` chunks in flight, a barrier per
+// buffer for the bytes and one for the warps that are done with it.  The four quarters'
+// partial sums of K S0 and Q S0 meet in shared memory in their order; u is solved by every
+// warp of the group (each needs it for its channels), o by one of them in turn.
+template <int NT>
+__global__ void __launch_bounds__(544)
 gated_delta_chunk_kernel(const float* __restrict__ qkv, const float* __restrict__ coef, float* __restrict__ state,
                          long long state_stride, long long state_off, const int* __restrict__ seq_slot,
                          const int* __restrict__ seq_row0, float* __restrict__ out, int H, int G, int d, int dv,
-                         int cols) {
-    constexpr int LDK = 8 * NT + 8;
+                         int cols, int stages, int* __restrict__ err) {
+    constexpr int DP = 32 * NT, LDK = DP + 8;
     extern __shared__ __align__(16) float sm[];
-    rfx::pdl_prologue();
+    __shared__ __align__(8) uint64_t full[MAX_STAGES], empty[MAX_STAGES];
+    __shared__ volatile int gave_up;
     const int seq = blockIdx.x, h = blockIdx.y, c_first = blockIdx.z * cols;
-    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, nwarps = blockDim.x >> 5;
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    const int n_warps = cols / 16 * 4;  // the walking warps
     const int l4 = lane >> 2, j = lane & 3;
     const int VLD = cols + 4, buf_floats = 2 * CH * LDK + COEF + CH * VLD;
-    const int C = 2 * G * d + H * dv, kvh = h / (H / G), d4 = d / 4;
+    const int C = 2 * G * d + H * dv, kvh = h / (H / G);
+    const int grp = warp >> 2, quarter = warp & 3;
+    // partial sums: [parity][group][tile of D][quarter][lane] four floats
+    float4* red = reinterpret_cast<float4*>(sm + stages * buf_floats);
+    // everything a copy does not reach stays zero: channels beyond d, rows beyond the first chunks'
+    for (int e = threadIdx.x; e < stages * buf_floats; e += blockDim.x) sm[e] = 0.0f;
+    if (threadIdx.x == 0) {
+        for (int i = 0; i < stages; ++i) {
+            sm100::mbar_init(&full[i], 1);
+            sm100::mbar_init(&empty[i], n_warps);
+        }
+        sm100::fence_barrier_init();
+        gave_up = 0;
+    }
+    asm volatile("fence.proxy.async.shared::cta;" ::: "memory");
+    __syncthreads();
+    rfx::pdl_prologue();
     const int row0 = seq_row0[seq], row1 = seq_row0[seq + 1];
     const int n_chunks = (row1 - row0 + CH - 1) / CH;
-    const int cl = warp * 16, col = c_first + cl;
-    const bool live = col < dv;  // dv is a multiple of sixteen: a warp's columns all or none
-    float* Sg = state + (size_t)seq_slot[seq] * state_stride + state_off + ((size_t)h * dv + (live ? col : 0)) * d;
+    if (warp == n_warps) {
+        const int v_bytes = min(cols, dv - c_first) * 4;
+        int buf = 0, round = 0;  // chunk c is the round-th use of its buffer
+        for (int c = 0; c < n_chunks; ++c) {
+            const int first = row0 + c * CH, n = min(CH, row1 - first);
+            if (round > 0 && !gave_up && !sm100::mbar_wait(&empty[buf], (round - 1) & 1)) {
+                if (lane == 0) atomicExch(err, 41);
+                gave_up = 1;
+            }
+            __syncwarp();
+            if (gave_up) break;
+            float* base = sm + (size_t)buf * buf_floats;
+            if (lane == 0) sm100::mbar_expect_tx(&full[buf], n * (8 * d + v_bytes) + COEF * 4);
+            __syncwarp();
+            if (lane < n) {
+                const float* src = qkv + (size_t)(first + lane) * C;
+                bulk_load(base + lane * LDK, src + G * d + kvh * d, 4 * d, &full[buf]);
+                bulk_load(base + (CH + lane) * LDK, src + kvh * d, 4 * d, &full[buf]);
+                bulk_load(base + 2 * CH * LDK + COEF + lane * VLD, src + 2 * G * d + h * dv + c_first, v_bytes, &full[buf]);
+            }
+            if (lane == 31)
+                bulk_load(base + 2 * CH * LDK, coef + (chunk_place(row0, seq, c) * H + h) * COEF, COEF * 4, &full[buf]);
+            if (++buf == stages) {
+                buf = 0;
+                ++round;
+            }
+        }
+        return;
+    }
+    const int cl = grp * 16, col = c_first + cl;
+    const bool live = col < dv;  // dv is a multiple of sixteen: a group's columns all or none
+    const int ch0 = quarter * 8 * NT;  // the warp's first channel
+    float* Sg = state + (size_t)seq_slot[seq] * state_stride + state_off + ((size_t)h * dv + (live ? col : 0)) * d + ch0;
     float S[NT][4];
 #pragma unroll
     for (int s = 0; s < NT; ++s) {
         float2 x = make_float2(0.0f, 0.0f), y = x;
-        if (live && 8 * s < d) {
+        if (live && ch0 + 8 * s < d) {
             x = *reinterpret_cast<const float2*>(Sg + (size_t)l4 * d + 8 * s + 2 * j);
             y = *reinterpret_cast<const float2*>(Sg + (size_t)(l4 + 8) * d + 8 * s + 2 * j);
         }
         S[s][0] = x.x; S[s][1] = x.y; S[s][2] = y.x; S[s][3] = y.y;
     }
-    // everything a copy does not reach stays zero: channels beyond d, rows beyond the last
-    for (int e = threadIdx.x; e < 2 * buf_floats; e += blockDim.x) sm[e] = 0.0f;
-    __syncthreads();
-    const int v4 = min(cols, dv - c_first) / 4;
-    const int q_src = kvh * d, k_src = G * d + kvh * d, v_src = 2 * G * d + h * dv + c_first;
-    auto stage = [&](int c, int buf) {
-        float* base = sm + (size_t)buf * buf_floats;
-        const int first = row0 + c * CH, n = min(CH, row1 - first);
-        for (int r = warp; r < CH; r += nwarps) {
-            float *k = base + r * LDK, *q = k + CH * LDK, *v = base + 2 * CH * LDK + COEF + r * VLD;
-            if (r < n) {
-                const float* src = qkv + (size_t)(first + r) * C;
-                for (int e = lane; e < d4; e += 32) {
-                    attn::cp_async_16(k + 4 * e, src + k_src + 4 * e, true);
-                    attn::cp_async_16(q + 4 * e, src + q_src + 4 * e, true);
-                }
-                for (int e = lane; e < v4; e += 32) attn::cp_async_16(v + 4 * e, src + v_src + 4 * e, true);
-            } else {  // the last chunk's missing rows: this buffer held others
-                for (int e = lane; e < d; e += 32) k[e] = q[e] = 0.0f;
-                for (int e = lane; e < cols; e += 32) v[e] = 0.0f;
-            }
-        }
-        const float* cf = coef + (chunk_place(row0, seq, c) * H + h) * COEF;
-        for (int e = threadIdx.x; e < COEF / 4; e += blockDim.x)
-            attn::cp_async_16(base + 2 * CH * LDK + 4 * e, cf + 4 * e, true);
-        attn::cp_async_commit();
-    };
-    if (n_chunks > 0) stage(0, 0);
+    int buf = 0, round = 0;
     for (int c = 0; c < n_chunks; ++c) {
-        const int buf = c & 1;
-        if (c + 1 < n_chunks) {
-            stage(c + 1, buf ^ 1);
-            attn::cp_async_wait<1>();
-        } else {
-            attn::cp_async_wait<0>();
+        const int par = c & 1;  // of the partial sums' two places
+        if (!gave_up && !sm100::mbar_wait(&full[buf], round & 1)) {  // reported; the walk ends without waiting on
+            if (lane == 0) atomicExch(err, 42);
+            gave_up = 1;
         }
-        __syncthreads();
-        const float* ks = sm + (size_t)buf * buf_floats;
-        const float *cf = ks + 2 * CH * LDK, *vs = cf + COEF;
-        // K S0 and Q S0, transposed: [0], [1] the k rows 0..7 and 8..15, [2], [3] the q rows
+        const float* base = sm + (size_t)buf * buf_floats;
+        const float *ks = base + ch0, *cf = base + 2 * CH * LDK, *vs = cf + COEF;
+        // this quarter's K S0 and Q S0, transposed: [0], [1] the k rows 0..7 and 8..15, [2], [3] the q rows
         float D[4][4] = {};
 #pragma unroll
         for (int s = 0; s < NT; ++s) {
@@ -232,32 +265,41 @@ gated_delta_chunk_kernel(const float* __restrict__ qkv, const float* __restrict_
                 b[n] = *reinterpret_cast<const float2*>(ks + (8 * n + l4) * LDK + 8 * s + 2 * j);
             product3<4>(D, a, b);
         }
+        float4* mine = red + ((size_t)(par * (n_warps >> 2) + grp) * 4 * 4 + quarter) * 32 + lane;
+#pragma unroll
+        for (int n = 0; n < 4; ++n) mine[n * 4 * 32] = make_float4(D[n][0], D[n][1], D[n][2], D[n][3]);
+        asm volatile("bar.sync %0, 128;" ::"r"(1 + grp) : "memory");  // the group's four warps
+        const float4* all4 = red + (size_t)(par * (n_warps >> 2) + grp) * 4 * 4 * 32 + lane;
+        auto total = [&](int n, float (&t)[4]) {
+            const float4 p0 = all4[n * 128], p1 = all4[n * 128 + 32], p2 = all4[n * 128 + 64], p3 = all4[n * 128 + 96];
+            t[0] = (p0.x + p1.x) + (p2.x + p3.x);
+            t[1] = (p0.y + p1.y) + (p2.y + p3.y);
+            t[2] = (p0.z + p1.z) + (p2.z + p3.z);
+            t[3] = (p0.w + p1.w) + (p2.w + p3.w);
+        };
         // v - c * (K S0), then u = T of it; a tile holds rows 8 t + 2 j and + 1 of columns l4 and l4 + 8
-        float U[2][4] = {}, O[2][4];
+        float U[2][4] = {};
         float2 ci[2];
 #pragma unroll
         for (int t = 0; t < 2; ++t) {
             ci[t] = *reinterpret_cast<const float2*>(cf + 2 * CH * TLD + 8 * t + 2 * j);
             const float* v = vs + (8 * t + 2 * j) * VLD + cl + l4;
             float x[4];
-            x[0] = fmaf(-ci[t].x, D[t][0], v[0]);
-            x[1] = fmaf(-ci[t].y, D[t][1], v[VLD]);
-            x[2] = fmaf(-ci[t].x, D[t][2], v[8]);
-            x[3] = fmaf(-ci[t].y, D[t][3], v[VLD + 8]);
+            total(t, x);
+            x[0] = fmaf(-ci[t].x, x[0], v[0]);
+            x[1] = fmaf(-ci[t].y, x[1], v[VLD]);
+            x[2] = fmaf(-ci[t].x, x[2], v[8]);
+            x[3] = fmaf(-ci[t].y, x[3], v[VLD + 8]);
             const Left a = left_of(x);
             float2 b[2];
 #pragma unroll
             for (int n = 0; n < 2; ++n)
                 b[n] = *reinterpret_cast<const float2*>(cf + (8 * n + l4) * TLD + 8 * t + 2 * j);
-            product3<2>(U, a, b);  // T is lower triangular: of t = 1 the rows 0..7 get zeros
+            // T is lower triangular: rows 8..15 of its right side meet rows 8..15 alone
+            if (t == 0) product3<2>(U, a, b);
+            else product3<1>(*reinterpret_cast<float(*)[1][4]>(&U[1]), a, *reinterpret_cast<const float2(*)[1]>(&b[1]));
         }
-#pragma unroll
-        for (int t = 0; t < 2; ++t) {
-            O[t][0] = ci[t].x * D[2 + t][0];
-            O[t][1] = ci[t].y * D[2 + t][1];
-            O[t][2] = ci[t].x * D[2 + t][2];
-            O[t][3] = ci[t].y * D[2 + t][3];
-        }
+        // the memory's step: K^T (r_last * u)
         const float all = cf[2 * CH * TLD + 2 * CH];
 #pragma unroll
         for (int s = 0; s < NT; ++s)
@@ -265,50 +307,64 @@ gated_delta_chunk_kernel(const float* __restrict__ qkv, const float* __restrict_
             for (int i = 0; i < 4; ++i) S[s][i] *= all;
 #pragma unroll
         for (int t = 0; t < 2; ++t) {
-            {
+            const float2 rl = *reinterpret_cast<const float2*>(cf + 2 * CH * TLD + CH + 8 * t + 2 * j);
+            const float w[4] = {U[t][0] * rl.x, U[t][1] * rl.y, U[t][2] * rl.x, U[t][3] * rl.y};
+            const Left a = left_of(w);
+            const float* k = ks + (8 * t + 2 * j) * LDK + l4;
+            float2 b[NT];
+#pragma unroll
+            for (int s = 0; s < NT; ++s) b[s] = make_float2(k[8 * s], k[LDK + 8 * s]);
+            product3<NT>(S, a, b);
+        }
+        if (quarter == (c & 3)) {
+            float O[2][4];
+#pragma unroll
+            for (int t = 0; t < 2; ++t) {
+                total(2 + t, O[t]);
+                O[t][0] *= ci[t].x;
+                O[t][1] *= ci[t].y;
+                O[t][2] *= ci[t].x;
+                O[t][3] *= ci[t].y;
+            }
+#pragma unroll
+            for (int t = 0; t < 2; ++t) {
                 const Left a = left_of(U[t]);
                 float2 b[2];
 #pragma unroll
                 for (int n = 0; n < 2; ++n)
                     b[n] = *reinterpret_cast<const float2*>(cf + CH * TLD + (8 * n + l4) * TLD + 8 * t + 2 * j);
-                product3<2>(O, a, b);
+                if (t == 0) product3<2>(O, a, b);
+                else product3<1>(*reinterpret_cast<float(*)[1][4]>(&O[1]), a, *reinterpret_cast<const float2(*)[1]>(&b[1]));
             }
-            // the memory's step: K^T (r_last * u), four tiles of channels at a time
-            const float2 rl = *reinterpret_cast<const float2*>(cf + 2 * CH * TLD + CH + 8 * t + 2 * j);
-            const float w[4] = {U[t][0] * rl.x, U[t][1] * rl.y, U[t][2] * rl.x, U[t][3] * rl.y};
-            const Left a = left_of(w);
-            const float* k = ks + (8 * t + 2 * j) * LDK + l4;
+            if (live) {
+                const int left = row1 - row0 - c * CH;
+                const size_t ld = (size_t)H * dv;
+                float* o = out + (size_t)(row0 + c * CH) * ld + (size_t)h * dv + col + l4;
 #pragma unroll
-            for (int s = 0; s < NT; s += 4) {
-                float2 b[4];
-#pragma unroll
-                for (int n = 0; n < 4; ++n) b[n] = make_float2(k[8 * (s + n)], k[LDK + 8 * (s + n)]);
-                product3<4>(*reinterpret_cast<float(*)[4][4]>(&S[s]), a, b);
-            }
-        }
-        if (live) {
-            const int left = row1 - row0 - c * CH;
-            float* o = out + (size_t)(row0 + c * CH) * H * dv + (size_t)h * dv + col + l4;
-            const size_t ld = (size_t)H * dv;
-#pragma unroll
-            for (int t = 0; t < 2; ++t) {
-                const int r = 8 * t + 2 * j;
-                if (r < left) {
-                    o[r * ld] = O[t][0];
-                    o[r * ld + 8] = O[t][2];
-                }
-                if (r + 1 < left) {
-                    o[(r + 1) * ld] = O[t][1];
-                    o[(r + 1) * ld + 8] = O[t][3];
+                for (int t = 0; t < 2; ++t) {
+                    const int r = 8 * t + 2 * j;
+                    if (r < left) {
+                        o[r * ld] = O[t][0];
+                        o[r * ld + 8] = O[t][2];
+                    }
+                    if (r + 1 < left) {
+                        o[(r + 1) * ld] = O[t][1];
+                        o[(r + 1) * ld + 8] = O[t][3];
+                    }
                 }
             }
         }
-        __syncthreads();  // this buffer is copied into again two chunks on
+        __syncwarp();
+        if (lane == 0) sm100::mbar_arrive(&empty[buf]);  // this warp is done with the chunk
+        if (++buf == stages) {
+            buf = 0;
+            ++round;
+        }
     }
     if (!live) return;
 #pragma unroll
     for (int s = 0; s < NT; ++s)
-        if (8 * s < d) {
+        if (ch0 + 8 * s < d) {
             *reinterpret_cast<float2*>(Sg + (size_t)l4 * d + 8 * s + 2 * j) = make_float2(S[s][0], S[s][1]);
             *reinterpret_cast<float2*>(Sg + (size_t)(l4 + 8) * d + 8 * s + 2 * j) = make_float2(S[s][2], S[s][3]);
         }
@@ -317,21 +373,27 @@ gated_delta_chunk_kernel(const float* __restrict__ qkv, const float* __restrict_
 template <int NT>
 int launch_chunk(const float* qkv, const float* coef, float* state, long long state_stride, long long state_off,
                  const int* seq_slot, const int* seq_row0, int n_seq, float* out, int H, int G, int d, int dv,
-                 cudaStream_t s) {
-    // value columns a block owns, sixteen a warp; fewer while the blocks do not fill the SMs
+                 int* err, cudaStream_t s) {
+    // value columns a block owns, sixteen a group of four warps; fewer while the blocks do not fill the SMs
     int cols = 64;
     while (cols > 16 && (cols / 2 >= dv ||
                          (long long)n_seq * H * ((dv + cols - 1) / cols) < rfx::sm_count() * 3LL / 4))
         cols /= 2;
-    const size_t smem = (size_t)2 * (2 * CH * (8 * NT + 8) + COEF + CH * (cols + 4)) * sizeof(float);
+    const size_t stage = (size_t)(2 * CH * (32 * NT + 8) + COEF + CH * (cols + 4)) * sizeof(float);
+    const size_t red = (size_t)2 * (cols / 16) * 4 * 4 * 32 * sizeof(float4);
+    // one block an SM: as many chunks in flight as fit, up to four; more blocks: two chunks each
+    int stages = (long long)n_seq * H * ((dv + cols - 1) / cols) <= rfx::sm_count() ? MAX_STAGES : 2;
+    while (stages > 2 && stages * stage + red > 220 * 1024) --stages;
+    const size_t smem = stages * stage + red;
+    if (smem > 220 * 1024) return RFX_ERR_UNSUPPORTED;
     auto kernel = gated_delta_chunk_kernel<NT>;
     if (smem > 48 * 1024) {
         cudaError_t e = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
         if (e != cudaSuccess) return (int)e;
     }
     dim3 grid(n_seq, H, (dv + cols - 1) / cols);
-    RFX_LAUNCH(kernel, grid, cols * 2, smem, s, qkv, coef, state, state_stride, state_off, seq_slot, seq_row0, out, H,
-               G, d, dv, cols);
+    RFX_LAUNCH(kernel, grid, cols / 16 * 128 + 32, smem, s, qkv, coef, state, state_stride, state_off, seq_slot,
+               seq_row0, out, H, G, d, dv, cols, stages, err);
     return 0;
 }
 
@@ -357,10 +419,11 @@ extern "C" int rfx_gated_delta_chunk_prep(const float* qkv, const float* gates, 
 }
 
 // The recurrence over the step's rows, chunk by chunk.  d a multiple of 8 up to 256, dv of 16;
-// the running state as rfx_gated_delta_scan keeps it.
+// the running state as rfx_gated_delta_scan keeps it.  `err`: a device word that receives a
+// non-zero code if a bounded wait ran out.
 extern "C" int rfx_gated_delta_chunk(const float* qkv, const float* coef, float* state, long long state_stride,
                                      long long state_off, const int* seq_slot, const int* seq_row0, int n_seq,
-                                     float* out, int H, int G, int d, int dv, void* stream) {
+                                     float* out, int H, int G, int d, int dv, int* err, void* stream) {
     if (n_seq <= 0) return 0;
     if (H <= 0 || G <= 0 || H % G || d <= 0 || dv <= 0) return RFX_ERR_BAD_ARG;
     if ((state_stride | state_off) & 3 || (reinterpret_cast<uintptr_t>(state) & 15)) return RFX_ERR_BAD_ARG;
@@ -368,13 +431,14 @@ extern "C" int rfx_gated_delta_chunk(const float* qkv, const float* coef, float*
         ((reinterpret_cast<uintptr_t>(qkv) | reinterpret_cast<uintptr_t>(coef)) & 15))
         return RFX_ERR_UNSUPPORTED;
     cudaStream_t s = (cudaStream_t)stream;
-#define RFX_CHUNK(N)                                                                                               \
-    return launch_chunk<N>(qkv, coef, state, state_stride, state_off, seq_slot, seq_row0, n_seq, out, H, G, d, dv, s)
-    if (d <= 32) RFX_CHUNK(4);
-    if (d <= 64) RFX_CHUNK(8);
-    if (d <= 96) RFX_CHUNK(12);
-    if (d <= 128) RFX_CHUNK(16);
-    if (d <= 192) RFX_CHUNK(24);
-    RFX_CHUNK(32);
+#define RFX_CHUNK(N)                                                                                              \
+    return launch_chunk<N>(qkv, coef, state, state_stride, state_off, seq_slot, seq_row0, n_seq, out, H, G, d, dv, \
+                           err, s)
+    if (d <= 32) RFX_CHUNK(1);
+    if (d <= 64) RFX_CHUNK(2);
+    if (d <= 96) RFX_CHUNK(3);
+    if (d <= 128) RFX_CHUNK(4);
+    if (d <= 192) RFX_CHUNK(6);
+    RFX_CHUNK(8);
 #undef RFX_CHUNK
 }

@@ -1684,7 +1684,7 @@ def gated_delta_scan(qkv: torch.Tensor, gates: torch.Tensor, state: torch.Tensor
         st = native.lib().rfx_gated_delta_chunk(
             qkv.data_ptr(), coef.data_ptr(), _chk(state, "state", torch.float32), state.stride(0), int(state_off),
             _chk(batch.seq_slot, "seq_slot", torch.int32), row0, S, out.data_ptr(), heads, kv_heads, dim, vdim,
-            _stream())
+            device_error_word(qkv.device).data_ptr(), _stream())
         native.check(st, f"gated_delta_chunk (heads={heads}, dim={dim}, vdim={vdim})")
         return out
     st = native.lib().rfx_gated_delta_scan(

@@ -127,7 +127,7 @@ _SIGNATURES = {
     "rfx_gated_delta_chunk_prep": [c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_int, c_int,
                                    c_void_p],
     "rfx_gated_delta_chunk": [c_void_p, c_void_p, c_void_p, c_longlong, c_longlong, c_void_p, c_void_p, c_int, c_void_p,
-                               c_int, c_int, c_int, c_int, c_void_p],
+                              c_int, c_int, c_int, c_int, c_void_p, c_void_p],
     "rfx_rot_qkv_post": [c_void_p, c_int, c_int, c_void_p, c_void_p, c_int, c_int, c_float, c_void_p, c_void_p,
                          c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_int, c_int,
                          c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p],
