@@ -36,14 +36,21 @@ __device__ __forceinline__ float softplus_f(float v) { return fmaxf(v, 0.0f) + l
 
 constexpr int PREP_THREADS = 256;
 
-template <bool BY4>
-__global__ void __launch_bounds__(PREP_THREADS)
+// y / (1 + e^-y) with the hardware's exponential and reciprocal (about 2^-21 off)
+__device__ __forceinline__ float silu_fast(float y) { return __fdividef(y, 1.0f + __expf(-y)); }
+
+// NV: a head's elements in 128s, four a lane (up to 512), 0: heads whose size is no multiple of four.
+// TAPS: the filters' length where it is known here (all taps' loads go out together), 0: `taps_any`.
+// `fast`: the activation with the hardware's approximations (rows of the bfloat16 path).
+template <int NV, int TAPS>
+__global__ void __launch_bounds__(PREP_THREADS, NV <= 1 ? 5 : 2)
 gated_delta_prep_kernel(const float* __restrict__ proj, int ld, int b_off, int a_off,
-                        const float* __restrict__ filters, int taps, float* state, long long slot_stride,
+                        const float* __restrict__ filters, int taps_any, float* state, long long slot_stride,
                         const int* __restrict__ row_slot, const float* __restrict__ dt_bias,
                         const float* __restrict__ A, float unit_eps, float q_scale, float* __restrict__ out,
-                        float* __restrict__ gates, int H, int G, int d, int dv, int update) {
+                        float* __restrict__ gates, int H, int G, int d, int dv, int update, int fast) {
     pdl_prologue();
+    const int taps = TAPS ? TAPS : taps_any;
     const int r = blockIdx.x;
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const int unit = blockIdx.y * (PREP_THREADS / 32) + warp;
@@ -64,15 +71,15 @@ gated_delta_prep_kernel(const float* __restrict__ proj, int ld, int b_off, int a
     const int T = taps - 1;
     float* orow = out + (size_t)r * C + c0;
     float ss = 0.0f;
-    if constexpr (BY4) {
-        constexpr int NV = 4;  // heads up to 512 wide
+    if constexpr (NV > 0) {
         float4 y[NV];
 #pragma unroll
         for (int i = 0; i < NV; ++i) {
             const int e = 4 * (lane + 32 * i);
             if (e < width) {
                 float4 t = conv4_at(proj, ld, 0, c0 + e, nullptr, filters, taps, tail, C, r, before);
-                t.x = silu_of(t.x); t.y = silu_of(t.y); t.z = silu_of(t.z); t.w = silu_of(t.w);
+                if (fast) { t.x = silu_fast(t.x); t.y = silu_fast(t.y); t.z = silu_fast(t.z); t.w = silu_fast(t.w); }
+                else { t.x = silu_of(t.x); t.y = silu_of(t.y); t.z = silu_of(t.z); t.w = silu_of(t.w); }
                 ss = fmaf(t.x, t.x, fmaf(t.y, t.y, fmaf(t.z, t.z, fmaf(t.w, t.w, ss))));
                 y[i] = t;
                 if (update && T > 0) {
@@ -304,11 +311,13 @@ int launch_scan(const float* qkv, const float* gates, float* state, long long st
 // and the decays' pre-activations at `b_off` and `a_off` (H each).  `filters` transposed,
 // [taps][2 G d + H dv]; `state` the slots' last taps - 1 inputs (the vector's start).  Out:
 // `out` float32 [R, 2 G d + H dv] and `gates` float32 [R, 2 H] (decays, write rates).
-// `update` 1: every sequence has exactly one of the R rows, and its last inputs move on.
+// `update` 1: every sequence has exactly one of the R rows, and its last inputs move on.  `fast`:
+// the filters' activation with the hardware's exponential.
 extern "C" int rfx_gated_delta_prep(const float* proj, int ld, int b_off, int a_off, const float* filters, int taps,
                                     float* state, long long slot_stride, const int* row_slot,
                                     const float* dt_bias, const float* A, float unit_eps, float q_scale, float* out,
-                                    float* gates, int R, int H, int G, int d, int dv, int update, void* stream) {
+                                    float* gates, int R, int H, int G, int d, int dv, int update, int fast,
+                                    void* stream) {
     if (R <= 0) return 0;
     if (H <= 0 || G <= 0 || H % G || d <= 0 || dv <= 0 || taps < 1 || taps > MAX_TAPS) return RFX_ERR_BAD_ARG;
     if (taps > 1 && !state) return RFX_ERR_BAD_ARG;
@@ -319,12 +328,16 @@ extern "C" int rfx_gated_delta_prep(const float* proj, int ld, int b_off, int a_
                      ((reinterpret_cast<uintptr_t>(proj) | reinterpret_cast<uintptr_t>(filters) |
                        reinterpret_cast<uintptr_t>(state) | reinterpret_cast<uintptr_t>(out)) & 15) == 0;
     cudaStream_t s = (cudaStream_t)stream;
-    if (by4)
-        RFX_LAUNCH(gated_delta_prep_kernel<true>, grid, PREP_THREADS, 0, s, proj, ld, b_off, a_off, filters, taps,
-                   state, slot_stride, row_slot, dt_bias, A, unit_eps, q_scale, out, gates, H, G, d, dv, update);
-    else
-        RFX_LAUNCH(gated_delta_prep_kernel<false>, grid, PREP_THREADS, 0, s, proj, ld, b_off, a_off, filters, taps,
-                   state, slot_stride, row_slot, dt_bias, A, unit_eps, q_scale, out, gates, H, G, d, dv, update);
+#define RFX_PREP(N, T)                                                                                              \
+    RFX_LAUNCH((gated_delta_prep_kernel<N, T>), grid, PREP_THREADS, 0, s, proj, ld, b_off, a_off, filters, taps, state, \
+               slot_stride, row_slot, dt_bias, A, unit_eps, q_scale, out, gates, H, G, d, dv, update, fast)
+    if (!by4) RFX_PREP(0, 0);
+    else if (d > 128 || dv > 128) RFX_PREP(4, 0);
+    else if (taps == 2) RFX_PREP(1, 2);
+    else if (taps == 3) RFX_PREP(1, 3);
+    else if (taps == 4) RFX_PREP(1, 4);
+    else RFX_PREP(1, 0);
+#undef RFX_PREP
     return 0;
 }
 

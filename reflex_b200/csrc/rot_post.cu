@@ -66,7 +66,8 @@ struct QkvPost {
     int nq, nkv, d, dv, pad, writes_cache;
 };
 
-template <typename TI, typename TO, bool BY4>
+// NV: a head's elements in 128s, four a lane (up to 512), 0: sizes that are no multiples of four
+template <typename TI, typename TO, int NV>
 __global__ void __launch_bounds__(RP_THREADS)
 rot_qkv_post_kernel(const TI* __restrict__ proj, int ldp, QkvPost a, const int* __restrict__ row_pos,
                     const int* __restrict__ row_slot, TO* __restrict__ q_out, TO* __restrict__ k_pages,
@@ -92,8 +93,7 @@ rot_qkv_post_kernel(const TI* __restrict__ proj, int ldp, QkvPost a, const int* 
         else dst = v_pages + kv_offset(cache, slot, pos, vh);
         const float lam = a.lambda ? *a.lambda : 0.0f;
         const size_t vrow = ((size_t)r * a.nkv + vh) * a.dv;
-        if constexpr (BY4) {
-            constexpr int NV = 4;  // heads up to 512 wide
+        if constexpr (NV > 0) {
             float4 y[NV];
             float ss = 0.0f;
 #pragma unroll
@@ -251,20 +251,21 @@ extern "C" int rfx_rot_qkv_post(const void* proj, int in_dt, int ld, const float
                      aligned(v_pages, out_al);
     dim3 grid(R, rows_blocks(R, nq + 2 * nkv));
     const size_t smem = (size_t)(rot_dims > 0 ? rot_dims : 1) * sizeof(float);
-#define RFX_GO(TI, TO)                                                                                            \
-    do {                                                                                                          \
-        if (by4)                                                                                                  \
-            RFX_LAUNCH((rot_qkv_post_kernel<TI, TO, true>), grid, RP_THREADS, smem, s, (const TI*)proj, ld, a,    \
-                       row_pos, row_slot, (TO*)q_out, (TO*)k_pages, (TO*)v_pages, cache);                         \
-        else                                                                                                      \
-            RFX_LAUNCH((rot_qkv_post_kernel<TI, TO, false>), grid, RP_THREADS, smem, s, (const TI*)proj, ld, a,   \
-                       row_pos, row_slot, (TO*)q_out, (TO*)k_pages, (TO*)v_pages, cache);                         \
+#define RFX_N(TI, TO, N)                                                                                          \
+    RFX_LAUNCH((rot_qkv_post_kernel<TI, TO, N>), grid, RP_THREADS, smem, s, (const TI*)proj, ld, a, row_pos,      \
+               row_slot, (TO*)q_out, (TO*)k_pages, (TO*)v_pages, cache)
+#define RFX_GO(TI, TO)                   \
+    do {                                 \
+        if (!by4) RFX_N(TI, TO, 0);      \
+        else if (pad <= 128) RFX_N(TI, TO, 1); \
+        else RFX_N(TI, TO, 4);           \
     } while (0)
     if (in_dt == RFX_DT_F32 && out_dt == RFX_DT_F32) RFX_GO(float, float);
     else if (in_dt == RFX_DT_F32 && out_dt == RFX_DT_BF16) RFX_GO(float, __nv_bfloat16);
     else if (in_dt == RFX_DT_BF16 && out_dt == RFX_DT_BF16) RFX_GO(__nv_bfloat16, __nv_bfloat16);
     else return RFX_ERR_BAD_ARG;
 #undef RFX_GO
+#undef RFX_N
     return 0;
 }
 

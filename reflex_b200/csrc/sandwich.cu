@@ -118,6 +118,12 @@ __device__ __forceinline__ float gate_of(float t, int act) {
     const float s = 1.0f / (1.0f + exact_expf(-t));
     return act ? t * s : s;
 }
+// the same for a result that is rounded to bfloat16: the hardware's exponential and division
+template <typename TO>
+__device__ __forceinline__ float gate_for(float t, int act) {
+    if constexpr (sizeof(TO) == 2) return __fdividef(act ? t : 1.0f, 1.0f + __expf(-t));
+    else return gate_of(t, act);
+}
 
 // One block a (row, part), 16 bytes an access: parts of many elements (a norm in a few equal
 // parts of a wide row), where a warp a part would leave a row to a warp or two.
@@ -149,6 +155,48 @@ group_norm_gate_wide_kernel(const float* __restrict__ x, const float* __restrict
             o.w *= gate_of(zp[3], act);
         }
         store4(out + base + 4 * (size_t)c, o);
+    }
+}
+
+// Parts of up to 512 elements, a multiple of four: a warp a part, the part in registers between
+// its sum of squares and the outputs, 16 bytes an access, the gate's loads beside the row's.
+template <typename TO>
+__global__ void __launch_bounds__(256)
+group_norm_gate4_kernel(const float* __restrict__ x, const float* __restrict__ w, float eps,
+                        const float* __restrict__ z, int ldz, int zcol, int act, int shared, TO* __restrict__ out,
+                        long long parts, int groups, int gs) {
+    pdl_prologue();
+    const long long part = (long long)blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
+    if (part >= parts) return;
+    const int lane = threadIdx.x & 31, g = (int)(part % groups);
+    const size_t r = (size_t)(part / groups), base = (size_t)part * gs;
+    constexpr int V = 4;
+    float4 v[V], t[V];
+    float ss = 0.0f;
+#pragma unroll
+    for (int i = 0; i < V; ++i) {
+        const int c = 4 * (lane + 32 * i);
+        if (c < gs) {
+            v[i] = *reinterpret_cast<const float4*>(x + base + c);
+            if (z) t[i] = *reinterpret_cast<const float4*>(z + r * ldz + zcol + (size_t)g * gs + c);
+            ss = fmaf(v[i].x, v[i].x, fmaf(v[i].y, v[i].y, fmaf(v[i].z, v[i].z, fmaf(v[i].w, v[i].w, ss))));
+        }
+    }
+    const float rs = 1.0f / sqrtf(warp_sum(ss) / (float)gs + eps);
+#pragma unroll
+    for (int i = 0; i < V; ++i) {
+        const int c = 4 * (lane + 32 * i);
+        if (c < gs) {
+            const float4 ww = *reinterpret_cast<const float4*>(w + (shared ? 0 : (size_t)g * gs) + c);
+            float4 o = make_float4((v[i].x * rs) * ww.x, (v[i].y * rs) * ww.y, (v[i].z * rs) * ww.z, (v[i].w * rs) * ww.w);
+            if (z) {
+                o.x *= gate_for<TO>(t[i].x, act);
+                o.y *= gate_for<TO>(t[i].y, act);
+                o.z *= gate_for<TO>(t[i].z, act);
+                o.w *= gate_for<TO>(t[i].w, act);
+            }
+            store4(out + base + c, o);
+        }
     }
 }
 
@@ -284,6 +332,19 @@ extern "C" int rfx_group_norm_gate(const float* x, const float* w, float eps, co
         else if (out_dt == RFX_DT_BF16)
             RFX_LAUNCH(group_norm_gate_wide_kernel<__nv_bfloat16>, grid, 256, 0, s, x, w, eps, z, ldz, zcol, act, shared,
                        (__nv_bfloat16*)out, C, gs);
+        else return RFX_ERR_BAD_ARG;
+        return 0;
+    }
+    const long long parts = (long long)R * groups;
+    if (gs % 4 == 0 && gs <= 512 && al && (!z || (ldz % 4 == 0 && zcol % 4 == 0 && (reinterpret_cast<uintptr_t>(z) & 15) == 0)) &&
+        (parts + 7) / 8 <= 2147483647LL) {
+        const int blocks = (int)((parts + 7) / 8);
+        if (out_dt == RFX_DT_F32)
+            RFX_LAUNCH(group_norm_gate4_kernel<float>, blocks, 256, 0, s, x, w, eps, z, ldz, zcol, act, shared,
+                       (float*)out, parts, groups, gs);
+        else if (out_dt == RFX_DT_BF16)
+            RFX_LAUNCH(group_norm_gate4_kernel<__nv_bfloat16>, blocks, 256, 0, s, x, w, eps, z, ldz, zcol, act, shared,
+                       (__nv_bfloat16*)out, parts, groups, gs);
         else return RFX_ERR_BAD_ARG;
         return 0;
     }

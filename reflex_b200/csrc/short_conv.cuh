@@ -14,6 +14,7 @@ constexpr int MAX_TAPS = 16;
 __device__ __forceinline__ int rows_before(const int* __restrict__ row_slot, int r, int cap) {
     const int slot = row_slot[r];
     int t = cap;  // the nearest row back that is not this sequence's ends the count (no early exit: no chain)
+#pragma unroll
     for (int j = cap - 1; j >= 0; --j) {
         const bool same = r - j - 1 >= 0 && row_slot[r - j - 1] == slot;
         if (!same) t = j;
@@ -47,15 +48,13 @@ __device__ __forceinline__ float4 conv4_at(const float* __restrict__ proj, int l
     const int T = taps - 1;
     const float4 b = bias ? *reinterpret_cast<const float4*>(bias + c) : make_float4(0.0f, 0.0f, 0.0f, 0.0f);
     float4 y = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+#pragma unroll
     for (int j = 0; j < taps; ++j) {
         const int back = T - j;
-        float4 u;
-        if (back <= before) {
-            u = *reinterpret_cast<const float4*>(proj + (size_t)(r - back) * ld + col0 + c);
-            u.x += b.x; u.y += b.y; u.z += b.z; u.w += b.w;
-        } else {
-            u = *reinterpret_cast<const float4*>(state_slot + (size_t)(T + before - back) * C + c);
-        }
+        const bool here = back <= before;  // one load from either place: no branch between the taps' loads
+        float4 u = *reinterpret_cast<const float4*>(here ? proj + (size_t)(r - back) * ld + col0 + c
+                                                         : state_slot + (size_t)(T + before - back) * C + c);
+        if (here) { u.x += b.x; u.y += b.y; u.z += b.z; u.w += b.w; }
         const float4 f = *reinterpret_cast<const float4*>(w + (size_t)j * C + c);
         y.x = fmaf(f.x, u.x, y.x);
         y.y = fmaf(f.y, u.y, y.y);

@@ -1631,14 +1631,15 @@ def delta_rule(proj: torch.Tensor, r_off: int, k_off: int, v_off: int, a_off: in
 
 def gated_delta_prep(proj: torch.Tensor, b_off: int, a_off: int, filters_t: torch.Tensor, state: torch.Tensor, batch,
                      dt_bias: torch.Tensor, A: torch.Tensor, unit_eps: float, q_scale: float, heads: int,
-                     kv_heads: int, dim: int, vdim: int, update_state: bool = False):
+                     kv_heads: int, dim: int, vdim: int, update_state: bool = False, exact: bool = True):
     """The rows of a stacked product [q | k | v | ..] (float32) through their short
     convolutions (`filters_t` float32 [taps, channels]) and silu, q and k made unit
     vectors per head (q also times `q_scale`): float32 [R, channels]; and from the
     columns at `b_off` and `a_off` the write rates sigmoid(b) and the decays exp(A
     softplus(a + dt_bias)): float32 [R, 2 heads], decays first.  `state` holds each
     slot's last inputs at its vector's start; `update_state`: one row a sequence,
-    and the launch moves them on."""
+    and the launch moves them on.  Without `exact` the filters' silu takes the
+    hardware's exponential."""
     if update_state and proj.shape[0] != batch.seq_slot.numel():
         raise InvalidInput("gated_delta_prep: update_state is for steps of one row a sequence")
     R, ld = proj.shape
@@ -1651,7 +1652,7 @@ def gated_delta_prep(proj: torch.Tensor, b_off: int, a_off: int, filters_t: torc
         _chk(proj, "proj", torch.float32), ld, int(b_off), int(a_off), _chk(filters_t, "filters_t", torch.float32),
         int(taps), _chk(state, "state", torch.float32), state.stride(0), _chk(batch.row_slot, "row_slot", torch.int32),
         _chk(dt_bias, "dt_bias", torch.float32), _chk(A, "A", torch.float32), float(unit_eps), float(q_scale),
-        out.data_ptr(), gates.data_ptr(), R, heads, kv_heads, dim, vdim, 1 if update_state else 0, _stream())
+        out.data_ptr(), gates.data_ptr(), R, heads, kv_heads, dim, vdim, 1 if update_state else 0, 0 if exact else 1, _stream())
     native.check(st, f"gated_delta_prep (heads={heads}, dim={dim}, vdim={vdim}, taps={taps})")
     return out, gates
 

@@ -121,7 +121,7 @@ _SIGNATURES = {
     "rfx_gemm_bf16_tc_geglu": [c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p],
     "rfx_gated_delta_prep": [c_void_p, c_int, c_int, c_int, c_void_p, c_int, c_void_p, c_longlong, c_void_p, c_void_p,
                              c_void_p, c_float, c_float, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int,
-                             c_void_p],
+                             c_int, c_void_p],
     "rfx_gated_delta_scan": [c_void_p, c_void_p, c_void_p, c_longlong, c_longlong, c_void_p, c_void_p, c_int, c_void_p,
                              c_int, c_int, c_int, c_int, c_int, c_void_p],
     "rfx_gated_delta_chunk_prep": [c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_int, c_int,

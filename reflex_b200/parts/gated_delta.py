@@ -97,7 +97,8 @@ class GatedDelta:
         single = proj.shape[0] == batch.seq_slot.numel()  # a row a sequence: the filters' launch moves their state on
         qkv, gates = ops.gated_delta_prep(
             proj, self.b_col, self.a_col, self.filters, state, batch, self.dt_bias, self.A, self.unit_eps,
-            self.spec.scale, self.heads, self.kv_heads, self.dim, self.vdim, update_state=single)
+            self.spec.scale, self.heads, self.kv_heads, self.dim, self.vdim, update_state=single,
+            exact=self.dtype == torch.float32)
         if not single:
             ops.conv_state_update(proj, 0, self.channels, None, self.taps, state, batch)
         ops.prof_mark("conv_post")
