@@ -182,13 +182,17 @@ class StateGroup:
         (src/model/mod.rs:1026-1030)."""
         if self.data is None:
             return None
-        idx = torch.tensor(list(slots), dtype=torch.int64, device=self.data.device)
-        return idx, self.data.index_select(1, idx)
+        slots = [int(s) for s in slots]
+        if self.data.is_cuda and self.data.element_size() == 4:
+            from ..ops import state_rows
+
+            return slots, state_rows(self.data, slots)
+        return slots, self.data.index_select(1, torch.tensor(slots, dtype=torch.int64, device=self.data.device))
 
     def restore(self, saved) -> None:
         if saved is not None:
-            idx, data = saved
-            self.data.index_copy_(1, idx, data)
+            slots, data = saved
+            self.data.index_copy_(1, torch.tensor(slots, dtype=torch.int64, device=self.data.device), data)
 
 
 class Cache:

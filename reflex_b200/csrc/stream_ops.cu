@@ -11,6 +11,7 @@
 //  * rfx_stream_concat: out[r] = [x[r] (+ delta[r]) | x0[r]], cast, the input of
 //    a product that mixes the stream with the embedding output.
 //  * rfx_logit_finish: z <- z * scale, then cap * tanh(z / cap) when cap > 0.
+//  * rfx_state_rows: the rows of chosen slots of a state group, copied aside.
 #include "common.cuh"
 
 namespace {
@@ -330,5 +331,62 @@ extern "C" int rfx_sigmoid_gate_mul(void* a, int a_dt, const void* z, int z_dt, 
                    (const __nv_bfloat16*)z, ldz, col, H);
     else
         return RFX_ERR_BAD_ARG;
+    return 0;
+}
+
+// ---- a state group's rows copied aside ------------------------------------------
+namespace {
+
+struct SlotList {
+    int slot[64];
+};
+
+// out[e][i] = data[e][slots[i]], rows of `n` elements of type T
+template <typename T>
+__global__ void __launch_bounds__(256)
+state_rows_kernel(const T* __restrict__ data, T* __restrict__ out, SlotList slots, long long n, long long entry_in,
+                  long long entry_out) {
+    pdl_prologue();
+    const T* src = data + blockIdx.z * entry_in + (long long)slots.slot[blockIdx.y] * n;
+    T* dst = out + blockIdx.z * entry_out + blockIdx.y * n;
+    const long long step = (long long)gridDim.x * blockDim.x;
+    long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x;
+    for (; i + 3 * step < n; i += 4 * step) {  // four loads in flight
+        const T a = src[i], b = src[i + step], c = src[i + 2 * step], d = src[i + 3 * step];
+        dst[i] = a;
+        dst[i + step] = b;
+        dst[i + 2 * step] = c;
+        dst[i + 3 * step] = d;
+    }
+    for (; i < n; i += step) dst[i] = src[i];
+}
+
+}  // namespace
+
+// data [entries][slots][words] 4-byte words, out [entries][n_slots][words]: the rows of the listed
+// slots (the list is on the host and travels with the launch).
+extern "C" int rfx_state_rows(const void* data, void* out, const int* slot_list, int n_slots, long long words,
+                              int entries, int slots, void* stream) {
+    if (n_slots <= 0 || words <= 0 || entries <= 0) return 0;
+    if (entries > 65535) return RFX_ERR_UNSUPPORTED;
+    for (int i = 0; i < n_slots; ++i)
+        if (slot_list[i] < 0 || slot_list[i] >= slots) return RFX_ERR_BAD_ARG;
+    const bool by4 = words % 4 == 0 && ((reinterpret_cast<uintptr_t>(data) | reinterpret_cast<uintptr_t>(out)) & 15) == 0;
+    const long long n = by4 ? words / 4 : words;
+    for (int at = 0; at < n_slots; at += 64) {
+        SlotList l{};
+        const int m = n_slots - at < 64 ? n_slots - at : 64;
+        for (int i = 0; i < m; ++i) l.slot[i] = slot_list[at + i];
+        long long gx = (n + 1023) / 1024, cap = 8LL * sm_count() / ((long long)m * entries) + 1;
+        if (gx > cap) gx = cap;
+        dim3 grid((unsigned)gx, m, entries);
+        const long long entry_in = (long long)slots * n, entry_out = (long long)n_slots * n;
+        if (by4)
+            RFX_LAUNCH(state_rows_kernel<uint4>, grid, 256, 0, (cudaStream_t)stream, (const uint4*)data,
+                       (uint4*)out + (size_t)at * n, l, n, entry_in, entry_out);
+        else
+            RFX_LAUNCH(state_rows_kernel<uint32_t>, grid, 256, 0, (cudaStream_t)stream, (const uint32_t*)data,
+                       (uint32_t*)out + (size_t)at * n, l, n, entry_in, entry_out);
+    }
     return 0;
 }

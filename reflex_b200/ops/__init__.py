@@ -1861,6 +1861,23 @@ LATENT_EXPAND_MIN_ROWS = _env_int("REFLEX_B200_LATENT_EXPAND_MIN_ROWS", 65, 2, 1
 LATENT_EXPAND_MAX_BYTES = 2 << 30
 
 
+def state_rows(data: torch.Tensor, slots) -> torch.Tensor:
+    """The rows of the listed slots (host integers) of `data` [entries, slots, *shape],
+    4-byte elements: a copy [entries, len(slots), *shape], one launch that waits for
+    nothing on the host."""
+    import ctypes
+
+    n = len(slots)
+    out = torch.empty((data.shape[0], n) + tuple(data.shape[2:]), dtype=data.dtype, device=data.device)
+    if data.element_size() != 4:
+        raise InvalidInput("state_rows: 4-byte elements only")
+    words = data[0, 0].numel()
+    st = native.lib().rfx_state_rows(_chk(data, "data"), out.data_ptr(), (ctypes.c_int * n)(*[int(s) for s in slots]), n,
+                                     words, data.shape[0], data.shape[1], _stream())
+    native.check(st, "state_rows")
+    return out
+
+
 # ------------------------------------------------------------------ sampling
 def argmax(logits: torch.Tensor, out: Optional[torch.Tensor] = None,
            scratch: Optional[torch.Tensor] = None) -> torch.Tensor:

@@ -176,6 +176,7 @@ _SIGNATURES = {
     "rfx_row_gate_add": [c_void_p, c_void_p, c_int, c_void_p, c_int, c_int, c_void_p, c_int, c_int, c_void_p],
     "rfx_stream_concat": [c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_void_p],
     "rfx_logit_finish": [c_void_p, c_longlong, c_float, c_float, c_void_p],
+    "rfx_state_rows": [c_void_p, c_void_p, c_void_p, c_int, c_longlong, c_int, c_int, c_void_p],
     "rfx_wait_probe": [c_longlong, c_void_p, c_void_p],
     "rfx_argmax": [c_void_p, c_longlong, c_int, c_int, c_void_p, c_void_p, c_void_p],
     "rfx_sample": [c_void_p, c_longlong, c_int, c_int, c_void_p, c_void_p, c_void_p, c_void_p,

@@ -680,3 +680,24 @@ def test_greedy_generation_through_the_entry_point(dtype):
 def test_decode_steps_are_captured_into_graphs(name):
     eng = make_engine(name, "bfloat16")
     assert eng.model.capturable and eng.use_graphs
+
+
+@pytest.mark.parametrize("shape,dtype", [((3,), torch.float32), ((8, 5), torch.float32), ((4096,), torch.float32), ((1,), torch.int32),
+                                         ((20000,), torch.float32)])
+@pytest.mark.parametrize("n", [1, 3, 70])
+def test_the_state_of_chosen_slots_is_copied_aside_and_put_back(shape, dtype, n):
+    from reflex_b200.cache.specs import StateSpec
+    from reflex_b200.cache.store import StateGroup
+
+    g = torch.Generator().manual_seed(n)
+    grp = StateGroup(StateSpec(shape, str(dtype).split(".")[1]), [0, 1, 2], 80, torch.device(DEV))
+    grp.data.copy_(torch.randint(-1000, 1000, tuple(grp.data.shape), generator=g).to(dtype))
+    slots = torch.randperm(80, generator=g)[:n].tolist()
+    before = grp.data.clone()
+    saved = grp.snapshot(slots)
+    assert torch.equal(saved[1], before[:, slots])
+    grp.data.add_(5)
+    grp.restore(saved)
+    assert torch.equal(grp.data[:, slots], before[:, slots])
+    others = [s for s in range(80) if s not in slots]
+    assert torch.equal(grp.data[:, others], before[:, others] + 5)
