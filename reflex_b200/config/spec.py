@@ -36,7 +36,9 @@ class NormSpec:
 class PositionSpec:
     """A position encoding applied to query and key head vectors."""
 
-    kind: str  # "rope_neox"; "rope_linear" (params: factor); "rope_scaled" (params: factor, low, high, original)
+    # "rope_neox"; "rope_linear" (params: factor); "rope_scaled" (params: factor, low, high, original);
+    # "rope_yarn" (params: factor, original, fast, slow); all: pairing ("half", "consecutive")
+    kind: str
     head_dim: int
     rotary_dim: int
     theta: float
@@ -61,10 +63,10 @@ class MixerSpec:
     position: Optional[PositionSpec] = None
     names: Tuple[Tuple[str, str], ...] = ()
     # what only some kinds have, by name: "latent_attention" reads q_rank, kv_rank,
-    # eps and sink; "mlstm" reads gate_cap and eps; "conv_attention" reads kv taps,
+    # rot_dim, eps, sink and gate; "mlstm" reads gate_cap and eps; "conv_attention" reads kv taps,
     # temp_coef, temp_every, sink and distance_slopes; "rglru" reads width, blocks,
     # taps and decay_scale; "pair" reads left and right (two `MixerSpec`s) and eps;
-    # "gqa_attention" reads values_are_keys, output_gate and keep_first; "selective_scan"
+    # "gqa_attention" reads values_are_keys, output_gate, head_gate, reads_cache and keep_first; "selective_scan"
     # reads inner, state, dt_rank and taps; "capped_attention" reads bias, unit_eps, softcap and
     # value_mix; "gated_delta" reads taps, unit_eps and eps
     params: Tuple[Tuple[str, Any], ...] = ()
@@ -82,7 +84,7 @@ class MixerSpec:
 @dataclass(frozen=True)
 class FeedForwardSpec:
     kind: str  # "swiglu"; "geglu"; "relu2"; "glu_clamped" (params: alpha, limit); "moe" (params: experts, top, activation,
-    # router_bias, scores, weight_input, alpha, limit, shared_ff, shared_limit)
+    # router_bias, scores, score_scale, groups, weight_input, alpha, limit, shared_ff, shared_limit)
     hidden_size: int
     intermediate_size: int
     names: Tuple[Tuple[str, str], ...] = ()

@@ -109,13 +109,6 @@ hyper_step_kernel(float* __restrict__ streams, const TY* __restrict__ y, const f
 // The same step, four neighbouring columns a thread and the stream count a
 // compile-time number: the copies move as 16-byte accesses and the small sums
 // over s unroll.  Per column the arithmetic and its order are those above.
-__device__ __forceinline__ float4 load4(const float* p) { return *reinterpret_cast<const float4*>(p); }
-__device__ __forceinline__ float4 load4(const __nv_bfloat16* p) {
-    const uint2 u = *reinterpret_cast<const uint2*>(p);
-    const float2 lo = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&u.x));
-    const float2 hi = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&u.y));
-    return make_float4(lo.x, lo.y, hi.x, hi.y);
-}
 __device__ __forceinline__ float4 fma4(float a, float4 b, float4 c) {
     return make_float4(fmaf(a, b.x, c.x), fmaf(a, b.y, c.y), fmaf(a, b.z, c.z), fmaf(a, b.w, c.w));
 }

@@ -4,8 +4,9 @@
 //    experts with the largest logits (ties: the lower index) and their weights:
 //    the softmax over the chosen logits only (mode 0), or each chosen logit's
 //    sigmoid, not renormalised (mode 1), or the softmax over all experts with the
-//    chosen ones' scores renormalised by their sum (mode 2); rfx_moe_route_scaled
-//    also multiplies the weights by a constant.  One warp a row.
+//    chosen ones' scores renormalised by their sum (mode 2) or as they are (mode 3);
+//    rfx_moe_route_groups also multiplies the weights by a constant and lets only the
+//    experts of the best groups be chosen.  One warp a row.
 //  * rfx_moe_up: act[(r, k), :] = f(W_up[e] (s x[r])) for expert e = ids[r, k];
 //    f = relu squared (act 0) or silu (act 1); act 2 is the gated, clamped form
 //    over W_up[e] = [gate rows | up rows]: g' = min(g, limit), u' = clamp(u,
@@ -32,7 +33,7 @@ constexpr int MAX_PER_LANE = 8;  // up to 256 experts
 
 __global__ void moe_route_kernel(const float* __restrict__ logits, int ld, const float* __restrict__ bias,
                                  int* __restrict__ ids, float* __restrict__ wts, int R, int E, int top,
-                                 int mode, float scale) {
+                                 int mode, float scale, int groups, int keep) {
     pdl_prologue();
     const int lane = threadIdx.x & 31;
     const int r = blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
@@ -42,6 +43,67 @@ __global__ void moe_route_kernel(const float* __restrict__ logits, int ld, const
     for (int i = 0; i < MAX_PER_LANE; ++i) {
         const int e = i * 32 + lane;
         z[i] = e < E ? logits[(size_t)r * ld + e] + (bias ? bias[e] : 0.0f) : -INFINITY;
+    }
+    // the softmax over all experts, before any of them is left out
+    float all_max = 0.0f, all_sum = 1.0f;
+    if (mode >= 2) {
+        float m = -INFINITY, s = 0.0f;
+#pragma unroll
+        for (int i = 0; i < MAX_PER_LANE; ++i) m = fmaxf(m, z[i]);
+        all_max = warp_max(m);
+#pragma unroll
+        for (int i = 0; i < MAX_PER_LANE; ++i)
+            if (i * 32 + lane < E) s += expf(z[i] - all_max);
+        all_sum = warp_sum(s);
+    }
+    if (keep < groups) {
+        // a group's score is the largest in it; the best `keep` groups stay, ties to the lower index
+        const int size = E / groups;
+        float best[MAX_PER_LANE];  // group g's best in lane g % 32
+#pragma unroll
+        for (int i = 0; i < MAX_PER_LANE; ++i) best[i] = -INFINITY;
+        for (int g = 0; g < groups; ++g) {
+            float m = -INFINITY;
+#pragma unroll
+            for (int i = 0; i < MAX_PER_LANE; ++i) {
+                const int e = i * 32 + lane;
+                if (e >= g * size && e < (g + 1) * size) m = fmaxf(m, z[i]);
+            }
+            m = warp_max(m);
+#pragma unroll
+            for (int i = 0; i < MAX_PER_LANE; ++i)
+                if (i * 32 + lane == g) best[i] = m;
+        }
+        unsigned kept[MAX_PER_LANE];  // a bit a group, the same in every lane
+#pragma unroll
+        for (int i = 0; i < MAX_PER_LANE; ++i) kept[i] = 0;
+        for (int k = 0; k < keep; ++k) {
+            float m = -INFINITY;
+            int at = 0x7fffffff;
+#pragma unroll
+            for (int i = 0; i < MAX_PER_LANE; ++i) {
+                const int g = i * 32 + lane;
+                if (g < groups && !(kept[i] >> lane & 1) && (at == 0x7fffffff || best[i] > m)) { m = best[i]; at = g; }
+            }
+#pragma unroll
+            for (int o = 16; o > 0; o >>= 1) {
+                const float om = __shfl_xor_sync(0xffffffffu, m, o);
+                const int oa = __shfl_xor_sync(0xffffffffu, at, o);
+                if (oa != 0x7fffffff && (at == 0x7fffffff || om > m || (om == m && oa < at))) { m = om; at = oa; }
+            }
+#pragma unroll
+            for (int i = 0; i < MAX_PER_LANE; ++i)
+                if (at / 32 == i) kept[i] |= 1u << (at & 31);
+        }
+#pragma unroll
+        for (int i = 0; i < MAX_PER_LANE; ++i) {
+            const int g = min((i * 32 + lane) / size, groups - 1);
+            unsigned word = 0;
+#pragma unroll
+            for (int j = 0; j < MAX_PER_LANE; ++j)
+                if (j == g / 32) word = kept[j];
+            if (!(word >> (g & 31) & 1)) z[i] = -INFINITY;
+        }
     }
     float zmax = 0.0f, sum = mode == 1 ? 1.0f : 0.0f, mine = 0.0f;  // lane k keeps the k-th choice's exponential
     int my_id = 0;
@@ -60,8 +122,9 @@ __global__ void moe_route_kernel(const float* __restrict__ logits, int ld, const
             if (ob > best || (ob == best && oe < best_e)) { best = ob; best_e = oe; }
         }
         if (k == 0) zmax = best;
+        best_e = min(best_e, E - 1);  // no logit above -inf is left (a row of NaNs): still an expert
         // mode 1: the chosen logit's sigmoid is the weight as it is (sum stays one)
-        const float p = mode == 1 ? 1.0f / (1.0f + expf(-best)) : expf(best - zmax);
+        const float p = mode == 1 ? 1.0f / (1.0f + expf(-best)) : expf(best - (mode >= 2 ? all_max : zmax));
         if (mode != 1) sum += p;
         if ((k & 31) == lane && k < 32) { mine = p; my_id = best_e; }
         if (k >= 32 && lane == 0) {  // more than 32 choices: written unnormalised, scaled below
@@ -72,22 +135,15 @@ __global__ void moe_route_kernel(const float* __restrict__ logits, int ld, const
         for (int i = 0; i < MAX_PER_LANE; ++i)
             if (i * 32 + lane == best_e) z[i] = -INFINITY;
     }
-    if (mode == 2) {
-        // scores are the softmax over all experts; the chosen ones' scores over their sum
-        // (+ 1e-20), times `scale`.  z holds -inf where an expert was chosen: the others'
-        // exponentials join the chosen ones' for the softmax's denominator
-        float rest = 0.0f;
-#pragma unroll
-        for (int i = 0; i < MAX_PER_LANE; ++i)
-            if (i * 32 + lane < E && z[i] != -INFINITY) rest += expf(z[i] - zmax);
-        const float total = sum + warp_sum(rest);
-        const float chosen = sum / total + 1e-20f;
+    if (mode >= 2) {
+        // scores are the softmax over all experts, as they are or over the chosen ones' sum (+ 1e-20)
+        const float chosen = mode == 2 ? sum / all_sum + 1e-20f : 1.0f;
         if (lane < top) {
             ids[(size_t)r * top + lane] = my_id;
-            wts[(size_t)r * top + lane] = (mine / total) / chosen * scale;
+            wts[(size_t)r * top + lane] = (mine / all_sum) / chosen * scale;
         }
         if (lane == 0)
-            for (int k = 32; k < top; ++k) wts[(size_t)r * top + k] = (wts[(size_t)r * top + k] / total) / chosen * scale;
+            for (int k = 32; k < top; ++k) wts[(size_t)r * top + k] = (wts[(size_t)r * top + k] / all_sum) / chosen * scale;
         return;
     }
     if (lane < top) {
@@ -389,22 +445,24 @@ extern "C" int rfx_moe_combine(const void* yg, int dt, const int* place, const f
 }
 
 // `ld`: floats between two rows of `logits` (>= E: further columns are ignored)
-// mode 2: the softmax over all experts, the chosen ones' scores over their sum (+ 1e-20);
-// `scale` multiplies the weights of every mode
-extern "C" int rfx_moe_route_scaled(const float* logits, int ld, const float* bias, int* ids, float* wts, int R,
-                                    int E, int top, int mode, float scale, void* stream) {
+// modes 2, 3: the softmax over all experts, the chosen ones' scores over their sum (+ 1e-20) or as
+// they are; `scale` multiplies the weights of every mode; of `groups` equal groups of neighbours
+// only the experts of the `keep` ones with the largest logit can be chosen
+extern "C" int rfx_moe_route_groups(const float* logits, int ld, const float* bias, int* ids, float* wts, int R,
+                                    int E, int top, int mode, float scale, int groups, int keep, void* stream) {
     if (R <= 0) return 0;
-    if (E <= 0 || top <= 0 || top > E || ld < E || mode < 0 || mode > 2) return RFX_ERR_BAD_ARG;
+    if (E <= 0 || top <= 0 || top > E || ld < E || mode < 0 || mode > 3) return RFX_ERR_BAD_ARG;
+    if (groups <= 0 || E % groups || keep <= 0 || keep > groups || top > keep * (E / groups)) return RFX_ERR_BAD_ARG;
     if (E > 32 * MAX_PER_LANE) return RFX_ERR_UNSUPPORTED;
     RFX_LAUNCH(moe_route_kernel, (R + 3) / 4, 128, 0, (cudaStream_t)stream, logits, ld, bias, ids, wts, R, E, top,
-               mode, scale);
+               mode, scale, groups, keep);
     return 0;
 }
 
 extern "C" int rfx_moe_route(const float* logits, int ld, const float* bias, int* ids, float* wts, int R, int E,
                              int top, int mode, void* stream) {
     if (mode != 0 && mode != 1) return RFX_ERR_BAD_ARG;
-    return rfx_moe_route_scaled(logits, ld, bias, ids, wts, R, E, top, mode, 1.0f, stream);
+    return rfx_moe_route_groups(logits, ld, bias, ids, wts, R, E, top, mode, 1.0f, 1, 1, stream);
 }
 
 extern "C" int rfx_moe_up(const void* x, const void* W, const int* ids, const float* in_scale, void* act, int dt,

@@ -12,6 +12,11 @@
 // (a normed embedding; y may be x).  A block a row; the row lives in shared memory between the sums of
 // squares and the outputs.
 //
+// sum_norm: x <- rms_norm(alpha * x + y) * (offset + w), and the new x in the product's type
+// where `out` is given: layers that norm the sum of the stream and a sublayer's result.  y is
+// 32-bit rows, or a mixture's expert rows in place order, whose weighted sum (in the order of
+// rank) is then made on the way.
+//
 // group_norm_gate: x [R, C] 32-bit in `groups` equal parts, each over its own
 // root mean square, times w[c] (or a weight the parts share, `shared`), times
 // sigmoid(z[r, col + c]) or silu of it (`act` 1) when a gate is given.
@@ -111,6 +116,140 @@ sandwich_norm4_kernel(const float* y, float* x, const float* __restrict__ w_post
                                (v[i].z * r2) * (next_offset + wn.z), (v[i].w * r2) * (next_offset + wn.w)));
         }
     }
+}
+
+// A sublayer's result: rows as they are, or (EXPERTS) sum_k wts[r, k] y[place[r top + k]].
+template <typename TY>
+struct SubResult {
+    const TY* y;
+    const int* place;
+    const float* wts;  // null: every weight is one
+    int top;
+};
+
+template <typename TY, typename TO, bool EXPERTS>
+__global__ void __launch_bounds__(256)
+sum_norm_kernel(SubResult<TY> s, float* __restrict__ x, float alpha, const float* __restrict__ w, float offset, float eps,
+                TO* __restrict__ out, int H) {
+    extern __shared__ __align__(16) float row[];  // [H]
+    __shared__ float scratch[32];
+    pdl_prologue();
+    const int r = blockIdx.x;
+    const size_t base = (size_t)r * H;
+    float ss = 0.0f;
+    for (int c = threadIdx.x; c < H; c += blockDim.x) {
+        float y = 0.0f;
+        if constexpr (EXPERTS)
+            for (int k = 0; k < s.top; ++k)
+                y = fmaf(s.wts ? s.wts[(size_t)r * s.top + k] : 1.0f, ld<TY>(s.y, (size_t)s.place[(size_t)r * s.top + k] * H + c), y);
+        else
+            y = ld<TY>(s.y, base + c);
+        const float v = fmaf(alpha, x[base + c], y);
+        row[c] = v;
+        ss = fmaf(v, v, ss);
+    }
+    const float f = 1.0f / sqrtf(block_sum(ss, scratch) / (float)H + eps);
+    for (int c = threadIdx.x; c < H; c += blockDim.x) {
+        const float v = (row[c] * f) * (offset + w[c]);
+        x[base + c] = v;
+        if (out) st<TO>(out, base + c, v);
+    }
+}
+
+// the same with four elements an access, the row in registers (up to V groups of four a thread)
+template <typename TY, typename TO, bool EXPERTS, int V>
+__global__ void __launch_bounds__(512)
+sum_norm4_kernel(SubResult<TY> s, float* __restrict__ x, float alpha, const float* __restrict__ w, float offset, float eps,
+                 TO* __restrict__ out, int H) {
+    __shared__ float scratch[32];
+    const int H4 = H / 4;
+    const int r = blockIdx.x;
+    const size_t base = (size_t)r * H;
+    const float4* w4 = reinterpret_cast<const float4*>(w);
+    float4* x4 = reinterpret_cast<float4*>(x + base);
+    float4 wv[V], v[V];
+    pdl_launch_dependents();
+#pragma unroll
+    for (int i = 0; i < V; ++i) {  // the weights are no kernel's output: they come before the wait
+        const int c = threadIdx.x + i * blockDim.x;
+        if (c < H4) wv[i] = w4[c];
+    }
+    pdl_wait();
+    float ss = 0.0f;
+    float4 y[V];
+#pragma unroll
+    for (int i = 0; i < V; ++i) {
+        const int c = threadIdx.x + i * blockDim.x;
+        if (c < H4) {
+            v[i] = x4[c];
+            y[i] = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+            if constexpr (!EXPERTS) y[i] = load4(s.y + base + 4 * (size_t)c);
+        }
+    }
+    if constexpr (EXPERTS) {
+        for (int k = 0; k < s.top; ++k) {
+            const TY* src = s.y + (size_t)s.place[(size_t)r * s.top + k] * H;
+            const float f = s.wts ? s.wts[(size_t)r * s.top + k] : 1.0f;
+#pragma unroll
+            for (int i = 0; i < V; ++i) {
+                const int c = threadIdx.x + i * blockDim.x;
+                if (c >= H4) continue;
+                const float4 t = load4(src + 4 * (size_t)c);
+                y[i].x = fmaf(f, t.x, y[i].x);
+                y[i].y = fmaf(f, t.y, y[i].y);
+                y[i].z = fmaf(f, t.z, y[i].z);
+                y[i].w = fmaf(f, t.w, y[i].w);
+            }
+        }
+    }
+#pragma unroll
+    for (int i = 0; i < V; ++i) {
+        const int c = threadIdx.x + i * blockDim.x;
+        if (c < H4) {
+            v[i].x = fmaf(alpha, v[i].x, y[i].x);
+            v[i].y = fmaf(alpha, v[i].y, y[i].y);
+            v[i].z = fmaf(alpha, v[i].z, y[i].z);
+            v[i].w = fmaf(alpha, v[i].w, y[i].w);
+            ss = fmaf(v[i].x, v[i].x, fmaf(v[i].y, v[i].y, fmaf(v[i].z, v[i].z, fmaf(v[i].w, v[i].w, ss))));
+        }
+    }
+    const float f = 1.0f / sqrtf(block_sum(ss, scratch) / (float)H + eps);
+#pragma unroll
+    for (int i = 0; i < V; ++i) {
+        const int c = threadIdx.x + i * blockDim.x;
+        if (c < H4) {
+            const float4 t = make_float4((v[i].x * f) * (offset + wv[i].x), (v[i].y * f) * (offset + wv[i].y),
+                                         (v[i].z * f) * (offset + wv[i].z), (v[i].w * f) * (offset + wv[i].w));
+            x4[c] = t;
+            if (out) store4(out + base + 4 * (size_t)c, t);
+        }
+    }
+}
+
+template <typename TY, typename TO, bool EXPERTS>
+int launch_sum_norm(const SubResult<TY>& y, float* x, float alpha, const float* w, float offset, float eps, TO* out, int R,
+                    int H, cudaStream_t s) {
+    const bool al = ((reinterpret_cast<uintptr_t>(y.y) | reinterpret_cast<uintptr_t>(x) | reinterpret_cast<uintptr_t>(w) |
+                      reinterpret_cast<uintptr_t>(out)) & 15) == 0;
+    if (H % 4 == 0 && H <= 4 * 512 * 4 && al) {
+        const int H4 = H / 4;
+        const int threads = H4 <= 128 ? 128 : H4 <= 256 ? 256 : 512;
+#define RFX_V(V) RFX_LAUNCH((sum_norm4_kernel<TY, TO, EXPERTS, V>), R, threads, 0, s, y, x, alpha, w, offset, eps, out, H)
+        if (H4 <= threads) RFX_V(1);
+        else if (H4 <= 2 * threads) RFX_V(2);
+        else RFX_V(4);
+#undef RFX_V
+        return 0;
+    }
+    const size_t smem = (size_t)H * sizeof(float);
+    if (smem > 200 * 1024) return RFX_ERR_UNSUPPORTED;
+    auto kernel = sum_norm_kernel<TY, TO, EXPERTS>;
+    if (smem > 48 * 1024) {
+        cudaError_t e = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+        if (e != cudaSuccess) return (int)e;
+    }
+    RFX_LAUNCH(kernel, R, 256, smem, s, y, x, alpha, w, offset, eps, out, H);
+    return 0;
 }
 
 // sigmoid(t), or (act 1) silu(t)
@@ -314,6 +453,32 @@ extern "C" int rfx_sandwich_norm(const float* y, float* x, const float* w_post, 
     else return RFX_ERR_BAD_ARG;
 #undef RFX_GO
     return 0;
+}
+
+// y: [R, H] (32-bit), or with `place` the expert rows that row r's `top` places name
+extern "C" int rfx_sum_norm(const void* y, int y_dt, const int* place, const float* wts, int top, float* x, float alpha,
+                            const float* w, float offset, float eps, void* out, int out_dt, int R, int H, void* stream) {
+    if (R <= 0) return 0;
+    if (H <= 0 || !w || (place && top <= 0)) return RFX_ERR_BAD_ARG;
+    cudaStream_t s = (cudaStream_t)stream;
+#define RFX_GO(TY, TO, EX)                                                                                              \
+    return launch_sum_norm<TY, TO, EX>(SubResult<TY>{(const TY*)y, place, wts, top}, x, alpha, w, offset, eps, (TO*)out, \
+                                       R, H, s)
+#define RFX_OUT(TY, EX)                                     \
+    do {                                                    \
+        if (out_dt == RFX_DT_F32) RFX_GO(TY, float, EX);    \
+        if (out_dt == RFX_DT_BF16) RFX_GO(TY, __nv_bfloat16, EX); \
+        return RFX_ERR_BAD_ARG;                             \
+    } while (0)
+    if (place) {
+        if (y_dt == RFX_DT_F32) RFX_OUT(float, true);
+        if (y_dt == RFX_DT_BF16) RFX_OUT(__nv_bfloat16, true);
+    } else if (y_dt == RFX_DT_F32) {
+        RFX_OUT(float, false);
+    }
+#undef RFX_OUT
+#undef RFX_GO
+    return RFX_ERR_BAD_ARG;
 }
 
 extern "C" int rfx_group_norm_gate(const float* x, const float* w, float eps, const float* z, int ldz, int zcol,

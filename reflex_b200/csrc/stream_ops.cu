@@ -334,6 +334,37 @@ extern "C" int rfx_sigmoid_gate_mul(void* a, int a_dt, const void* z, int z_dt, 
     return 0;
 }
 
+// a[r, h, :] *= sigmoid(z[r, col + h]), heads of `n` elements
+namespace {
+
+template <typename TA, typename TZ>
+__global__ void __launch_bounds__(256)
+head_gate_mul_kernel(TA* __restrict__ a, const TZ* __restrict__ z, int ldz, int col, int heads, int n) {
+    pdl_prologue();
+    const size_t r = blockIdx.x;
+    const int H = heads * n;
+    for (int c = blockIdx.y * blockDim.x + threadIdx.x; c < H; c += gridDim.y * blockDim.x)
+        st<TA>(a, r * H + c, ld<TA>(a, r * H + c) / (1.0f + expf(-ld<TZ>(z, r * ldz + col + c / n))));
+}
+
+}  // namespace
+
+extern "C" int rfx_head_gate_mul(void* a, int a_dt, const void* z, int z_dt, int ldz, int col, int R, int heads, int n,
+                                 void* stream) {
+    if (R <= 0 || heads <= 0 || n <= 0) return 0;
+    if (col < 0 || col + heads > ldz) return RFX_ERR_BAD_ARG;
+    cudaStream_t s = (cudaStream_t)stream;
+    const dim3 grid(R, row_chunks(R, heads * n));
+#define RFX_GO(TA, TZ) \
+    RFX_LAUNCH((head_gate_mul_kernel<TA, TZ>), grid, 256, 0, s, (TA*)a, (const TZ*)z, ldz, col, heads, n)
+    if (a_dt == RFX_DT_F32 && z_dt == RFX_DT_F32) RFX_GO(float, float);
+    else if (a_dt == RFX_DT_BF16 && z_dt == RFX_DT_F32) RFX_GO(__nv_bfloat16, float);
+    else if (a_dt == RFX_DT_BF16 && z_dt == RFX_DT_BF16) RFX_GO(__nv_bfloat16, __nv_bfloat16);
+    else return RFX_ERR_BAD_ARG;
+#undef RFX_GO
+    return 0;
+}
+
 // ---- a state group's rows copied aside ------------------------------------------
 namespace {
 

@@ -886,17 +886,18 @@ def mlstm_out(num, den, proj, g_off: int, weight, eps: float, heads: int, vdim: 
 MOE_ACTIVATIONS = {"relu2": 0, "silu": 1, "glu_clamped": 2, "swiglu": 3}
 
 
-MOE_SCORES = {"softmax_top": 0, "sigmoid": 1, "softmax_all": 2}
+MOE_SCORES = {"softmax_top": 0, "sigmoid": 1, "softmax_all": 2, "softmax": 3}
 
 
 def moe_route(logits: torch.Tensor, bias: Optional[torch.Tensor], top: int, experts: Optional[int] = None,
-              scores: str = "softmax_top", col0: int = 0, scale: float = 1.0):
+              scores: str = "softmax_top", col0: int = 0, scale: float = 1.0, groups=None):
     """Router logits float32 [R, experts] (+ bias) -> ids int32 [R, top], the
     experts with the largest logits, and weights float32 [R, top]: the softmax
     over the chosen logits only ("softmax_top"), or each chosen logit's sigmoid
     as it is ("sigmoid"), or the softmax over all experts with the chosen ones'
-    scores divided by their sum + 1e-20 ("softmax_all"); `scale` multiplies the
-    weights.  With `experts` only that many columns of `logits`,
+    scores divided by their sum + 1e-20 ("softmax_all") or as they are ("softmax");
+    `scale` multiplies the weights.  `groups` = (count, keep): of `count` equal groups of
+    neighbours only the `keep` ones with the largest best logit can be chosen from.  With `experts` only that many columns of `logits`,
     from column `col0` on, are router logits (the rest belongs to the caller: a
     product stacked with others')."""
     R, ld = logits.shape
@@ -905,16 +906,35 @@ def moe_route(logits: torch.Tensor, bias: Optional[torch.Tensor], top: int, expe
         raise InvalidInput("moe_route: the router's columns do not fit into the logits' rows")
     ids = _new((R, top), torch.int32, logits.device)
     wts = _new((R, top), torch.float32, logits.device)
-    st = native.lib().rfx_moe_route_scaled(_chk(logits, "logits", torch.float32) + 4 * int(col0), ld,
+    count, keep = (int(g) for g in groups) if groups else (1, 1)
+    if count <= 0 or E % count or not (0 < keep <= count) or top > keep * (E // count):
+        raise InvalidInput("moe_route: the groups must divide the experts and the kept ones hold the chosen")
+    st = native.lib().rfx_moe_route_groups(_chk(logits, "logits", torch.float32) + 4 * int(col0), ld,
                                            _chk(bias, "bias", torch.float32), ids.data_ptr(), wts.data_ptr(), R, E,
-                                           int(top), MOE_SCORES[scores], float(scale), _stream())
+                                           int(top), MOE_SCORES[scores], float(scale), count, keep, _stream())
     native.check(st, f"moe_route (experts={E}, top={top})")
     return ids, wts
 
 
+class ExpertRows:
+    """A mixture's expert results before their weighted sum: row r's is sum_k wts[r, k]
+    rows[place[r top + k]] (`wts` None: every weight is one).  `summed` makes it."""
+
+    def __init__(self, rows: torch.Tensor, place: torch.Tensor, wts: Optional[torch.Tensor], n_rows: int, top: int):
+        self.rows, self.place, self.wts, self.n_rows, self.top = rows, place, wts, n_rows, top
+
+    def summed(self) -> torch.Tensor:
+        width = self.rows.shape[1]
+        y = _new((self.n_rows, width), torch.float32, self.rows.device)
+        native.check(native.lib().rfx_moe_combine(
+            _chk(self.rows, "rows"), dt_code(self.rows.dtype), self.place.data_ptr(),
+            _chk(self.wts, "wts", torch.float32), y.data_ptr(), self.n_rows, self.top, width, _stream()), "moe_combine")
+        return y
+
+
 def moe_experts(x: torch.Tensor, up: torch.Tensor, down: torch.Tensor, ids: torch.Tensor,
                 wts: torch.Tensor, activation: str = "relu2", weight_input: bool = False,
-                alpha: float = 1.0, limit: float = 0.0) -> torch.Tensor:
+                alpha: float = 1.0, limit: float = 0.0, leave_sum: bool = False):
     """sum_k wts[r, k] down[e] act(up[e] x[r]), e = ids[r, k]; up [experts, ff,
     width], down [experts, width, ff]; float32 [R, width].  Every (row, choice)
     reads its expert's matrices itself: the form for a few rows, and the exact
@@ -922,7 +942,8 @@ def moe_experts(x: torch.Tensor, up: torch.Tensor, down: torch.Tensor, ids: torc
     gate rows and then its up rows, and act is the clamped gated form with
     `alpha` and `limit` (`glu_clamped`); "swiglu": the same layout, silu(gate) * up.  `weight_input`: the weight multiplies
     the expert's input instead of its output, sum_k down[e] act(up[e] (wts[r, k]
-    x[r]))."""
+    x[r])).  `leave_sum`: the grouped form may hand back the experts' rows (`ExpertRows`)
+    in place of their sum."""
     R, width = x.shape
     E, ff, _w = up.shape
     gated = activation in ("glu_clamped", "swiglu")
@@ -933,7 +954,8 @@ def moe_experts(x: torch.Tensor, up: torch.Tensor, down: torch.Tensor, ids: torc
     if x.dtype == torch.bfloat16 and MOE_GROUPED and R >= MOE_GROUPED_MIN_ROWS:
         # captured steps too, as long as the library's grouped product (no wait for the host) is there
         if not torch.cuda.is_current_stream_capturing() or (_GROUPED_MM[0] and width % 8 == 0 and ff % 8 == 0):
-            return moe_experts_grouped(x, up, down, ids, wts, activation, weight_input, alpha, limit)
+            rows = moe_experts_grouped(x, up, down, ids, wts, activation, weight_input, alpha, limit)
+            return rows if leave_sum else rows.summed()
     act = _new((R * top, ff), x.dtype, x.device)
     st = native.lib().rfx_moe_up(_chk(x, "x"), _chk(up, "up", x.dtype), _chk(ids, "ids", torch.int32),
                                  _chk(in_scale, "wts", torch.float32), act.data_ptr(), dt_code(x.dtype), R, top,
@@ -956,13 +978,13 @@ MOE_GROUPED_MIN_ROWS = _env_int("REFLEX_B200_MOE_GROUPED_MIN_ROWS", 2, 1, 1 << 3
 
 def moe_experts_grouped(x: torch.Tensor, up: torch.Tensor, down: torch.Tensor, ids: torch.Tensor,
                         wts: torch.Tensor, activation: str = "relu2", weight_input: bool = False,
-                        alpha: float = 1.0, limit: float = 0.0) -> torch.Tensor:
-    """The same sum for many bfloat16 rows (prefill): the (row, choice) pairs are
+                        alpha: float = 1.0, limit: float = 0.0) -> ExpertRows:
+    """The same for many bfloat16 rows (prefill), up to the sum: the (row, choice) pairs are
     placed expert by expert on the device, each expert's block of rows goes
     through its two matrices as library products (where the dense layers use
     them too: the library's grouped product, or one product an expert where it
-    has none, for which the host reads the experts' offsets once), and a row's
-    results are summed in the order of their rank."""
+    has none, for which the host reads the experts' offsets once); a row's results
+    are to be summed in the order of their rank."""
     R, width = x.shape
     E, ff, _w = up.shape
     gated = activation in ("glu_clamped", "swiglu")
@@ -1007,11 +1029,7 @@ def moe_experts_grouped(x: torch.Tensor, up: torch.Tensor, down: torch.Tensor, i
             _GROUPED_MM[0] = False  # this build of the library has none for these operands: one product an expert
             yg = None
         if yg is not None:
-            y = _new((R, width), torch.float32, x.device)
-            native.check(lib.rfx_moe_combine(_chk(yg, "yg"), dt_code(yg.dtype), place.data_ptr(),
-                                             _chk(out_wts, "wts", torch.float32), y.data_ptr(), R, top, width,
-                                             _stream()), "moe_combine")
-            return y
+            return ExpertRows(yg, place, out_wts, R, top)
     off = offsets.tolist()  # the one wait for the device
     act = _new((n, up.shape[1]), x.dtype, x.device)
     for e in range(E):
@@ -1022,11 +1040,7 @@ def moe_experts_grouped(x: torch.Tensor, up: torch.Tensor, down: torch.Tensor, i
     for e in range(E):
         if off[e + 1] > off[e]:
             torch.mm(act[off[e]:off[e + 1]], down[e].t(), out_dtype=torch.float32, out=yg[off[e]:off[e + 1]])
-    y = _new((R, width), torch.float32, x.device)
-    native.check(lib.rfx_moe_combine(yg.data_ptr(), dt_code(yg.dtype), place.data_ptr(),
-                                     _chk(out_wts, "wts", torch.float32), y.data_ptr(), R, top, width, _stream()),
-                 "moe_combine")
-    return y
+    return ExpertRows(yg, place, out_wts, R, top)
 
 
 _GROUPED_MM = [True, True]  # whether the library's grouped product is tried, and its 32-bit output
@@ -1304,9 +1318,18 @@ def hyper_collapse(streams: torch.Tensor, write: Optional["StreamWrite"], n_stre
 
 
 # ------------------------------------------------------------ gates, activations
-def sigmoid_gate_mul_(a: torch.Tensor, z: torch.Tensor, col: int) -> torch.Tensor:
-    """a[r, c] *= sigmoid(z[r, col + c]), in place; the sigmoid is 32-bit."""
+def sigmoid_gate_mul_(a: torch.Tensor, z: torch.Tensor, col: int, heads: int = 0) -> torch.Tensor:
+    """a[r, c] *= sigmoid(z[r, col + c]), in place; the sigmoid is 32-bit.  `heads`: one
+    number for each of that many equal parts of a row, a[r, c] *= sigmoid(z[r, col +
+    c / (H / heads)])."""
     R, H = a.shape
+    if heads:
+        if H % heads or col < 0 or col + heads > z.shape[1] or z.shape[0] != R:
+            raise InvalidInput("sigmoid_gate_mul: the gate's columns do not fit into z or the heads into a row")
+        st = native.lib().rfx_head_gate_mul(_chk(a, "a"), dt_code(a.dtype), _chk(z, "z"), dt_code(z.dtype),
+                                            z.shape[1], int(col), R, heads, H // heads, _stream())
+        native.check(st, "head_gate_mul")
+        return a
     if col < 0 or col + H > z.shape[1] or z.shape[0] != R:
         raise InvalidInput("sigmoid_gate_mul: the gate's columns do not fit into z")
     st = native.lib().rfx_sigmoid_gate_mul(_chk(a, "a"), dt_code(a.dtype), _chk(z, "z"), dt_code(z.dtype),
@@ -1421,6 +1444,28 @@ def post_norm(y: torch.Tensor, x: torch.Tensor, weight: torch.Tensor, weight_off
         float(weight_offset), 1.0, float(eps), 0, 0.0, 0.0, out.data_ptr() if out is not None else 0,
         dt_code(out_dtype) if out_dtype is not None else F32, 1 if fresh else 0, R, H, _stream())
     native.check(st, f"post_norm (H={H})")
+    return out
+
+
+def sum_norm(y, x: torch.Tensor, alpha: float, weight: torch.Tensor, weight_offset: float, eps: float,
+             out_dtype: Optional[torch.dtype]):
+    """x <- rms_norm(alpha * x + y) * (weight_offset + weight) in place, float32 [R, H];
+    `y` float32 [R, H] or `ExpertRows`, whose weighted sum is then made here.  With
+    `out_dtype` also returns the new x in that type, the next product's input."""
+    R, H = x.shape
+    rows = y if isinstance(y, ExpertRows) else None
+    if (rows.n_rows, rows.rows.shape[1]) != (R, H) if rows is not None else tuple(y.shape) != (R, H):
+        raise InvalidInput("sum_norm: y and x must have the same shape")
+    out = _new((R, H), out_dtype, x.device) if out_dtype is not None else None
+    src = rows.rows if rows is not None else y
+    st = native.lib().rfx_sum_norm(
+        _chk(src, "y", None if rows is not None else torch.float32), dt_code(src.dtype),
+        rows.place.data_ptr() if rows is not None else 0,
+        _chk(rows.wts, "wts", torch.float32) if rows is not None else 0, rows.top if rows is not None else 1,
+        _chk(x, "x", torch.float32), float(alpha), _chk(weight, "weight", torch.float32), float(weight_offset),
+        float(eps), out.data_ptr() if out is not None else 0, dt_code(out_dtype) if out_dtype is not None else F32,
+        R, H, _stream())
+    native.check(st, f"sum_norm (H={H})")
     return out
 
 
@@ -1698,21 +1743,29 @@ def gated_delta_scan(qkv: torch.Tensor, gates: torch.Tensor, state: torch.Tensor
 
 
 # --------------------------------- rotation, then the norm; latents with a rotated part
-def _plain_rotation(rotation, what: str):
+def _half_rotation(rotation, what: str):
     if rotation is None:
-        return None, 0
-    if rotation.pairing != "half" or rotation.magnitude != 1.0:
-        raise InvalidInput(f"{what}: takes a plain half-split rotation")
-    return rotation.denominators, int(rotation.rotary_dim)
+        return None, 0, 1.0
+    if rotation.pairing != "half":
+        raise InvalidInput(f"{what}: takes a half-split rotation")
+    return rotation.denominators, int(rotation.rotary_dim), float(rotation.magnitude)
+
+
+def _plain_rotation(rotation, what: str):
+    denom, dims, magnitude = _half_rotation(rotation, what)
+    if magnitude != 1.0:
+        raise InvalidInput(f"{what}: takes a rotation of magnitude one")
+    return denom, dims
 
 
 def rot_qkv_post(proj: torch.Tensor, bias: Optional[torch.Tensor], rotation, unit_eps: Optional[float],
                  mix: Optional[torch.Tensor], v_first: Optional[torch.Tensor], keep_values: bool, row_pos, row_slot,
                  k_pages, v_pages, page_table, page_size: int, nq: int, nkv: int, dim: int, vdim: int, pad: int,
-                 writes_cache: bool, out_dtype: torch.dtype):
+                 writes_cache: bool, out_dtype: torch.dtype, norms=None):
     """Rows [q | k | v] plus `bias` (float32): q and k rotated (a half-split
     `parts.Rotation` or None), then, with `unit_eps`, divided by their root mean
-    square per head; q out as [R, nq * pad], k and v into the cache, heads `pad`
+    square per head; or, with `norms` = (q weight, k weight, eps, weight offset), normed
+    per head first and rotated after it (a row without a k part needs no k weight); q out as [R, nq * pad], k and v into the cache, heads `pad`
     wide (zeros beyond `dim` and `vdim`).  `v_first` (float32 [R, nkv * vdim]) and
     `mix` (one float32 number): the values become (1 - mix) v + mix v_first first.
     Returns (q, values): `keep_values` asks for the step's unmixed values as
@@ -1722,12 +1775,17 @@ def rot_qkv_post(proj: torch.Tensor, bias: Optional[torch.Tensor], rotation, uni
         raise InvalidInput("rot_qkv_post: the q | k | v columns do not fit into the rows")
     if v_first is not None and (tuple(v_first.shape) != (R, nkv * vdim) or mix is None):
         raise InvalidInput("rot_qkv_post: the first values' rows must match the values and come with a mix")
-    denom, rot = _plain_rotation(rotation, "rot_qkv_post")
+    denom, rot, magnitude = _half_rotation(rotation, "rot_qkv_post")
+    if norms is not None and (unit_eps is not None or (writes_cache and norms[1] is None)):
+        raise InvalidInput("rot_qkv_post: one kind of norm, with a weight for each part that is there")
+    q_w, k_w, n_eps, n_off = norms if norms is not None else (None, None, 0.0, 0.0)
+    unit = 2 if norms is not None else 0 if unit_eps is None else 1
     q = _new((R, nq * pad), out_dtype, proj.device)
     kept = _new((R, nkv * vdim), torch.float32, proj.device, keep=True) if keep_values else None
     st = native.lib().rfx_rot_qkv_post(
         _chk(proj, "proj"), dt_code(proj.dtype), proj.shape[1], _chk(bias, "bias", torch.float32),
-        _chk(denom, "denominators", torch.float32), rot, 0 if unit_eps is None else 1, float(unit_eps or 0.0),
+        _chk(denom, "denominators", torch.float32), rot, magnitude, unit, float(n_eps if unit == 2 else unit_eps or 0.0),
+        _chk(q_w, "q weight", torch.float32), _chk(k_w, "k weight", torch.float32), float(n_off),
         _chk(mix, "mix", torch.float32) if v_first is not None else 0, _chk(v_first, "v_first", torch.float32),
         kept.data_ptr() if kept is not None else 0, _chk(row_pos, "row_pos", torch.int32),
         _chk(row_slot, "row_slot", torch.int32), q.data_ptr(), _chk(k_pages, "k_pages", out_dtype),
@@ -1769,6 +1827,27 @@ def latent_rot_post(proj: torch.Tensor, kv_weight: torch.Tensor, eps: float, rot
         page_table.shape[1], page_size, R, heads, dim, rot_dim, rank, width, 1 if writes_cache else 0, _stream())
     native.check(st, f"latent_rot_post (rank={rank}, rot={rot_dim})")
     return out
+
+
+def latent_low_post(proj: torch.Tensor, q_weight: torch.Tensor, kv_weight: torch.Tensor, eps: float, rotation, row_pos,
+                    row_slot, pages, page_table, page_size: int, q_rank: int, rank: int, rot_dim: int, width: int,
+                    writes_cache: bool, out_dtype: torch.dtype) -> torch.Tensor:
+    """Rows [query latent | latent | shared key part | ...]: returns the RMS-normed
+    query latent [R, q_rank] and writes [normed latent | rotated key part | zeros],
+    `width` elements, into the cache at the rows' positions."""
+    R = proj.shape[0]
+    denom, rot = _plain_rotation(rotation, "latent_low_post")
+    if rot not in (0, rot_dim):
+        raise InvalidInput("latent_low_post: the rotation covers the whole rotated part")
+    q = _new((R, q_rank), out_dtype, proj.device)
+    st = native.lib().rfx_latent_low_post(
+        _chk(proj, "proj"), dt_code(proj.dtype), proj.shape[1], _chk(q_weight, "q_weight", torch.float32),
+        _chk(kv_weight, "kv_weight", torch.float32), float(eps), _chk(denom, "denominators", torch.float32),
+        _chk(row_pos, "row_pos", torch.int32), _chk(row_slot, "row_slot", torch.int32), q.data_ptr(),
+        _chk(pages, "pages", out_dtype), dt_code(out_dtype), _chk(page_table, "page_table", torch.int32),
+        page_table.shape[1], page_size, R, q_rank, rank, rot_dim, width, 1 if writes_cache else 0, _stream())
+    native.check(st, f"latent_low_post (q_rank={q_rank}, rank={rank}, rot={rot_dim})")
+    return q
 
 
 LATENT_WIDTH_STEP = 64   # cached latent rows the tensor-core kernels take: in steps of this, up to

@@ -111,8 +111,8 @@ _SIGNATURES = {
     "rfx_moe_gather": [c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_void_p],
     "rfx_moe_activation": [c_void_p, c_int, c_longlong, c_int, c_void_p],
     "rfx_moe_combine": [c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_void_p],
-    "rfx_moe_route_scaled": [c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_float,
-                             c_void_p],
+    "rfx_moe_route_groups": [c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_float,
+                             c_int, c_int, c_void_p],
     "rfx_sandwich_norm": [c_void_p, c_void_p, c_void_p, c_float, c_float, c_float, c_void_p, c_float, c_float,
                           c_void_p, c_int, c_int, c_int, c_int, c_void_p],
     "rfx_group_norm_gate": [c_void_p, c_void_p, c_float, c_void_p, c_int, c_int, c_int, c_int, c_void_p, c_int, c_int,
@@ -128,12 +128,18 @@ _SIGNATURES = {
                                    c_void_p],
     "rfx_gated_delta_chunk": [c_void_p, c_void_p, c_void_p, c_longlong, c_longlong, c_void_p, c_void_p, c_int, c_void_p,
                               c_int, c_int, c_int, c_int, c_void_p, c_void_p],
-    "rfx_rot_qkv_post": [c_void_p, c_int, c_int, c_void_p, c_void_p, c_int, c_int, c_float, c_void_p, c_void_p,
+    "rfx_rot_qkv_post": [c_void_p, c_int, c_int, c_void_p, c_void_p, c_int, c_float, c_int, c_float, c_void_p, c_void_p,
+                         c_float, c_void_p, c_void_p,
                          c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_int, c_int,
                          c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p],
     "rfx_latent_decode": [c_void_p, c_void_p, c_void_p, c_int, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_int,
                           c_int, c_int, c_int, c_int, c_int, c_float, c_void_p, c_longlong, c_int, c_int, c_void_p,
                           c_void_p],
+    "rfx_latent_low_post": [c_void_p, c_int, c_int, c_void_p, c_void_p, c_float, c_void_p, c_void_p, c_void_p, c_void_p,
+                            c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p],
+    "rfx_head_gate_mul": [c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p],
+    "rfx_sum_norm": [c_void_p, c_int, c_void_p, c_void_p, c_int, c_void_p, c_float, c_void_p, c_float, c_float,
+                     c_void_p, c_int, c_int, c_int, c_void_p],
     "rfx_latent_gather": [c_void_p, c_void_p, c_int, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int,
                           c_int, c_int, c_void_p],
     "rfx_latent_value_columns": [c_int, c_int],

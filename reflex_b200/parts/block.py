@@ -5,7 +5,8 @@
 one norm that both sublayers read.  "sandwich": a norm on both sides of every
 sublayer, h += m * post1(mixer(norm1(h))); h += m * post2(ffn(norm2(h))), m one
 number of the layer.  "postnorm": a norm only on what a sublayer gives,
-h += norm1(mixer(h)); h += norm2(ffn(h)).  The residual stream is 32-bit; each add is
+h += norm1(mixer(h)); h += norm2(ffn(h)).  "sum_norm": the norm of the sum,
+h = norm1(a h + mixer(h)); h = norm2(a h + ffn(h)), a one number of the layer.  The residual stream is 32-bit; each add is
 fused into the norm that follows it, so a block hands its last delta on as
 `pending` and the next block's (or the model's final) norm adds it
 (src/model/decode_step.rs:199-210, 293-300).
@@ -332,5 +333,43 @@ class PostNormBlock(PreNormBlock):
             y = self.feed_forward.forward(x)
             n = self.feed_forward_norm
             x = ops.post_norm(y, hidden, n.weight, n.spec.weight_offset, n.spec.eps, after)
+            ops.prof_mark("norm")
+        return hidden, (ReadyRows(x) if x is not None else None)
+
+
+@register_block("sum_norm")
+class SumNormBlock(PostNormBlock):
+    """h = norm1(a h + mixer(h)); h = norm2(a h + ffn(h)): the stream itself is normed
+    after every sublayer, `alpha` (the spec's parameter) times it beside what the
+    sublayer gives (RMS norms with any weight offset).  Multiple, sum, norm and the
+    rounded rows of the next sublayer are one pass (`ops.sum_norm`), which also makes
+    the weighted sum of a mixture's expert rows where the feed-forward leaves that to
+    it (`leaves_sum`)."""
+
+    def __init__(self, spec: LayerSpec, dtype: torch.dtype, device):
+        super().__init__(spec, dtype, device)
+        self.alpha = float(dict(spec.params).get("alpha", 1.0))
+
+    def forward(self, hidden: torch.Tensor, pending, ctx, next_norm=None):
+        from .. import ops
+
+        if isinstance(pending, ReadyRows):
+            x = pending.rows
+        else:
+            if pending is not None and not isinstance(pending, ops.NormedInput):
+                ops.add_(hidden, pending)
+            x = ops.cast_rows(hidden, self.dtype)
+            ops.prof_mark("norm")
+        after = self.dtype if next_norm is PostNormBlock.READS_STREAM else None
+        y = self.mixer.forward(x, ctx)
+        n = self.mixer_norm
+        x = ops.sum_norm(y, hidden, self.alpha, n.weight, n.spec.weight_offset, n.spec.eps,
+                         self.dtype if self.has_feed_forward else after)
+        ops.prof_mark("norm")
+        if self.has_feed_forward:
+            leaves = getattr(self.feed_forward, "leaves_sum", False)
+            y = self.feed_forward.forward(x, leave_sum=True) if leaves else self.feed_forward.forward(x)
+            n = self.feed_forward_norm
+            x = ops.sum_norm(y, hidden, self.alpha, n.weight, n.spec.weight_offset, n.spec.eps, after)
             ops.prof_mark("norm")
         return hidden, (ReadyRows(x) if x is not None else None)

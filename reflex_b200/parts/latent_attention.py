@@ -10,10 +10,14 @@ With h the mixer's input [rows, hidden]:
   out = W_o concat_h( sigmoid(W_g h)_h * sum_j p_ij v_j )
 There is no position encoding.
 
-Without `q_rank` (the other form) q = W_q h, per head `head_dim` unrotated and
-`rot_dim` rotated elements, [unrotated | rotated], and W_dkv h has `rot_dim` more
-rows: one rotated key part r_j all heads share, not normed:
+With `rot_dim` (the rotated form; without `q_rank` it takes q = W_q h) q has per head
+`head_dim` unrotated and `rot_dim` rotated elements, [unrotated | rotated], and
+W_dkv h has `rot_dim` more rows: one rotated key part r_j all heads share, not normed:
   s_ij = (q_i . k_j + rot(q_i') . rot(r_j)) * scale
+`gate` "element" (of this form): out = W_o (sigmoid(W_g h) * concat_h(...)), element by
+element.  A rotation of neighbouring elements (`pairing` "consecutive") becomes one of
+halves by the order of the rotated rows of W_uq and W_dkv, the same for both, which
+changes no score.
 The cached row is then [c | rot(r) | zeros], and the folded query is followed by
 its rotated part.  For a prompt's many rows the other order of the same products is
 cheaper: every head's keys [W_uk c | rot(r)] and values W_uv c of the step's
@@ -30,6 +34,7 @@ head.  Norms, scores, the softmax and the gates are 32-bit.
 
 from __future__ import annotations
 
+import dataclasses
 from typing import Dict
 
 import torch
@@ -47,7 +52,7 @@ class LatentAttention:
 
     @property
     def supports_fused_residual(self) -> bool:
-        return self.q_rank > 0
+        return not self.rotated
 
     def __init__(self, spec: MixerSpec, dtype: torch.dtype, device):
         self.spec = spec
@@ -60,18 +65,20 @@ class LatentAttention:
         self.kv_rank = int(spec.param("kv_rank"))
         self.eps = float(spec.param("eps"))
         self.has_sink = bool(spec.param("sink", False))
+        self.rotated = self.rot_dim > 0 or not self.q_rank  # cached rows with room beside the latent
         self.has_gate = spec.param("gate") == "head"
-        if self.q_rank and (self.rot_dim or self.position is not None):
-            raise InvalidInput("latent_attention: a rotated part goes with queries straight from the input")
-        if not self.q_rank and self.has_gate:
-            raise InvalidInput("latent_attention: a gate goes with queries through a latent")
+        self.element_gate = spec.param("gate") == "element"
+        if not self.rotated and self.position is not None:
+            raise InvalidInput("latent_attention: a rotation needs a rotated part")
+        if self.has_gate if self.rotated else self.element_gate:
+            raise InvalidInput("latent_attention: a gate per head goes with no rotated part, one per element with one")
         # elements of a cached row: the latent and the rotated part, in steps the tensor-core kernels take
         step = ops.LATENT_WIDTH_STEP if dtype == torch.bfloat16 else 16
-        self.width = self.kv_rank if self.q_rank else (self.kv_rank + self.rot_dim + step - 1) // step * step
+        self.width = (self.kv_rank + self.rot_dim + step - 1) // step * step if self.rotated else self.kv_rank
         # the form that makes every head's keys and values (prompts): padded key and value sizes
         d, dv = spec.head_dim + self.rot_dim, spec.value_dim
         self.dk, self.dvp = (d + 63) // 64 * 64, (dv + 63) // 64 * 64
-        self.expands = (not self.q_rank and dtype == torch.bfloat16 and self.dk <= 192 and self.dvp <= 128
+        self.expands = (self.rotated and dtype == torch.bfloat16 and self.dk <= 192 and self.dvp <= 128
                         and self.dvp <= self.dk and dv % 16 == 0 and spec.scale > 0)
         self.kv_up = None
         self.down = self.q_up = self.k_absorb = self.v_up = self.o = None
@@ -84,7 +91,7 @@ class LatentAttention:
         rot = int(spec.param("rot_dim", 0) or 0)
         if qr:
             out = {"q_down": TensorInfo((qr, W), "matrix"), "q_norm": TensorInfo((qr,), "norm"),
-                   "q_up": TensorInfo((H * d, qr), "matrix")}
+                   "q_up": TensorInfo((H * (d + rot), qr), "matrix")}
         else:
             out = {"q_proj": TensorInfo((H * (d + rot), W), "matrix")}
         out.update({
@@ -96,6 +103,8 @@ class LatentAttention:
             out["sink"] = TensorInfo((H,), "bias")
         if spec.param("gate") == "head":
             out["gate"] = TensorInfo((H, W), "matrix")
+        elif spec.param("gate") == "element":
+            out["gate"] = TensorInfo((H * dv, W), "matrix")
         return out
 
     def cache_spec(self) -> KVSpec:
@@ -112,16 +121,29 @@ class LatentAttention:
         def f32(t):
             return t.to(device=self.device, dtype=torch.float32).contiguous()
 
-        parts = [dev(tensors["q_down" if self.q_rank else "q_proj"]), dev(tensors["kv_down"])]
+        q_rows, kv_down = dev(tensors["q_up" if self.q_rank else "q_proj"]), dev(tensors["kv_down"])
+        order = self._pair_order()
+        if order is not None:  # rotated rows: all pairs' first elements, then all second ones
+            q_rows = q_rows.view(H, d + self.rot_dim, -1)[:, order["query"]].reshape(q_rows.shape)
+            kv_down = kv_down[order["key"]]
+        parts = [dev(tensors["q_down"]) if self.q_rank else q_rows, kv_down]
         if self.has_gate:
             parts.append(dev(tensors["gate"]))
-        if not self.q_rank:
+
+        def padded():
             # zero rows up to a multiple of 8: the product's rows stay 16-byte aligned
             rows = sum(p.shape[0] for p in parts)
             parts.append(torch.zeros((-rows % 8, s.hidden_size), dtype=self.dtype, device=self.device))
+
+        if self.rotated:
+            padded()
+        if self.element_gate:
+            self.gate_col = sum(p.shape[0] for p in parts)
+            parts.append(dev(tensors["gate"]))
+            padded()
         self.down = torch.cat(parts, dim=0).contiguous()  # one product for both latents and the gates
         if self.q_rank:
-            self.q_up = dev(tensors["q_up"]).contiguous()
+            self.q_up = q_rows.contiguous()
             self.q_norm = f32(tensors["q_norm"])
         # W_uk per head, transposed: [H, kv_rank, dim], so that q_h -> W_uk,h^T q_h is a per-head product
         self.k_absorb = dev(tensors["k_up"]).view(H, d, self.kv_rank).transpose(1, 2).contiguous()
@@ -145,8 +167,8 @@ class LatentAttention:
         s = self.spec
         kv, batch = ctx.kv, ctx.batch
         H = s.num_heads
-        if not self.q_rank:
-            return self._forward_direct(x, ctx)
+        if self.rotated:
+            return self._forward_rotated(x, ctx)
         proj = ops.linear(x, self.down, out_dtype=torch.float32)
         ops.prof_mark("qkv_gemm")
         cq, gate = ops.latent_post(proj, self.q_norm, self.kv_norm, self.eps, batch.row_pos, batch.row_slot,
@@ -171,16 +193,41 @@ class LatentAttention:
         ops.prof_mark("o_proj")
         return out
 
-    def _forward_direct(self, x, ctx):
-        """The form without a query latent; the delta [rows, hidden] comes back 32-bit."""
+    def _pair_order(self):
+        """The order that turns pairs of neighbours into pairs of halves, for a head's query
+        rows and for the rows of W_dkv; None where the pairs are halves already."""
+        if self.position is None or self.position.rotation().pairing == "half":
+            return None
+        pairs = torch.arange(self.rot_dim, device=self.device)
+        halves = torch.cat([pairs[0::2], pairs[1::2]])
+        return {"query": torch.cat([torch.arange(self.spec.head_dim, device=self.device), self.spec.head_dim + halves]),
+                "key": torch.cat([torch.arange(self.kv_rank, device=self.device), self.kv_rank + halves])}
+
+    def _rotation(self):
+        if self.position is None:
+            return None
+        return dataclasses.replace(self.position.rotation(), pairing="half")  # `_pair_order` made it so
+
+    def _forward_rotated(self, x, ctx):
+        """The form with a rotated part; the delta [rows, hidden] comes back 32-bit."""
         s, kv, batch = self.spec, ctx.kv, ctx.batch
-        H = s.num_heads
+        H, d = s.num_heads, s.head_dim
         proj = ops.linear(x, self.down, out_dtype=torch.float32)
         ops.prof_mark("qkv_gemm")
-        rotation = None if self.position is None else self.position.rotation()
-        post = (proj, self.kv_norm, self.eps, rotation, batch.row_pos, batch.row_slot, kv.k_pages, kv.page_table,
-                kv.page_size, H, s.head_dim, self.rot_dim, self.kv_rank, self.width, ctx.writes_cache, self.dtype)
-        if self._expand(batch):
+        rotation = self._rotation()
+        expand = self._expand(batch)
+        rows, writes = proj, ctx.writes_cache
+        if self.q_rank:
+            cq = ops.latent_low_post(proj, self.q_norm, self.kv_norm, self.eps, rotation, batch.row_pos, batch.row_slot,
+                                     kv.k_pages, kv.page_table, kv.page_size, self.q_rank, self.kv_rank, self.rot_dim,
+                                     self.width, writes, self.dtype)
+            ops.prof_mark("latent_post")
+            rows = ops.linear(cq, self.q_up, out_dtype=torch.float32 if x.shape[0] <= ops.GEMV_MAX_ROWS else None)
+            ops.prof_mark("q_up")
+            writes = False  # the latents are cached already: only queries are left
+        post = (rows, self.kv_norm, self.eps, rotation, batch.row_pos, batch.row_slot, kv.k_pages, kv.page_table,
+                kv.page_size, H, d, self.rot_dim, self.kv_rank, self.width, writes, self.dtype)
+        if expand:
             q = ops.latent_rot_post(*post, query_width=self.dk)
             ops.prof_mark("latent_post")
             rows, base = ops.latent_gather(kv.k_pages, kv.page_table, kv.page_size, batch, self.width)
@@ -199,6 +246,8 @@ class LatentAttention:
             ops.prof_mark("attn")
             vals = ops.heads_linear(attn, self.v_up)  # of each head the latent's elements; the rest is dropped
             ops.prof_mark("v_up")
+        if self.element_gate:
+            ops.sigmoid_gate_mul_(vals, proj, self.gate_col)
         out = ops.linear(vals, self.o, out_dtype=torch.float32)
         ops.prof_mark("o_proj")
         return out

@@ -19,7 +19,10 @@ width (the same clamped gated form with `shared_limit`) runs for every row and
 is added times sigmoid(w_sg . x), one number a row; its gate's row rides along
 as one more row of the router's matrix.  `scores` "softmax_all": the weights are
 the softmax over all experts' logits, the chosen ones' divided by their sum
-(+ 1e-20); `score_scale` multiplies the weights.  `activation` "swiglu": an
+(+ 1e-20); "softmax": the same scores as they are; `score_scale` multiplies the
+weights.  `groups` (count, keep): the experts form `count` equal groups of
+neighbours, a group's score is the largest in it, and only experts of the `keep`
+best groups can be chosen (ties: the lower index).  `activation` "swiglu": an
 expert is W_down (silu(W_gate x) * (W_up x)).  `shared_kind` "swiglu" (with
 `shared_ff`): the shared expert is that gated silu form and is added as it is,
 with no gate of its own.
@@ -55,6 +58,7 @@ class MixtureOfExperts:
         self.shared_limit = float(spec.param("shared_limit", 0.0))
         self.shared_kind = str(spec.param("shared_kind", "glu_clamped_gated"))
         self.score_scale = float(spec.param("score_scale", 1.0))
+        self.groups = spec.param("groups")
         self.router = self.router_bias = self.up = self.down = None
         self.shared_gate_up = self.shared_down = None
 
@@ -109,7 +113,14 @@ class MixtureOfExperts:
     def adopt_input_weight(self, rows: torch.Tensor) -> None:
         self.router = rows
 
-    def forward(self, x, residual=None, onto=None, proj=None):
+    @property
+    def leaves_sum(self) -> bool:
+        """Whether `forward(..., leave_sum=True)` is understood: the caller's next kernel
+        makes the weighted sum of the experts' rows (`ops.ExpertRows`) where the
+        grouped form has made them."""
+        return not self.shared_ff
+
+    def forward(self, x, residual=None, onto=None, proj=None, leave_sum=False):
         """`onto`: a 32-bit delta another part made from the same input (a mixer
         beside this feed-forward); the result is added onto it and it is returned.
         `proj` = (float32 rows, first column): the router's product, already made
@@ -119,10 +130,10 @@ class MixtureOfExperts:
         else:
             logits, col0 = proj
         ids, wts = ops.moe_route(logits, self.router_bias, self.top, experts=self.experts, scores=self.scores,
-                                 col0=col0, scale=self.score_scale)
+                                 col0=col0, scale=self.score_scale, groups=self.groups)
         ops.prof_mark("moe_router")
         out = ops.moe_experts(x, self.up, self.down, ids, wts, self.activation, self.weight_input, self.alpha,
-                              self.limit)
+                              self.limit, leave_sum=leave_sum and self.leaves_sum and onto is None)
         ops.prof_mark("moe_experts")
         if self.shared_ff and self.shared_kind == "swiglu":
             # the shared expert as it is: gate and up woven into one product, added to the experts' sum

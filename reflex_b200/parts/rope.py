@@ -1,4 +1,5 @@
-"""Rotary position encoding, half-split (NeoX) pairing.
+"""Rotary position encoding, half-split (NeoX) pairing unless the spec's `pairing`
+parameter says "consecutive".
 
 For a head vector t[0..d) and i < rd/2:  theta = (float)pos / base^(2i/rd);
 (t_i, t_{i+rd/2}) <- (t_i cos - t_{i+rd/2} sin, t_i sin + t_{i+rd/2} cos);
@@ -25,6 +26,7 @@ from .registry import Rotation, TensorInfo, register_position
 @register_position("rope_neox")
 class RotaryNeox:
     capturable = True
+    magnitude = 1.0  # of the cosines and sines
 
     def __init__(self, spec: PositionSpec, dtype: torch.dtype, device):
         if spec.rotary_dim % 2 or not (0 < spec.rotary_dim <= spec.head_dim):
@@ -45,7 +47,8 @@ class RotaryNeox:
         pass
 
     def rotation(self) -> Rotation:
-        return Rotation(self.denominators, self.spec.rotary_dim, "half", 1.0)
+        pairing = str(dict(self.spec.params).get("pairing", "half"))
+        return Rotation(self.denominators, self.spec.rotary_dim, pairing, self.magnitude)
 
 
 @register_position("rope_linear")
@@ -95,3 +98,36 @@ class RotaryScaled(RotaryNeox):
                 g = (1.0 - s) * f / factor + s * f
             denom.append(1.0 / g)
         self.denominators = torch.tensor(denom, dtype=torch.float64).to(torch.float32).to(device)
+
+
+@register_position("rope_yarn")
+class RotaryYarn(RotaryNeox):
+    """The rotation with frequencies scaled by how often a pair turns within the
+    original context, and a magnitude.
+
+    With f_i = theta^(-2i/rd), the parameters `factor`, `original`, `fast`, `slow`,
+    and n(t) = rd ln(original / (2 pi t)) / (2 ln theta), the (fractional) index of the
+    pair that turns t times within `original` positions: lo = max(floor(n(fast)), 0),
+    hi = min(ceil(n(slow)), rd - 1), ramp_i = (i - lo) / max(hi - lo, 0.001) within
+    [0, 1], and the frequency is f_i (1 - ramp_i) + f_i / factor * ramp_i.  Cosine and
+    sine are multiplied by 0.1 ln(factor) + 1."""
+
+    def __init__(self, spec: PositionSpec, dtype: torch.dtype, device):
+        super().__init__(spec, dtype, device)
+        p = dict(spec.params)
+        factor, original, fast, slow = (float(p[k]) for k in ("factor", "original", "fast", "slow"))
+        if min(factor, original, fast, slow) <= 0 or spec.theta <= 0 or spec.theta == 1:
+            raise InvalidInput("rope_yarn: factor, original, fast and slow must be positive, theta positive and not 1")
+        rd, base = spec.rotary_dim, float(spec.theta)
+
+        def index_of(turns: float) -> float:
+            return rd * math.log(original / (2.0 * math.pi * turns)) / (2.0 * math.log(base))
+
+        lo, hi = max(math.floor(index_of(fast)), 0), min(math.ceil(index_of(slow)), rd - 1)
+        denom = []
+        for i in range(rd // 2):
+            f = math.pow(base, -2.0 * i / float(rd))
+            ramp = min(max((i - lo) / max(hi - lo, 0.001), 0.0), 1.0)
+            denom.append(1.0 / (f / factor * ramp + f * (1.0 - ramp)))
+        self.denominators = torch.tensor(denom, dtype=torch.float64).to(torch.float32).to(device)
+        self.magnitude = 0.1 * math.log(factor) + 1.0
