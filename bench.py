@@ -365,6 +365,30 @@ def zivulix_config(z):
             "layers": layers}
 
 
+def pidodra_config(z):
+    """Pidodra at the sizes of `z`: of four layers two are a latent attention (a rotated part
+    of 64 beside the models' head size, queries through a latent, a gate per element), one a
+    grouped attention (a quarter as many key/value heads, YaRN frequencies, a gate per head)
+    and one the same with that one's keys and values, every layer with experts in four groups
+    of which two are kept; every earlier key."""
+    lat = {"type": "latent_attention",
+           "mixer": {"heads": z["heads"], "dim": z["dim"], "rot_dim": 64, "vdim": z["dim"], "q_rank": z["q_rank"],
+                     "kv_rank": z["kv_rank"], "scale": (z["dim"] + 64) ** -0.5, "rot": {"base": 500000.0, "dims": 64}}}
+    att = {"heads": z["heads"], "kv_heads": max(1, z["heads"] // 4), "dim": z["dim"], "vdim": z["dim"],
+           "scale": z["dim"] ** -0.5,
+           "rot": {"base": 500000.0, "dims": z["dim"],
+                   "scaling": {"factor": 4.0, "original": 8192, "fast": 32.0, "slow": 1.0}}}
+    moe = {"kind": "moe", "expert": {"ff": z["expert_ff"]},
+           "router": {"experts": z["experts"], "top": z["top"], "scale": 1.5, "groups": {"count": 4, "keep": 2}}}
+    layers = []
+    for i in range(z["layers"]):
+        mixer = [lat, {"type": "attention", "mixer": att}, lat,
+                 {"type": "attention", "mixer": dict(att, kv_from=i - 2)}][i % 4]
+        layers.append(dict(mixer, mlp=moe))
+    return {"architecture": "Pidodra", "vocab": z["vocab"], "width": z["width"], "norm": {"eps": 1e-5},
+            "embedding": {"scale": 1.0}, "postln_alpha": 2.0, "layers": layers}
+
+
 def qwen3_config_like(z):
     cfg = dict(QWEN3_8B)
     cfg.update({"num_hidden_layers": z["layers"], "hidden_size": z["width"], "num_attention_heads": z["heads"],
@@ -379,7 +403,9 @@ def design_comparison(args) -> int:
     equal sizes (and, for Pakarax, beside Kegasun too: the model with a
     recurrence and experts; for Zelinex beside Pakarax: the model with two mixers
     side by side, experts and a loop; for Zivulix beside Kegasun, the model with a latent
-    attention, and Zelinex, the model with a delta rule), with every phase's time in a
+    attention, and Zelinex, the model with a delta rule; for Pidodra beside Zivulix, the
+    model with a rotated latent attention, and Kegasun, the model with a latent attention and
+    experts), with every phase's time in a
     prefill and in a decode step."""
     import torch
 
@@ -393,9 +419,10 @@ def design_comparison(args) -> int:
     mine = args.design
     beside = [("qwen3", qwen3_config_like)] + {
         "pakarax": [("kegasun", kegasun_config)], "zelinex": [("pakarax", pakarax_config)],
-        "zivulix": [("kegasun", kegasun_config), ("zelinex", zelinex_config)]}.get(mine, [])
+        "zivulix": [("kegasun", kegasun_config), ("zelinex", zelinex_config)],
+        "pidodra": [("zivulix", zivulix_config), ("kegasun", kegasun_config), ("zelinex", zelinex_config)]}.get(mine, [])
     mine_config = {"kegasun": kegasun_config, "pakarax": pakarax_config, "purusun": purusun_config,
-                   "zelinex": zelinex_config, "zivulix": zivulix_config}[mine]
+                   "zelinex": zelinex_config, "zivulix": zivulix_config, "pidodra": pidodra_config}[mine]
     out = {"metric": f"prefill and decode tokens/s, {mine} beside " + " and ".join(n for n, _ in beside)
                      + " at equal sizes", "unit": "tokens/s",
            "dtype": "bf16", "data": "synthetic: seeded uniform token ids, random-init weights",
@@ -520,7 +547,7 @@ def main() -> int:
                     help="workloads beside the headline: 14b and 32b add their points (default: all)")
     ap.add_argument("--prompt", type=int, default=PROMPT, help="prompt tokens before the decode steps")
     ap.add_argument("--context", type=int, default=CONTEXT, help="cache positions per sequence")
-    ap.add_argument("--design", default="", choices=["", "kegasun", "pakarax", "purusun", "zelinex", "zivulix"],
+    ap.add_argument("--design", default="", choices=["", "kegasun", "pakarax", "pidodra", "purusun", "zelinex", "zivulix"],
                     help="instead of the headline: this design beside Qwen3 at equal sizes (prefill, decode, phases)")
     ap.add_argument("--sizes", default="w1024,w2048,w4096", help="with --design: which of the sizes " +
                     ", ".join(sorted(DESIGN_SIZES)))

@@ -31,7 +31,7 @@ int decode_entry(const void* q, const void* k_pages, const void* v_pages, const 
                  int max_pages, int page_size, const int* row_pos, const int* row_slot, void* out,
                  float* partial, int R, int nq, int nkv, int head_dim, int n_splits, int window,
                  int keep_first, float scale, const float* sink, const float* slopes, float softcap, int cluster_merge,
-                 long long pool_pages, int* err, void* stream) {
+                 long long pool_pages, int* err, void* stream, rfx::RowGate gate = rfx::RowGate{nullptr, 0, 0, 0}) {
     if (R <= 0) return 0;
     if (page_size != PAGE || nkv <= 0 || nq % nkv != 0 || n_splits < 1) return RFX_ERR_BAD_ARG;
     if (softcap < 0.0f || (softcap > 0.0f && slopes)) return RFX_ERR_UNSUPPORTED;  // one or the other
@@ -53,7 +53,8 @@ int decode_entry(const void* q, const void* k_pages, const void* v_pages, const 
     // with slopes or a cap: the kernel's form that has that term
 #define RFX_FORM(DD, T, M)                                                                                  \
     launch_decode<DD, T, M>(q, k_pages, v_pages, pool_pages, cache, row_pos, row_slot, out, partial, R, nq, \
-                            n_splits, window, keep_first, scale, sink, slopes, softcap, cluster_merge, 1, err, s)
+                            n_splits, window, keep_first, scale, sink, slopes, softcap, cluster_merge, 1, err, s, \
+                            gate)
 #define RFX_GO(DD, T) (slopes ? RFX_FORM(DD, T, 1) : softcap > 0.0f ? RFX_FORM(DD, T, 2) : RFX_FORM(DD, T, 0))
 #define RFX_CASE(DD)                                        \
     case DD:                                                \
@@ -98,18 +99,21 @@ extern "C" int rfx_attention_decode(const void* q, const void* k_pages, const vo
 
 // The same with `keep_first` (the first so many positions of a sequence stay
 // visible beyond the window) and `softcap` (> 0: a score s becomes softcap * tanh(s / softcap)
-// before the softmax; not together with slopes).
+// before the softmax; not together with slopes).  `gate_z` (or null): rows of `gate_ld` elements; head
+// h's output of row r is multiplied by sigmoid(gate_z[r, gate_col + h]).
 extern "C" int rfx_attention_decode_kf(const void* q, const void* k_pages, const void* v_pages,
                                        const int* page_table, int max_pages, int page_size,
                                        const int* row_pos, const int* row_slot, void* out,
                                        float* partial, int R, int nq, int nkv, int head_dim,
                                        int n_splits, int window, int keep_first, float scale, const float* sink,
                                        const float* slopes, float softcap, long long pool_pages, int cluster,
-                                       int* err, void* stream) {
-    if (keep_first < 0) return RFX_ERR_BAD_ARG;
+                                       const void* gate_z, int gate_dt, int gate_ld, int gate_col, int* err,
+                                       void* stream) {
+    rfx::RowGate gate;
+    if (keep_first < 0 || !rfx::row_gate(&gate, gate_z, gate_dt, gate_ld, gate_col, nq)) return RFX_ERR_BAD_ARG;
     return decode_entry(q, k_pages, v_pages, page_table, max_pages, page_size, row_pos, row_slot, out,
                         cluster ? nullptr : partial, R, nq, nkv, head_dim, n_splits, window, keep_first, scale,
-                        sink, slopes, softcap, cluster ? 1 : 0, pool_pages, err, stream);
+                        sink, slopes, softcap, cluster ? 1 : 0, pool_pages, err, stream, gate);
 }
 
 // The same with 2, 4, 8 or (where the device places such a cluster) 16 splits that

@@ -71,7 +71,7 @@ attention_decode_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_
                         __nv_bfloat16* __restrict__ out, float* __restrict__ partial, int nq,
                         int n_htiles, int n_splits, int window, int keep_first, float scale_log2,
                         const float* __restrict__ sink, const float* __restrict__ slopes, float softcap,
-                        int cluster_merge, int early, int trace_id, int* __restrict__ err) {
+                        int cluster_merge, int early, rfx::RowGate gate, int trace_id, int* __restrict__ err) {
     constexpr int LD = D + 8;
     constexpr int TILE = TMA ? PAGE * D : PAGE * LD;  // elements of a page's key (or value) tile
     extern __shared__ __align__(16) uint8_t smem_raw[];
@@ -405,7 +405,9 @@ attention_decode_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_
         if (n_splits == 1) {
             // a sink adds exp(sink - max) to the denominator, once, with no value
             if (sink) L += exp2f(sink[h0 + row] * LOG2E - M);
-            out[head * DV + e] = __float2bfloat16_rn(A / L);
+            float y = A / L;
+            if (gate.z) y *= gate.factor(r, h0 + row);
+            out[head * DV + e] = __float2bfloat16_rn(y);
         } else if (!cluster_merge) {
             float* p = partial + (head * n_splits + split) * (DV + 2);
             p[e] = A;
@@ -448,7 +450,8 @@ attention_decode_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_
                 A += recv_a[(size_t)sidx * slice + off] * f;
             }
             if (sink) L = __fadd_rn(L, exp2f(sink[h0 + row] * LOG2E - M));
-            const float inv = 1.0f / L;
+            float inv = 1.0f / L;
+            if (gate.z) inv *= gate.factor(r, h0 + row);
             out[((size_t)r * nq + h0 + row) * DV + e] = __float2bfloat16_rn(A * inv);
         }
     }
@@ -460,7 +463,7 @@ attention_decode_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_
 constexpr int MAX_SPLITS = 64;
 __global__ void attention_combine_kernel(const float* __restrict__ partial,
                                          __nv_bfloat16* __restrict__ out, int D, int n_splits,
-                                         const float* __restrict__ sink, int nq) {
+                                         const float* __restrict__ sink, int nq, rfx::RowGate gate) {
     __shared__ float wgt[MAX_SPLITS];
     __shared__ float lw[MAX_SPLITS];
     __shared__ float inv_l;
@@ -498,6 +501,7 @@ __global__ void attention_combine_kernel(const float* __restrict__ partial,
                 for (int sidx = 0; sidx < n_splits; ++sidx) L += lw[sidx];
                 if (sink && !dry) L = __fadd_rn(L, exp2f(sink[head % nq] * LOG2E - M));
                 inv_l = 1.0f / L;
+                if (gate.z && !dry) inv_l *= gate.factor(head / nq, (int)(head % nq));
             }
         }
         __syncthreads();
@@ -535,7 +539,8 @@ template <int D, bool TMA, int MODE, int DV = D, bool SHARED = false, int STG = 
 int launch_decode(const void* q, const void* k_pages, const void* v_pages, long long pool_pages,
                   const PagedKV& cache, const int* row_pos, const int* row_slot, void* out, float* partial,
                   int R, int nq, int n_splits, int window, int keep_first, float scale, const float* sink,
-                  const float* slopes, float softcap, int cluster_merge, int early, int* err, cudaStream_t s) {
+                  const float* slopes, float softcap, int cluster_merge, int early, int* err, cudaStream_t s,
+                  rfx::RowGate gate = rfx::RowGate{nullptr, 0, 0, 0}) {
     constexpr int LD = D + 8;
     const int g = nq / cache.n_kv_heads;
     const int n_htiles = (g + 7) / 8;
@@ -588,11 +593,11 @@ int launch_decode(const void* q, const void* k_pages, const void* v_pages, long 
                     (const __nv_bfloat16*)q, (const __nv_bfloat16*)k_pages, (const __nv_bfloat16*)v_pages,
                     cache, row_pos, row_slot, (__nv_bfloat16*)out, partial, nq, n_htiles, n_splits, window,
                     keep_first, scale * LOG2E, sink, slopes, softcap, cluster_merge, early,
-                    g_dtrace_next++, err);
+                    gate, g_dtrace_next++, err);
     if (e != cudaSuccess) return (int)e;
     if (n_splits > 1 && !cluster_merge)
         RFX_LAUNCH(attention_combine_kernel, R * nq, DV <= 128 ? 64 : 128, 0, s, (const float*)partial,
-                   (__nv_bfloat16*)out, DV, n_splits, sink, nq);
+                   (__nv_bfloat16*)out, DV, n_splits, sink, nq, gate);
     return 0;
 }
 

@@ -122,6 +122,31 @@ struct Smem {
     }
 };
 
+// 16 neighbouring gate logits; the place is a multiple of 16 bytes
+__device__ __forceinline__ void load_logits16(const rfx::RowGate& gate, size_t at, float (&z)[16]) {
+    if (gate.bf16) {
+        const __nv_bfloat16* p = reinterpret_cast<const __nv_bfloat16*>(gate.z) + at;
+#pragma unroll
+        for (int i = 0; i < 2; ++i) {
+            const uint4 u = reinterpret_cast<const uint4*>(p)[i];
+            const __nv_bfloat162* h = reinterpret_cast<const __nv_bfloat162*>(&u);
+#pragma unroll
+            for (int j = 0; j < 4; ++j) {
+                const float2 f = __bfloat1622float2(h[j]);
+                z[8 * i + 2 * j] = f.x;
+                z[8 * i + 2 * j + 1] = f.y;
+            }
+        }
+    } else {
+        const float4* p = reinterpret_cast<const float4*>(reinterpret_cast<const float*>(gate.z) + at);
+#pragma unroll
+        for (int i = 0; i < 4; ++i) {
+            const float4 f = p[i];
+            z[4 * i] = f.x, z[4 * i + 1] = f.y, z[4 * i + 2] = f.z, z[4 * i + 3] = f.w;
+        }
+    }
+}
+
 // SLOPES: a linear distance bias, slope_h * (query position - key position) off
 // every score of head h; taken off the raw score as (slope / scale) * distance,
 // so that the scale's multiply-add in the exponent covers it.  Without it the
@@ -134,6 +159,7 @@ struct Smem {
 // values made for this step): position p of sequence i is row seq_base[i] + p, head h's key its
 // columns h DK .., its value its columns v_col + h DV .. (map_k and map_v then are the same
 // matrix).  `dv` columns of a value are written out (DV without CONTIG).
+// `gate`: a head's output times one number a row and head, or (CONTIG) element by element.
 template <int DK, int DV, int MODE, bool CONTIG>
 __global__ void __launch_bounds__(THREADS)
 attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q,
@@ -144,7 +170,7 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q,
                             __nv_bfloat16* __restrict__ out, int nq, int bq, int window, int keep_first,
                             float scale_log2, float in_scale, const float* __restrict__ sink,
                             const float* __restrict__ slopes, const int* __restrict__ seq_base, int v_col, int dv,
-                            int* __restrict__ err) {
+                            rfx::RowGate gate, int* __restrict__ err) {
     constexpr bool SLOPES = MODE == 1;
     static_assert(DK % 64 == 0 && DK <= 192 && (DV == 64 || DV == 128), "keys up to 192, values 64 or 128");
     constexpr int KB = DK / 64, VB = DV / 64;  // 64-column blocks of a row
@@ -485,18 +511,30 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q,
         if (ok && n_pages > 0) {
             tc_fence_after_sync();
             // a sink adds exp(sink - reference) to the denominator, once, with no value
-            const float inv = 1.0f / (sink ? l + ex2(fmaf(sink[kvh * g + row_h], 1.4426950408889634f, -m)) : l);
+            float inv = 1.0f / (sink ? l + ex2(fmaf(sink[kvh * g + row_h], 1.4426950408889634f, -m)) : l);
+            if (!CONTIG && gate.z && row_valid) inv *= gate.factor(row0 + q0 + row_p, kvh * g + row_h);
             const int ow = CONTIG ? dv : DV;  // columns of an output head
             __nv_bfloat16* o = out + ((size_t)(row0 + q0 + row_p) * nq + kvh * g + row_h) * ow;
             // two loads of 16 columns in flight: the next one travels while this one is stored
             uint32_t rr[2][16];
             tmem_ld_16_nowait(tmem + lane_addr + O_COL, rr[0]);
+            // an element gate's next 16 logits travel likewise, 16 bytes an access
+            const bool element_gate = CONTIG && gate.z != nullptr;
+            const size_t gate_at = (size_t)(row0 + q0 + row_p) * gate.ld + gate.col + (size_t)(kvh * g + row_h) * ow;
+            float zz[2][16];
+            if (element_gate && row_valid) load_logits16(gate, gate_at, zz[0]);
 #pragma unroll
             for (int c = 0; c < DV / 16; ++c) {
                 tmem_ld_wait_16(rr[c & 1]);
                 if (c + 1 < DV / 16) tmem_ld_16_nowait(tmem + lane_addr + O_COL + (c + 1) * 16, rr[(c + 1) & 1]);
                 uint32_t(&r)[16] = rr[c & 1];
                 if (row_valid && (!CONTIG || c * 16 < ow)) {
+                    if (element_gate) {
+                        if ((c + 1) * 16 < ow) load_logits16(gate, gate_at + (c + 1) * 16, zz[(c + 1) & 1]);
+#pragma unroll
+                        for (int e = 0; e < 16; ++e)
+                            r[e] = __float_as_uint(__fdividef(__uint_as_float(r[e]), 1.0f + __expf(-zz[c & 1][e])));
+                    }
                     uint4 v[2];
                     __nv_bfloat162* pv2 = reinterpret_cast<__nv_bfloat162*>(v);
 #pragma unroll
@@ -540,7 +578,8 @@ template <int D, int MODE>
 int launch_tc(const void* q, const void* k_pages, const void* v_pages, long long n_pages_total,
               const PagedKV& cache, const int* seq_slot, const int* seq_start, const int* seq_new,
               const int* seq_row0, void* out, int S, int max_new, int R, int nq, int window, int keep_first,
-              float scale, const float* sink, const float* slopes, float softcap, int* err, cudaStream_t s) {
+              float scale, const float* sink, const float* slopes, float softcap, rfx::RowGate gate, int* err,
+              cudaStream_t s) {
     const int g = nq / cache.n_kv_heads;
     if (g > ROWS) return RFX_ERR_UNSUPPORTED;
     const int bq = ROWS / g;
@@ -559,7 +598,7 @@ int launch_tc(const void* q, const void* k_pages, const void* v_pages, long long
     RFX_LAUNCH(kernel, grid, THREADS, smem, s, mq, mk, mv, cache, seq_slot, seq_start, seq_new, seq_row0,
                (__nv_bfloat16*)out, nq, bq, window, keep_first,
                (MODE >= 2 ? softcap : scale) * 1.4426950408889634f, MODE >= 2 ? scale / softcap : 1.0f, sink, slopes,
-               (const int*)nullptr, 0, D, err);
+               (const int*)nullptr, 0, D, gate, err);
     return 0;
 }
 
@@ -579,7 +618,8 @@ bool make_map_matrix(CUtensorMap* map, const void* base, long long rows, long lo
 template <int DK, int DV>
 int launch_contig(const void* q, const void* kv, long long kv_rows, const int* seq_base, const int* seq_slot,
                   const int* seq_start, const int* seq_new, const int* seq_row0, void* out, int S, int max_new, int R,
-                  int heads, int dv, int window, float scale, const float* sink, int* err, cudaStream_t s) {
+                  int heads, int dv, int window, float scale, const float* sink, rfx::RowGate gate, int* err,
+                  cudaStream_t s) {
     CUtensorMap mq, mkv;
     if (!make_map_q(&mq, q, R, heads, DK, 1, ROWS) ||
         !make_map_matrix(&mkv, kv, kv_rows, (long long)heads * (DK + DV)))
@@ -593,7 +633,7 @@ int launch_contig(const void* q, const void* kv, long long kv_rows, const int* s
     PagedKV cache{nullptr, 0, PAGE, heads, DK};
     RFX_LAUNCH(kernel, grid, THREADS, smem, s, mq, mkv, mkv, cache, seq_slot, seq_start, seq_new, seq_row0,
                (__nv_bfloat16*)out, heads, ROWS, window, 0, scale * 1.4426950408889634f, 1.0f, sink,
-               (const float*)nullptr, seq_base, heads * DK, dv, err);
+               (const float*)nullptr, seq_base, heads * DK, dv, gate, err);
     return 0;
 }
 
@@ -615,15 +655,19 @@ extern "C" int rfx_attention_prefill_tc_trace(void* buffer, int ctas) {
 
 // `keep_first`: with a window, the first so many positions of a sequence stay visible
 // beyond it.  `softcap` > 0: a score s becomes softcap * tanh(s / softcap) (not with slopes);
-// `score_bound` > 0: the caller's word that no |s| is larger.
+// `score_bound` > 0: the caller's word that no |s| is larger.  `gate_z` (or null): rows of
+// `gate_ld` elements; head h's output of row r is multiplied by sigmoid(gate_z[r, gate_col + h]).
 extern "C" int rfx_attention_prefill_tc_kf(const void* q, const void* k_pages, const void* v_pages,
                                            long long n_pages_total, const int* page_table, int max_pages,
                                            int page_size, const int* seq_slot, const int* seq_start,
                                            const int* seq_new, const int* seq_row0, void* out, int S,
                                            int max_new, int R, int nq, int nkv, int head_dim, int window,
                                            int keep_first, float scale, const float* sink, const float* slopes,
-                                           float softcap, float score_bound, int* err, void* stream) {
+                                           float softcap, float score_bound, const void* gate_z, int gate_dt,
+                                           int gate_ld, int gate_col, int* err, void* stream) {
     if (S <= 0 || max_new <= 0 || R <= 0) return 0;
+    rfx::RowGate gate;
+    if (!rfx::row_gate(&gate, gate_z, gate_dt, gate_ld, gate_col, nq)) return RFX_ERR_BAD_ARG;
     if (keep_first < 0 || !(scale > 0.0f)) return RFX_ERR_UNSUPPORTED;  // the maximum is taken before the scale
     if (page_size != PAGE || nkv <= 0 || nq % nkv != 0) return RFX_ERR_BAD_ARG;
     if (softcap < 0.0f || (softcap > 0.0f && slopes)) return RFX_ERR_UNSUPPORTED;
@@ -635,7 +679,7 @@ extern "C" int rfx_attention_prefill_tc_kf(const void* q, const void* k_pages, c
     cudaStream_t s = (cudaStream_t)stream;
 #define RFX_GO(DD, M)                                                                                   \
     launch_tc<DD, M>(q, k_pages, v_pages, n_pages_total, cache, seq_slot, seq_start, seq_new, seq_row0, \
-                      out, S, max_new, R, nq, window, keep_first, scale, sink, slopes, softcap, err, s)
+                      out, S, max_new, R, nq, window, keep_first, scale, sink, slopes, softcap, gate, err, s)
     const int mode = slopes ? 1 : !(softcap > 0.0f) ? 0 : (score_bound > 0.0f && score_bound <= attn::TANH_SMALL * softcap) ? 3 : 2;
 #define RFX_D(DD)                             \
     if (head_dim == DD) {                     \
@@ -660,27 +704,33 @@ extern "C" int rfx_attention_prefill_tc(const void* q, const void* k_pages, cons
                                         void* stream) {
     return rfx_attention_prefill_tc_kf(q, k_pages, v_pages, n_pages_total, page_table, max_pages, page_size,
                                        seq_slot, seq_start, seq_new, seq_row0, out, S, max_new, R, nq, nkv,
-                                       head_dim, window, 0, scale, sink, slopes, 0.0f, 0.0f, err, stream);
+                                       head_dim, window, 0, scale, sink, slopes, 0.0f, 0.0f, nullptr, 0, 0, 0, err, stream);
 }
 
 // Attention over keys and values that lie as rows of one matrix, one key and value per head
 // and position (a latent's, made for this step): `kv` bfloat16 [kv_rows, heads * (dk + dvp)], a
 // row's keys head by head, dk elements each, then its values, dvp each (dv of them used); position
 // p of sequence i is row seq_base[i] + p.  q [R, heads, dk], out [R, heads, dv].  dk: 64, 128 or
-// 192; dvp: 64 or 128, at most dk; dv a multiple of 16; scale > 0.
+// 192; dvp: 64 or 128, at most dk; dv a multiple of 16; scale > 0.  `gate_z` (or null): out[r, h, i]
+// is multiplied by sigmoid(gate_z[r, gate_col + h dv + i]); gate_ld and gate_col multiples of 8.
 extern "C" int rfx_attention_prefill_tc_rows(const void* q, const void* kv, long long kv_rows, const int* seq_base,
                                              const int* seq_slot, const int* seq_start, const int* seq_new,
                                              const int* seq_row0, void* out, int S, int max_new, int R, int heads,
                                              int dk, int dvp, int dv, int window, float scale, const float* sink,
-                                             int* err, void* stream) {
+                                             const void* gate_z, int gate_dt, int gate_ld, int gate_col, int* err,
+                                             void* stream) {
     if (S <= 0 || max_new <= 0 || R <= 0) return 0;
+    rfx::RowGate gate;
+    if (!rfx::row_gate(&gate, gate_z, gate_dt, gate_ld, gate_col, heads * dv)) return RFX_ERR_BAD_ARG;
+    // the logits come 16 bytes an access
+    if (gate_z && (gate_ld % 8 || gate_col % 8 || (reinterpret_cast<uintptr_t>(gate_z) & 15))) return RFX_ERR_UNSUPPORTED;
     if (!(scale > 0.0f) || dv <= 0 || dv % 16 || dv > dvp || heads <= 0 || kv_rows <= 0) return RFX_ERR_UNSUPPORTED;
     if ((reinterpret_cast<uintptr_t>(q) | reinterpret_cast<uintptr_t>(kv) | reinterpret_cast<uintptr_t>(out)) & 15)
         return RFX_ERR_BAD_ARG;
 #define RFX_CASE(A, B)                                                                                              \
     if (dk == A && dvp == B)                                                                                        \
         return launch_contig<A, B>(q, kv, kv_rows, seq_base, seq_slot, seq_start, seq_new, seq_row0, out, S,        \
-                                   max_new, R, heads, dv, window, scale, sink, err, (cudaStream_t)stream);
+                                   max_new, R, heads, dv, window, scale, sink, gate, err, (cudaStream_t)stream);
     RFX_CASE(64, 64) RFX_CASE(128, 64) RFX_CASE(128, 128) RFX_CASE(192, 64) RFX_CASE(192, 128)
 #undef RFX_CASE
     return RFX_ERR_UNSUPPORTED;

@@ -167,6 +167,23 @@ __device__ __forceinline__ float gated_mul_for(float g, float u) {
     else return silu_mul_for<TO>(g, u);
 }
 
+// A gate on a kernel's results: sigmoid(z[row, col + i]) for a row's element (or head) i, z the
+// rows of an earlier product, 32-bit or bfloat16.  Null z: no gate.
+struct RowGate {
+    const void* z;
+    int bf16, ld, col;
+    __device__ __forceinline__ float logit(size_t row, int i) const {
+        const size_t at = row * ld + col + i;
+        return bf16 ? __bfloat162float(reinterpret_cast<const __nv_bfloat16*>(z)[at]) : reinterpret_cast<const float*>(z)[at];
+    }
+    __device__ __forceinline__ float factor(size_t row, int i) const { return 1.0f / (1.0f + expf(-logit(row, i))); }
+};
+// whether the arguments of an entry point make one; `n` gate columns
+inline bool row_gate(RowGate* g, const void* z, int dt, int ld, int col, int n) {
+    *g = RowGate{z, dt == RFX_DT_BF16, ld, col};
+    return !z || ((dt == RFX_DT_BF16 || dt == RFX_DT_F32) && col >= 0 && col + n <= ld);
+}
+
 // Sum over the 32 lanes in a fixed butterfly order; every lane gets the total.
 __device__ __forceinline__ float warp_sum(float v) {
 #pragma unroll

@@ -9,9 +9,10 @@ namespace {
 using namespace rfx;
 
 // hidden[r, :] = table[ids[r], :] * scale       (src/model/dense.rs:1959-1967)
+// `rows` (or null): the same in the table's type, for a layer that reads the stream unnormed.
 template <typename T>
 __global__ void embed_kernel(const T* __restrict__ table, const int* __restrict__ ids,
-                             float* __restrict__ out, int H, int V, float scale,
+                             float* __restrict__ out, T* __restrict__ rows, int H, int V, float scale,
                              int* __restrict__ err) {
     // The first kernel of every step.  It does not let its dependents start
     // early: kernels of this step may read, before their own wait, cache pages
@@ -22,12 +23,18 @@ __global__ void embed_kernel(const T* __restrict__ table, const int* __restrict_
     const int id = ids[r];
     if (id < 0 || id >= V) {
         if (threadIdx.x == 0) atomicExch(err, 1 + r);
-        for (int c = threadIdx.x; c < H; c += blockDim.x) out[(size_t)r * H + c] = 0.0f;
+        for (int c = threadIdx.x; c < H; c += blockDim.x) {
+            out[(size_t)r * H + c] = 0.0f;
+            if (rows) st<T>(rows, (size_t)r * H + c, 0.0f);
+        }
         return;
     }
     const T* row = table + (size_t)id * H;
-    for (int c = threadIdx.x; c < H; c += blockDim.x)
-        out[(size_t)r * H + c] = ld<T>(row, c) * scale;
+    for (int c = threadIdx.x; c < H; c += blockDim.x) {
+        const float v = ld<T>(row, c) * scale;
+        out[(size_t)r * H + c] = v;
+        if (rows) st<T>(rows, (size_t)r * H + c, v);
+    }
 }
 
 // One block per output row.
@@ -197,15 +204,16 @@ int norm_threads(int H) {
 }  // namespace
 
 extern "C" int rfx_embed(const void* table, int table_dt, const int* ids, int R, int H, int V,
-                         float scale, float* out, int* err, void* stream) {
+                         float scale, float* out, void* rows, int* err, void* stream) {
     if (R <= 0) return 0;
     cudaStream_t s = (cudaStream_t)stream;
     const int threads = H >= 1024 ? 256 : 128;
     if (table_dt == RFX_DT_F32)
-        RFX_LAUNCH(embed_kernel<float>, R, threads, 0, s, (const float*)table, ids, out, H, V, scale, err);
+        RFX_LAUNCH(embed_kernel<float>, R, threads, 0, s, (const float*)table, ids, out, (float*)rows, H, V,
+                   scale, err);
     else if (table_dt == RFX_DT_BF16)
         RFX_LAUNCH(embed_kernel<__nv_bfloat16>, R, threads, 0, s, (const __nv_bfloat16*)table, ids, out,
-                   H, V, scale, err);
+                   (__nv_bfloat16*)rows, H, V, scale, err);
     else
         return RFX_ERR_BAD_ARG;
     return 0;

@@ -7,7 +7,8 @@
 //    cache at the row's position (one "head" of kv_rank elements a position),
 //    sigmoid of the per-head gates (32-bit).
 //  * rfx_heads_linear: y[r, b, :] = x[r, b, :] W_b^T for every head b, W
-//    [heads, N, K]; optionally times a per-(row, head) factor.  32-bit
+//    [heads, N, K]; optionally times a per-(row, head) factor, or an element's
+//    sigmoid gate.  32-bit
 //    accumulation, each output reduced over k in index order by one thread.
 #include "common.cuh"
 #include "paged.cuh"
@@ -63,7 +64,7 @@ constexpr int TM = 64, TN = 64, TK = 16;
 template <typename T, typename TO>
 __global__ void __launch_bounds__(256)
 heads_linear_kernel(const T* __restrict__ x, int ldx, int xh, const T* __restrict__ W, TO* __restrict__ y,
-                    int ldy, int yh, const float* __restrict__ scale, int R, int N, int K, int heads) {
+                    int ldy, int yh, const float* __restrict__ scale, RowGate gate, int R, int N, int K, int heads) {
     __shared__ float xs[TK][TM + 1];
     __shared__ float ws[TK][TN + 1];
     pdl_prologue();
@@ -109,7 +110,8 @@ heads_linear_kernel(const T* __restrict__ x, int ldx, int xh, const T* __restric
 #pragma unroll
         for (int j = 0; j < 4; ++j) {
             const int n = n0 + tx * 4 + j;
-            if (n < N) st<TO>(y + (size_t)r * ldy + (size_t)b * yh, n, acc[i][j] * f);
+            if (n < N)
+                st<TO>(y + (size_t)r * ldy + (size_t)b * yh, n, acc[i][j] * (gate.z ? gate.factor(r, b * N + n) : f));
         }
     }
 }
@@ -123,7 +125,7 @@ constexpr int GV_ROWS = 16;
 template <typename T, typename TO>
 __global__ void __launch_bounds__(256)
 heads_gemv_kernel(const T* __restrict__ x, int ldx, int xh, const T* __restrict__ W, TO* __restrict__ y, int ldy,
-                  int yh, const float* __restrict__ scale, int R, int N, int K, int heads) {
+                  int yh, const float* __restrict__ scale, RowGate gate, int R, int N, int K, int heads) {
     extern __shared__ __align__(16) float xs[];  // [R][K]
     pdl_prologue();
     const int b = blockIdx.x;
@@ -135,6 +137,7 @@ heads_gemv_kernel(const T* __restrict__ x, int ldx, int xh, const T* __restrict_
     const bool vec = sizeof(T) == 2 && (K & 7) == 0 && (reinterpret_cast<uintptr_t>(wb) & 15) == 0;
     for (int n = blockIdx.y * nwarps + warp; n < N; n += gridDim.y * nwarps) {
         const T* wrow = wb + (size_t)n * K;
+        const float gl = gate.z && lane < R ? gate.logit(lane, b * N + n) : 0.0f;  // row `lane`'s, on its way meanwhile
         float acc[GV_ROWS];
 #pragma unroll
         for (int r = 0; r < GV_ROWS; ++r) acc[r] = 0.0f;
@@ -165,11 +168,13 @@ heads_gemv_kernel(const T* __restrict__ x, int ldx, int xh, const T* __restrict_
                     if (r < R) acc[r] = fmaf(xs[r * K + c], w, acc[r]);
             }
         }
+        const float gf = 1.0f / (1.0f + expf(-gl));
 #pragma unroll
         for (int r = 0; r < GV_ROWS; ++r) {
             if (r >= R) break;
             const float v = warp_sum(acc[r]);
-            if (lane == 0) st<TO>(y + (size_t)r * ldy + (size_t)b * yh, n, v * (scale ? scale[(size_t)r * heads + b] : 1.0f));
+            const float f = gate.z ? __shfl_sync(0xffffffffu, gf, r) : scale ? scale[(size_t)r * heads + b] : 1.0f;
+            if (lane == 0) st<TO>(y + (size_t)r * ldy + (size_t)b * yh, n, v * f);
         }
     }
 }
@@ -206,10 +211,14 @@ extern "C" int rfx_latent_post(const void* proj, int in_dt, int ld, const float*
     return 0;
 }
 
+// `gate_z` (or null, not with `scale`): y[r, b, n] is multiplied by sigmoid(gate_z[r, gate_col + b N + n])
 extern "C" int rfx_heads_linear(const void* x, int ldx, int xh, const void* W, void* y, int ldy, int yh, int dt,
-                                const float* scale, int R, int N, int K, int heads, void* stream) {
+                                const float* scale, const void* gate_z, int gate_dt, int gate_ld, int gate_col, int R,
+                                int N, int K, int heads, void* stream) {
     if (R <= 0 || N <= 0 || heads <= 0) return 0;
-    if (K <= 0 || xh < K || yh < N) return RFX_ERR_BAD_ARG;
+    RowGate gate;
+    if (K <= 0 || xh < K || yh < N || (scale && gate_z) || !row_gate(&gate, gate_z, gate_dt, gate_ld, gate_col, heads * N))
+        return RFX_ERR_BAD_ARG;
     cudaStream_t s = (cudaStream_t)stream;
     if (R <= GV_ROWS && (size_t)R * K * sizeof(float) <= 48 * 1024) {
         // a few rows: every weight is read once and meets all rows
@@ -219,11 +228,11 @@ extern "C" int rfx_heads_linear(const void* x, int ldx, int xh, const void* W, v
         const size_t smem = (size_t)R * K * sizeof(float);
         if (dt == RFX_DT_F32)
             RFX_LAUNCH((heads_gemv_kernel<float, float>), g, 256, smem, s, (const float*)x, ldx, xh, (const float*)W,
-                       (float*)y, ldy, yh, scale, R, N, K, heads);
+                       (float*)y, ldy, yh, scale, gate, R, N, K, heads);
         else if (dt == RFX_DT_BF16)
             RFX_LAUNCH((heads_gemv_kernel<__nv_bfloat16, __nv_bfloat16>), g, 256, smem, s,
-                       (const __nv_bfloat16*)x, ldx, xh, (const __nv_bfloat16*)W, (__nv_bfloat16*)y, ldy, yh, scale, R, N,
-                       K, heads);
+                       (const __nv_bfloat16*)x, ldx, xh, (const __nv_bfloat16*)W, (__nv_bfloat16*)y, ldy, yh, scale, gate,
+                       R, N, K, heads);
         else
             return RFX_ERR_BAD_ARG;
         return 0;
@@ -232,10 +241,10 @@ extern "C" int rfx_heads_linear(const void* x, int ldx, int xh, const void* W, v
     if (grid.y > 65535 || grid.z > 65535) return RFX_ERR_UNSUPPORTED;
     if (dt == RFX_DT_F32)
         RFX_LAUNCH((heads_linear_kernel<float, float>), grid, 256, 0, s, (const float*)x, ldx, xh,
-                   (const float*)W, (float*)y, ldy, yh, scale, R, N, K, heads);
+                   (const float*)W, (float*)y, ldy, yh, scale, gate, R, N, K, heads);
     else if (dt == RFX_DT_BF16)
         RFX_LAUNCH((heads_linear_kernel<__nv_bfloat16, __nv_bfloat16>), grid, 256, 0, s,
-                   (const __nv_bfloat16*)x, ldx, xh, (const __nv_bfloat16*)W, (__nv_bfloat16*)y, ldy, yh, scale, R,
+                   (const __nv_bfloat16*)x, ldx, xh, (const __nv_bfloat16*)W, (__nv_bfloat16*)y, ldy, yh, scale, gate, R,
                    N, K, heads);
     else
         return RFX_ERR_BAD_ARG;

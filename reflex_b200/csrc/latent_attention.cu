@@ -23,10 +23,12 @@ latent_gather_kernel(const uint4* __restrict__ pages, const int* __restrict__ pa
     for (int i = 0; i < seq; ++i) base += seq_start[i] + seq_new[i];
     if (blockIdx.x == 0 && threadIdx.x == 0) seq_base[seq] = base;
     const int n = seq_start[seq] + seq_new[seq];
-    const int first = blockIdx.x * PAGE, count = min(PAGE, n - first);
+    // a block a quarter of a page
+    constexpr int PART = PAGE / 4;
+    const int first = blockIdx.x * PART, count = min(PART, n - first);
     if (count <= 0) return;
-    const int page = page_table[(size_t)seq_slot[seq] * max_pages + blockIdx.x];
-    const uint4* src = pages + (size_t)page * PAGE * w16;
+    const int page = page_table[(size_t)seq_slot[seq] * max_pages + blockIdx.x / 4];
+    const uint4* src = pages + ((size_t)page * PAGE + first % PAGE) * w16;
     uint4* dst = rows + (size_t)(base + first) * w16;
     for (int i = threadIdx.x; i < count * w16; i += blockDim.x) dst[i] = src[i];
 }
@@ -82,7 +84,7 @@ extern "C" int rfx_latent_gather(const void* pages, const int* page_table, int m
                                  int* seq_base, int S, int max_context, int width, void* stream) {
     if (S <= 0 || max_context <= 0) return 0;
     if (page_size != PAGE || width % 8 || S > 65535) return RFX_ERR_BAD_ARG;
-    dim3 grid((max_context + PAGE - 1) / PAGE, S);
+    dim3 grid((max_context + PAGE / 4 - 1) / (PAGE / 4), S);
     RFX_LAUNCH(latent_gather_kernel, grid, 256, 0, (cudaStream_t)stream, (const uint4*)pages, page_table, max_pages,
                seq_slot, seq_start, seq_new, (uint4*)rows, seq_base, width / 8);
     return 0;

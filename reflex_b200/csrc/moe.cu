@@ -31,16 +31,15 @@ using namespace rfx;
 
 constexpr int MAX_PER_LANE = 8;  // up to 256 experts
 
-__global__ void moe_route_kernel(const float* __restrict__ logits, int ld, const float* __restrict__ bias,
-                                 int* __restrict__ ids, float* __restrict__ wts, int R, int E, int top,
-                                 int mode, float scale, int groups, int keep) {
-    pdl_prologue();
+// One row's choice by one warp; PL: experts a lane holds (up to 32 PL in all).
+template <int PL>
+__device__ __forceinline__ void route_row(const float* __restrict__ logits, int ld, const float* __restrict__ bias,
+                                          int* __restrict__ ids, float* __restrict__ wts, int r, int E, int top,
+                                          int mode, float scale, int groups, int keep) {
     const int lane = threadIdx.x & 31;
-    const int r = blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
-    if (r >= R) return;
-    float z[MAX_PER_LANE];
+    float z[PL];
 #pragma unroll
-    for (int i = 0; i < MAX_PER_LANE; ++i) {
+    for (int i = 0; i < PL; ++i) {
         const int e = i * 32 + lane;
         z[i] = e < E ? logits[(size_t)r * ld + e] + (bias ? bias[e] : 0.0f) : -INFINITY;
     }
@@ -49,39 +48,39 @@ __global__ void moe_route_kernel(const float* __restrict__ logits, int ld, const
     if (mode >= 2) {
         float m = -INFINITY, s = 0.0f;
 #pragma unroll
-        for (int i = 0; i < MAX_PER_LANE; ++i) m = fmaxf(m, z[i]);
+        for (int i = 0; i < PL; ++i) m = fmaxf(m, z[i]);
         all_max = warp_max(m);
 #pragma unroll
-        for (int i = 0; i < MAX_PER_LANE; ++i)
+        for (int i = 0; i < PL; ++i)
             if (i * 32 + lane < E) s += expf(z[i] - all_max);
         all_sum = warp_sum(s);
     }
     if (keep < groups) {
         // a group's score is the largest in it; the best `keep` groups stay, ties to the lower index
         const int size = E / groups;
-        float best[MAX_PER_LANE];  // group g's best in lane g % 32
+        float best[PL];  // group g's best in lane g % 32
 #pragma unroll
-        for (int i = 0; i < MAX_PER_LANE; ++i) best[i] = -INFINITY;
+        for (int i = 0; i < PL; ++i) best[i] = -INFINITY;
         for (int g = 0; g < groups; ++g) {
             float m = -INFINITY;
 #pragma unroll
-            for (int i = 0; i < MAX_PER_LANE; ++i) {
+            for (int i = 0; i < PL; ++i) {
                 const int e = i * 32 + lane;
                 if (e >= g * size && e < (g + 1) * size) m = fmaxf(m, z[i]);
             }
             m = warp_max(m);
 #pragma unroll
-            for (int i = 0; i < MAX_PER_LANE; ++i)
+            for (int i = 0; i < PL; ++i)
                 if (i * 32 + lane == g) best[i] = m;
         }
-        unsigned kept[MAX_PER_LANE];  // a bit a group, the same in every lane
+        unsigned kept[PL];  // a bit a group, the same in every lane
 #pragma unroll
-        for (int i = 0; i < MAX_PER_LANE; ++i) kept[i] = 0;
+        for (int i = 0; i < PL; ++i) kept[i] = 0;
         for (int k = 0; k < keep; ++k) {
             float m = -INFINITY;
             int at = 0x7fffffff;
 #pragma unroll
-            for (int i = 0; i < MAX_PER_LANE; ++i) {
+            for (int i = 0; i < PL; ++i) {
                 const int g = i * 32 + lane;
                 if (g < groups && !(kept[i] >> lane & 1) && (at == 0x7fffffff || best[i] > m)) { m = best[i]; at = g; }
             }
@@ -92,15 +91,15 @@ __global__ void moe_route_kernel(const float* __restrict__ logits, int ld, const
                 if (oa != 0x7fffffff && (at == 0x7fffffff || om > m || (om == m && oa < at))) { m = om; at = oa; }
             }
 #pragma unroll
-            for (int i = 0; i < MAX_PER_LANE; ++i)
+            for (int i = 0; i < PL; ++i)
                 if (at / 32 == i) kept[i] |= 1u << (at & 31);
         }
 #pragma unroll
-        for (int i = 0; i < MAX_PER_LANE; ++i) {
+        for (int i = 0; i < PL; ++i) {
             const int g = min((i * 32 + lane) / size, groups - 1);
             unsigned word = 0;
 #pragma unroll
-            for (int j = 0; j < MAX_PER_LANE; ++j)
+            for (int j = 0; j < PL; ++j)
                 if (j == g / 32) word = kept[j];
             if (!(word >> (g & 31) & 1)) z[i] = -INFINITY;
         }
@@ -111,7 +110,7 @@ __global__ void moe_route_kernel(const float* __restrict__ logits, int ld, const
         float best = -INFINITY;
         int best_e = 0x7fffffff;
 #pragma unroll
-        for (int i = 0; i < MAX_PER_LANE; ++i) {
+        for (int i = 0; i < PL; ++i) {
             const int e = i * 32 + lane;
             if (z[i] > best) { best = z[i]; best_e = e; }  // within a lane e rises: the lower index wins a tie
         }
@@ -132,7 +131,7 @@ __global__ void moe_route_kernel(const float* __restrict__ logits, int ld, const
             wts[(size_t)r * top + k] = p;
         }
 #pragma unroll
-        for (int i = 0; i < MAX_PER_LANE; ++i)
+        for (int i = 0; i < PL; ++i)
             if (i * 32 + lane == best_e) z[i] = -INFINITY;
     }
     if (mode >= 2) {
@@ -152,6 +151,51 @@ __global__ void moe_route_kernel(const float* __restrict__ logits, int ld, const
     }
     if (lane == 0)
         for (int k = 32; k < top; ++k) wts[(size_t)r * top + k] = wts[(size_t)r * top + k] / sum * scale;
+}
+
+template <int PL>
+__global__ void __launch_bounds__(128)
+moe_route_kernel(const float* __restrict__ logits, int ld, const float* __restrict__ bias, int* __restrict__ ids,
+                 float* __restrict__ wts, int R, int E, int top, int mode, float scale, int groups, int keep) {
+    pdl_prologue();
+    const int r = blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
+    if (r < R) route_row<PL>(logits, ld, bias, ids, wts, r, E, top, mode, scale, groups, keep);
+}
+
+// Counts per expert, offsets (exclusive prefix, [E + 1]) and each pair's place in the
+// expert-by-expert order, by one block; `cnt`: 2 E ints of shared memory, counts and cursors.
+__device__ __forceinline__ void place_pairs(const int* ids, int n_pairs, int E, int* __restrict__ offsets,
+                                            int* __restrict__ place, int* cnt) {
+    int* cursor = cnt + E;
+    for (int e = threadIdx.x; e < E; e += blockDim.x) cnt[e] = 0;
+    __syncthreads();
+    for (int p = threadIdx.x; p < n_pairs; p += blockDim.x) atomicAdd(&cnt[ids[p]], 1);
+    __syncthreads();
+    if (threadIdx.x == 0) {
+        int run = 0;
+        for (int e = 0; e < E; ++e) {
+            offsets[e] = run;
+            cursor[e] = run;
+            run += cnt[e];
+        }
+        offsets[E] = run;
+    }
+    __syncthreads();
+    for (int p = threadIdx.x; p < n_pairs; p += blockDim.x) place[p] = atomicAdd(&cursor[ids[p]], 1);
+}
+
+// A few rows (decode): the choice and the pairs' places in one launch, a warp a row.
+template <int PL>
+__global__ void __launch_bounds__(1024)
+moe_route_place_kernel(const float* __restrict__ logits, int ld, const float* __restrict__ bias, int* ids,
+                       float* __restrict__ wts, int R, int E, int top, int mode, float scale, int groups, int keep,
+                       int* __restrict__ offsets, int* __restrict__ place) {
+    extern __shared__ int cnt[];
+    pdl_prologue();
+    for (int r = threadIdx.x >> 5; r < R; r += blockDim.x >> 5)
+        route_row<PL>(logits, ld, bias, ids, wts, r, E, top, mode, scale, groups, keep);
+    __syncthreads();
+    place_pairs(ids, R * top, E, offsets, place, cnt);
 }
 
 // sum_c xs[c] * w[c] over a warp; bfloat16 rows that start on 16 bytes go eight
@@ -259,30 +303,14 @@ moe_down_kernel(const T* __restrict__ act, const T* __restrict__ W, const int* _
     }
 }
 
-// One block: counts per expert, offsets (exclusive prefix, [E + 1]) and each
-// pair's place in the expert-by-expert order.  Places within an expert are
-// handed out as the threads arrive; a pair's result does not depend on its place.
+// Places within an expert are handed out as the threads arrive; a pair's result does not
+// depend on its place.
 __global__ void __launch_bounds__(1024)
 moe_group_kernel(const int* __restrict__ ids, int n_pairs, int E, int* __restrict__ offsets,
                  int* __restrict__ place) {
     extern __shared__ int cnt[];  // [E] counts, then [E] cursors
-    int* cursor = cnt + E;
     pdl_prologue();
-    for (int e = threadIdx.x; e < E; e += blockDim.x) cnt[e] = 0;
-    __syncthreads();
-    for (int p = threadIdx.x; p < n_pairs; p += blockDim.x) atomicAdd(&cnt[ids[p]], 1);
-    __syncthreads();
-    if (threadIdx.x == 0) {
-        int run = 0;
-        for (int e = 0; e < E; ++e) {
-            offsets[e] = run;
-            cursor[e] = run;
-            run += cnt[e];
-        }
-        offsets[E] = run;
-    }
-    __syncthreads();
-    for (int p = threadIdx.x; p < n_pairs; p += blockDim.x) place[p] = atomicAdd(&cursor[ids[p]], 1);
+    place_pairs(ids, n_pairs, E, offsets, place, cnt);
 }
 
 // xg[place[p], :] = x[p / top, :] (times scale[p], when given)
@@ -448,21 +476,38 @@ extern "C" int rfx_moe_combine(const void* yg, int dt, const int* place, const f
 // modes 2, 3: the softmax over all experts, the chosen ones' scores over their sum (+ 1e-20) or as
 // they are; `scale` multiplies the weights of every mode; of `groups` equal groups of neighbours
 // only the experts of the `keep` ones with the largest logit can be chosen
+// `offsets` [E + 1] and `place` [R top] (or both null; up to 64 rows): the pairs' places too, as
+// rfx_moe_group gives them.
 extern "C" int rfx_moe_route_groups(const float* logits, int ld, const float* bias, int* ids, float* wts, int R,
-                                    int E, int top, int mode, float scale, int groups, int keep, void* stream) {
+                                    int E, int top, int mode, float scale, int groups, int keep, int* offsets,
+                                    int* place, void* stream) {
     if (R <= 0) return 0;
-    if (E <= 0 || top <= 0 || top > E || ld < E || mode < 0 || mode > 3) return RFX_ERR_BAD_ARG;
+    if (E <= 0 || top <= 0 || top > E || ld < E || mode < 0 || mode > 3 || !offsets != !place) return RFX_ERR_BAD_ARG;
     if (groups <= 0 || E % groups || keep <= 0 || keep > groups || top > keep * (E / groups)) return RFX_ERR_BAD_ARG;
-    if (E > 32 * MAX_PER_LANE) return RFX_ERR_UNSUPPORTED;
-    RFX_LAUNCH(moe_route_kernel, (R + 3) / 4, 128, 0, (cudaStream_t)stream, logits, ld, bias, ids, wts, R, E, top,
-               mode, scale, groups, keep);
+    if (E > 32 * MAX_PER_LANE || (place && R > 64)) return RFX_ERR_UNSUPPORTED;
+    cudaStream_t s = (cudaStream_t)stream;
+#define RFX_GO(PL)                                                                                                     \
+    do {                                                                                                               \
+        if (place)                                                                                                     \
+            RFX_LAUNCH(moe_route_place_kernel<PL>, 1, R >= 32 ? 1024 : 32 * R < 128 ? 128 : 32 * R,                    \
+                       (size_t)2 * E * sizeof(int), s, logits, ld, bias, ids, wts, R, E, top, mode, scale, groups,     \
+                       keep, offsets, place);                                                                          \
+        else                                                                                                           \
+            RFX_LAUNCH(moe_route_kernel<PL>, (R + 3) / 4, 128, 0, s, logits, ld, bias, ids, wts, R, E, top, mode,      \
+                       scale, groups, keep);                                                                           \
+    } while (0)
+    if (E <= 32) RFX_GO(1);
+    else if (E <= 64) RFX_GO(2);
+    else if (E <= 128) RFX_GO(4);
+    else RFX_GO(8);
+#undef RFX_GO
     return 0;
 }
 
 extern "C" int rfx_moe_route(const float* logits, int ld, const float* bias, int* ids, float* wts, int R, int E,
                              int top, int mode, void* stream) {
     if (mode != 0 && mode != 1) return RFX_ERR_BAD_ARG;
-    return rfx_moe_route_groups(logits, ld, bias, ids, wts, R, E, top, mode, 1.0f, 1, 1, stream);
+    return rfx_moe_route_groups(logits, ld, bias, ids, wts, R, E, top, mode, 1.0f, 1, 1, nullptr, nullptr, stream);
 }
 
 extern "C" int rfx_moe_up(const void* x, const void* W, const int* ids, const float* in_scale, void* act, int dt,

@@ -15,14 +15,16 @@
 //    latent over its root mean square and times a weight goes out (for the query
 //    up-projection); the latent, likewise, and the turned key part go into the page of the
 //    row's position as one row [latent | key part | zeros].
+//  * rfx_rotate_tails: the last `rot` elements of every head turn where they stand.
 //  * rfx_latent_rot_post: rows [q | latent | shared key part]: per head the unrotated
 //    part of q and the turned rotated part with zeros behind it go to places of the caller's
 //    (apart, where the product with W_uk follows; side by side as one query); the latent, over its root
 //    mean square and times a weight, and the turned key part go into the page of the
 //    row's position as one row [latent | key part | zeros].
 //
-// A warp a head of a row; everything is 32-bit; sine and cosine come from
-// `exact_sincosf`, once a row and block into shared memory.
+// A warp a head of a row; everything is 32-bit; sine and cosine are taken once a row and
+// block into shared memory, by `exact_sincosf` (whose range reduction runs in double precision,
+// at a small fraction of this GPU's 32-bit rate) for 32-bit results, by sincosf for rounded ones.
 #include "common.cuh"
 #include "exact_math.cuh"
 #include "paged.cuh"
@@ -35,10 +37,12 @@ constexpr int RP_THREADS = 256;
 constexpr int RP_WARPS = RP_THREADS / 32;
 
 // cos and sin of a row's angles into cs[0 .. half) and cs[half .. 2 half)
+template <typename TO>
 __device__ __forceinline__ void angles(float* cs, const float* denom, int half, int pos, float magnitude = 1.0f) {
     for (int i = threadIdx.x; i < half; i += blockDim.x) {
         float s, c;
-        exact_sincosf((float)pos / denom[i], &s, &c);
+        if constexpr (sizeof(TO) == 2) sincosf((float)pos / denom[i], &s, &c);
+        else exact_sincosf((float)pos / denom[i], &s, &c);
         cs[i] = c * magnitude;
         cs[half + i] = s * magnitude;
     }
@@ -78,7 +82,7 @@ rot_qkv_post_kernel(const TI* __restrict__ proj, int ldp, QkvPost a, const int* 
     const int r = blockIdx.x;
     const int pos = row_pos[r], slot = row_slot[r];
     const int half = a.rot_dims / 2;
-    angles(cs, a.denom, half, pos, a.magnitude);
+    angles<TO>(cs, a.denom, half, pos, a.magnitude);
     const int lane = threadIdx.x & 31;
     const int units = a.nq + (a.writes_cache ? 2 * a.nkv : 0);
     for (int u = blockIdx.y * RP_WARPS + (threadIdx.x >> 5); u < units; u += gridDim.y * RP_WARPS) {
@@ -241,7 +245,7 @@ latent_rot_post_kernel(const TI* __restrict__ proj, int ldp, const float* __rest
     const int r = blockIdx.x;
     const int pos = row_pos[r], slot = row_slot[r];
     const int half = rot / 2;
-    angles(cs, denom, half, pos);
+    angles<TO>(cs, denom, half, pos);
     const int lane = threadIdx.x & 31;
     const TI* row = proj + (size_t)r * ldp;
     auto turn_into = [&](TO* dst, const TI* x, int n) {  // the rotated part and the zeros behind it
@@ -304,7 +308,7 @@ latent_low_post_kernel(const TI* __restrict__ proj, int ldp, const float* __rest
     pdl_launch_dependents();
     if (cached) {  // positions are the step's inputs: none of this waits for the kernel before
         const int pos = row_pos[r];
-        angles(cs, denom, half, pos);
+        angles<TO>(cs, denom, half, pos);
         dst = pages + kv_offset(cache, row_slot[r], pos, 0);
     }
     pdl_wait();
@@ -335,6 +339,27 @@ latent_low_post_kernel(const TI* __restrict__ proj, int ldp, const float* __rest
     for (int e = threadIdx.x; e < width - rank; e += blockDim.x)
         st<TO>(dst + rank, e,
                e < rot ? turned(ld<TI>(x, e), ld<TI>(x, e < half ? e + half : e - half), e, cs, half) : 0.0f);
+}
+
+// x [R, H, n]: of every head the last `rot` elements, half-split pairs, in place; a thread two
+// neighbouring pairs (rot a multiple of 4)
+template <typename T>
+__global__ void __launch_bounds__(RP_THREADS)
+rotate_tails_kernel(T* __restrict__ x, const float* __restrict__ denom, const int* __restrict__ row_pos, int H, int n,
+                    int rot) {
+    extern __shared__ float cs[];
+    pdl_launch_dependents();
+    const int r = blockIdx.x, half = rot / 2, quads = half / 2;
+    angles<T>(cs, denom, half, row_pos[r]);  // positions are the step's inputs
+    pdl_wait();
+    T* row = x + (size_t)r * H * n + (n - rot);
+    for (int u = threadIdx.x; u < H * quads; u += blockDim.x) {
+        const int i = 2 * (u % quads);
+        T* p = row + (size_t)(u / quads) * n + i;
+        const float a0 = ld<T>(p, 0), a1 = ld<T>(p, 1), b0 = ld<T>(p, half), b1 = ld<T>(p, half + 1);
+        store2(p, fmaf(b0, -cs[half + i], __fmul_rn(a0, cs[i])), fmaf(b1, -cs[half + i + 1], __fmul_rn(a1, cs[i + 1])));
+        store2(p + half, fmaf(a0, cs[half + i], __fmul_rn(b0, cs[i])), fmaf(a1, cs[half + i + 1], __fmul_rn(b1, cs[i + 1])));
+    }
 }
 
 // blocks of a row: few rows spread their heads over blocks, many rows keep a row's angles in one
@@ -455,5 +480,19 @@ extern "C" int rfx_latent_low_post(const void* proj, int in_dt, int ld, const fl
     else return RFX_ERR_BAD_ARG;
 #undef RFX_GO
 #undef RFX_N
+    return 0;
+}
+
+// x [R, H, n], n - rot and rot / 2 even
+extern "C" int rfx_rotate_tails(void* x, int dt, const float* denom, const int* row_pos, int R, int H, int n, int rot,
+                                void* stream) {
+    if (R <= 0 || H <= 0) return 0;
+    if (rot <= 0 || rot > n || rot % 4 || n % 2 || !aligned(x, 8)) return RFX_ERR_BAD_ARG;
+    cudaStream_t s = (cudaStream_t)stream;
+    const size_t smem = (size_t)rot * sizeof(float);
+    if (dt == RFX_DT_F32) RFX_LAUNCH(rotate_tails_kernel<float>, R, RP_THREADS, smem, s, (float*)x, denom, row_pos, H, n, rot);
+    else if (dt == RFX_DT_BF16)
+        RFX_LAUNCH(rotate_tails_kernel<__nv_bfloat16>, R, RP_THREADS, smem, s, (__nv_bfloat16*)x, denom, row_pos, H, n, rot);
+    else return RFX_ERR_BAD_ARG;
     return 0;
 }

@@ -160,15 +160,22 @@ class CausalLM:
         keeps the residual in a form of its own makes the ordinary one at the end,
         and then only for the rows that are wanted)."""
         ops.prof_mark("start")
+        # a first block that reads the stream itself gets its rows ready
+        first = self.spec.run_order[0]
+        reads = (isinstance(self.layers[first.layer], PostNormBlock) and not self.embedding_terms
+                 and not first.mixes_input and first.pass_vector is None)
+        plain = reads and self.embedding_norm is None
         # a token id outside the vocabulary (possible only for ids fed from the device)
         # gives a zero row and sets the device's error word, which `check_errors` reads
         h = ops.embed(self.embedding, batch.tokens, self.spec.embedding_scale,
-                      ops.device_error_word(self.device))
+                      ops.device_error_word(self.device), with_rows=plain)
         pending = None
+        if plain:
+            h, x = h
+            pending = ReadyRows(x)
         if self.embedding_norm is not None:
-            # the stream starts normed; a first block that reads the stream itself gets its rows too
-            n, first = self.embedding_norm, self.layers[self.spec.run_order[0].layer]
-            reads = isinstance(first, PostNormBlock) and not self.embedding_terms
+            # the stream starts normed
+            n = self.embedding_norm
             x = ops.post_norm(h, h, n.weight, n.spec.weight_offset, n.spec.eps, self.dtype if reads else None, fresh=True)
             pending = ReadyRows(x) if x is not None else None
         for ti, term in enumerate(self.embedding_terms):

@@ -52,16 +52,19 @@ def _chk(t: Optional[torch.Tensor], name: str, dtype=None) -> int:
 
 
 # ---------------------------------------------------------------- elementwise
-def embed(table: torch.Tensor, ids: torch.Tensor, scale: float, err_flag: torch.Tensor) -> torch.Tensor:
-    """hidden[r] = table[ids[r]] * scale, as float32 [R, H]."""
+def embed(table: torch.Tensor, ids: torch.Tensor, scale: float, err_flag: torch.Tensor, with_rows: bool = False):
+    """hidden[r] = table[ids[r]] * scale, as float32 [R, H]; `with_rows`: (hidden, the same
+    in the table's type), for a first layer that reads the stream unnormed."""
     V, H = table.shape
     R = ids.numel()
     out = _new((R, H), torch.float32, table.device, keep=True)  # the residual stream: lives for the whole step
+    rows = _new((R, H), table.dtype, table.device) if with_rows else None
     st = native.lib().rfx_embed(
         _chk(table, "table"), dt_code(table.dtype), _chk(ids, "ids", torch.int32), R, H, V,
-        float(scale), out.data_ptr(), _chk(err_flag, "err_flag", torch.int32), _stream())
+        float(scale), out.data_ptr(), rows.data_ptr() if with_rows else 0, _chk(err_flag, "err_flag", torch.int32),
+        _stream())
     native.check(st, "embed")
-    return out
+    return (out, rows) if with_rows else out
 
 
 def rmsnorm(x: torch.Tensor, weight: torch.Tensor, eps: float, out_dtype: torch.dtype,
@@ -584,13 +587,24 @@ def decode_splits(n_rows: int, nq: int, nkv: int, max_pages: int = 64) -> int:
     return best
 
 
+def _gate_args(gate, rows: int):
+    """The entry points' gate arguments of `gate` = (rows of a product, first column) or None."""
+    if gate is None:
+        return 0, 0, 0, 0
+    z, col = gate
+    if z.shape[0] != rows:
+        raise InvalidInput("the gate's rows do not match")
+    return _chk(z, "gate"), dt_code(z.dtype), z.shape[1], int(col)
+
+
 def attention_decode(q, k_pages, v_pages, page_table, page_size, row_pos, row_slot, nq, nkv,
                      head_dim, window, scale, n_splits: Optional[int] = None,
                      sink: Optional[torch.Tensor] = None,
                      slopes: Optional[torch.Tensor] = None, keep_first: int = 0,
-                     softcap: float = 0.0) -> torch.Tensor:
+                     softcap: float = 0.0, gate=None) -> torch.Tensor:
     """bfloat16 tensor-core attention for rows that are each one query
-    position (decode), split over the keys."""
+    position (decode), split over the keys.  `gate` = (rows, first column): head h's
+    output is multiplied by sigmoid(rows[r, column + h])."""
     keep_first = int(keep_first) if window else 0
     R = q.shape[0]
     _chk(q, "q", torch.bfloat16)
@@ -609,7 +623,7 @@ def attention_decode(q, k_pages, v_pages, page_table, page_size, row_pos, row_sl
             _chk(row_pos, "row_pos", torch.int32), _chk(row_slot, "row_slot", torch.int32), out.data_ptr(), 0,
             R, nq, nkv, head_dim, n_splits, int(window or 0), keep_first, float(scale),
             _chk(sink, "sink", torch.float32), _chk(slopes, "slopes", torch.float32), float(softcap), pool_pages, 1,
-            device_error_word(q.device).data_ptr(), _stream())
+            *_gate_args(gate, R), device_error_word(q.device).data_ptr(), _stream())
         if st != native.ERR_UNSUPPORTED:
             native.check(st, f"attention_decode_cluster (head_dim={head_dim}, splits={n_splits})")
             return out
@@ -620,7 +634,8 @@ def attention_decode(q, k_pages, v_pages, page_table, page_size, row_pos, row_sl
         _chk(row_pos, "row_pos", torch.int32), _chk(row_slot, "row_slot", torch.int32), out.data_ptr(),
         partial.data_ptr() if partial is not None else 0, R, nq, nkv, head_dim, n_splits,
         int(window or 0), keep_first, float(scale), _chk(sink, "sink", torch.float32),
-        _chk(slopes, "slopes", torch.float32), float(softcap), pool_pages, 0, device_error_word(q.device).data_ptr(), _stream())
+        _chk(slopes, "slopes", torch.float32), float(softcap), pool_pages, 0, *_gate_args(gate, R),
+        device_error_word(q.device).data_ptr(), _stream())
     native.check(st, f"attention_decode (head_dim={head_dim}, splits={n_splits})")
     return out
 
@@ -654,11 +669,11 @@ def attention_prefill(q, k_pages, v_pages, page_table, page_size, seq_slot, seq_
 def attention_prefill_tc(q, k_pages, v_pages, page_table, page_size, seq_slot, seq_start, seq_new,
                          seq_row0, max_new: int, nq, nkv, head_dim, window, scale, sink=None,
                          slopes=None, keep_first: int = 0, softcap: float = 0.0,
-                         score_bound: float = 0.0) -> torch.Tensor:
+                         score_bound: float = 0.0, gate=None) -> torch.Tensor:
     """The tcgen05/TMEM form of `attention_prefill`, for head sizes 64 and 128
     (the scale must be positive).  `score_bound` > 0: no scaled score is larger
     (queries and keys of known length); with a cap twice that, its tanh is a
-    polynomial."""
+    polynomial.  `gate` as in `attention_decode`."""
     _chk(q, "q", torch.bfloat16)
     if head_dim not in (64, 128):
         raise InvalidInput(f"attention_prefill_tc takes head_dim 64 or 128, got {head_dim}")
@@ -673,13 +688,13 @@ def attention_prefill_tc(q, k_pages, v_pages, page_table, page_size, seq_slot, s
         seq_slot.numel(), int(max_new), q.shape[0], nq, nkv, head_dim, int(window or 0),
         int(keep_first) if window else 0, float(scale),
         _chk(sink, "sink", torch.float32), _chk(slopes, "slopes", torch.float32), float(softcap), float(score_bound),
-        device_error_word(q.device).data_ptr(), _stream())
+        *_gate_args(gate, q.shape[0]), device_error_word(q.device).data_ptr(), _stream())
     native.check(st, f"attention_prefill_tc (head_dim={head_dim})")
     return out
 
 
 def attention(q, k_pages, v_pages, page_table, page_size, batch, nq, nkv, head_dim, window, scale,
-              sink=None, slopes=None, keep_first: int = 0, softcap: float = 0.0, score_bound: float = 0.0):
+              sink=None, slopes=None, keep_first: int = 0, softcap: float = 0.0, score_bound: float = 0.0, gate=None):
     """Attention of the step's rows over their sequences' cached keys and
     values; picks the kernel for the dtype and the kind of step.  `sink`: one
     float32 per query head whose exponential joins the softmax's denominator.
@@ -687,7 +702,8 @@ def attention(q, k_pages, v_pages, page_table, page_size, batch, nq, nkv, head_d
     position) is taken off every score.  `keep_first`: with a window, the first
     so many positions of a sequence stay visible beyond it.  `softcap` > 0: a score
     s becomes softcap * tanh(s / softcap) before the softmax; `score_bound` > 0: the
-    caller knows that no |s| is larger."""
+    caller knows that no |s| is larger.  `gate` = (rows of a product, first column): head
+    h's output is multiplied by sigmoid(rows[r, column + h])."""
     fast = q.dtype == torch.bfloat16 and head_dim % 16 == 0 and head_dim <= 256
     keep_first = int(keep_first) if window else 0
     if fast and batch.is_decode:
@@ -696,17 +712,19 @@ def attention(q, k_pages, v_pages, page_table, page_size, batch, nq, nkv, head_d
         return attention_decode(q, k_pages, v_pages, page_table, page_size, batch.row_pos,
                                 batch.row_slot, nq, nkv, head_dim, window, scale,
                                 n_splits=decode_splits(q.shape[0], nq, nkv, pages), sink=sink, slopes=slopes,
-                                keep_first=keep_first, softcap=softcap)
+                                keep_first=keep_first, softcap=softcap, gate=gate)
     if fast and nq // nkv <= 128 and head_dim in (64, 128) and scale > 0:
         return attention_prefill_tc(q, k_pages, v_pages, page_table, page_size, batch.seq_slot,
                                     batch.seq_start, batch.seq_new, batch.seq_row0, batch.max_new, nq,
-                                    nkv, head_dim, window, scale, sink, slopes, keep_first, softcap, score_bound)
+                                    nkv, head_dim, window, scale, sink, slopes, keep_first, softcap, score_bound, gate)
     if fast and nq // nkv <= 128:
-        return attention_prefill(q, k_pages, v_pages, page_table, page_size, batch.seq_slot,
+        out = attention_prefill(q, k_pages, v_pages, page_table, page_size, batch.seq_slot,
                                  batch.seq_start, batch.seq_new, batch.seq_row0, batch.max_new, nq,
                                  nkv, head_dim, window, scale, sink, slopes, keep_first, softcap)
-    return attention_plain(q, k_pages, v_pages, page_table, page_size, batch.row_pos,
-                           batch.row_slot, nq, nkv, head_dim, window, scale, sink, slopes, keep_first, softcap)
+    else:
+        out = attention_plain(q, k_pages, v_pages, page_table, page_size, batch.row_pos,
+                              batch.row_slot, nq, nkv, head_dim, window, scale, sink, slopes, keep_first, softcap)
+    return out if gate is None else sigmoid_gate_mul_(out, gate[0], gate[1], heads=nq)
 
 
 # ------------------------------------------------- further norms and embedding terms
@@ -785,10 +803,12 @@ HEADS_LINEAR_MAX_ROWS = _env_int("REFLEX_B200_HEADS_LINEAR_MAX_ROWS", 64, 0, 1 <
 
 
 def heads_linear(x: torch.Tensor, weight: torch.Tensor, scale: Optional[torch.Tensor] = None,
-                 out_dtype: Optional[torch.dtype] = None, out: Optional[torch.Tensor] = None) -> torch.Tensor:
+                 out_dtype: Optional[torch.dtype] = None, out: Optional[torch.Tensor] = None,
+                 gate=None) -> torch.Tensor:
     """y[r, b, :] = x[r, b, :K] @ weight[b].T for every head b: x [R, heads * xh] with
     xh >= K elements a head (the first K are read), weight [heads, N, K], y [R, heads
-    * N]; with `scale` (float32 [R, heads]) y[r, b, :] is multiplied by scale[r, b].
+    * N]; with `scale` (float32 [R, heads]) y[r, b, :] is multiplied by scale[r, b]; with
+    `gate` = (rows of a product, first column) y[r, b, n] by sigmoid(rows[r, column + b N + n]).
     `out` [R, heads * yh], yh >= N: the results go into the first N elements of each of
     its heads.  float32 and a few bfloat16 rows: this library's kernel (32-bit
     accumulation in index order); more bfloat16 rows: the library's batched product,
@@ -821,10 +841,10 @@ def heads_linear(x: torch.Tensor, weight: torch.Tensor, scale: Optional[torch.Te
             st = native.lib().rfx_scale_heads(y.data_ptr(), dt_code(y.dtype), _chk(scale, "scale", torch.float32),
                                               y.numel(), N, _stream())
             native.check(st, "scale_heads")
-        return y
+        return y if gate is None else sigmoid_gate_mul_(y, gate[0], gate[1])
     st = native.lib().rfx_heads_linear(x.data_ptr(), heads * xh, xh, weight.data_ptr(), y.data_ptr(), heads * yh, yh,
-                                       dt_code(x.dtype), _chk(scale, "scale", torch.float32), R, N, K, heads,
-                                       _stream())
+                                       dt_code(x.dtype), _chk(scale, "scale", torch.float32), *_gate_args(gate, R), R, N,
+                                       K, heads, _stream())
     native.check(st, f"heads_linear (heads={heads}, N={N}, K={K})")
     return y
 
@@ -890,7 +910,7 @@ MOE_SCORES = {"softmax_top": 0, "sigmoid": 1, "softmax_all": 2, "softmax": 3}
 
 
 def moe_route(logits: torch.Tensor, bias: Optional[torch.Tensor], top: int, experts: Optional[int] = None,
-              scores: str = "softmax_top", col0: int = 0, scale: float = 1.0, groups=None):
+              scores: str = "softmax_top", col0: int = 0, scale: float = 1.0, groups=None, place: bool = False):
     """Router logits float32 [R, experts] (+ bias) -> ids int32 [R, top], the
     experts with the largest logits, and weights float32 [R, top]: the softmax
     over the chosen logits only ("softmax_top"), or each chosen logit's sigmoid
@@ -899,7 +919,9 @@ def moe_route(logits: torch.Tensor, bias: Optional[torch.Tensor], top: int, expe
     `scale` multiplies the weights.  `groups` = (count, keep): of `count` equal groups of
     neighbours only the `keep` ones with the largest best logit can be chosen from.  With `experts` only that many columns of `logits`,
     from column `col0` on, are router logits (the rest belongs to the caller: a
-    product stacked with others')."""
+    product stacked with others').  `place`: (ids, weights, placed) comes back, `placed`
+    what `moe_experts` takes: the pairs' places expert by expert, made in the same launch
+    (up to MOE_PLACE_MAX_ROWS rows)."""
     R, ld = logits.shape
     E = ld if experts is None else int(experts)
     if not (0 <= col0 <= ld - E):
@@ -909,11 +931,18 @@ def moe_route(logits: torch.Tensor, bias: Optional[torch.Tensor], top: int, expe
     count, keep = (int(g) for g in groups) if groups else (1, 1)
     if count <= 0 or E % count or not (0 < keep <= count) or top > keep * (E // count):
         raise InvalidInput("moe_route: the groups must divide the experts and the kept ones hold the chosen")
+    if place:
+        offsets = _new((E + 1,), torch.int32, logits.device)
+        at = _new((R * top,), torch.int32, logits.device)
     st = native.lib().rfx_moe_route_groups(_chk(logits, "logits", torch.float32) + 4 * int(col0), ld,
                                            _chk(bias, "bias", torch.float32), ids.data_ptr(), wts.data_ptr(), R, E,
-                                           int(top), MOE_SCORES[scores], float(scale), count, keep, _stream())
+                                           int(top), MOE_SCORES[scores], float(scale), count, keep,
+                                           offsets.data_ptr() if place else 0, at.data_ptr() if place else 0, _stream())
     native.check(st, f"moe_route (experts={E}, top={top})")
-    return ids, wts
+    return (ids, wts, (offsets, at)) if place else (ids, wts)
+
+
+MOE_PLACE_MAX_ROWS = 64  # one block chooses for that many rows and places their pairs
 
 
 class ExpertRows:
@@ -934,7 +963,7 @@ class ExpertRows:
 
 def moe_experts(x: torch.Tensor, up: torch.Tensor, down: torch.Tensor, ids: torch.Tensor,
                 wts: torch.Tensor, activation: str = "relu2", weight_input: bool = False,
-                alpha: float = 1.0, limit: float = 0.0, leave_sum: bool = False):
+                alpha: float = 1.0, limit: float = 0.0, leave_sum: bool = False, placed=None):
     """sum_k wts[r, k] down[e] act(up[e] x[r]), e = ids[r, k]; up [experts, ff,
     width], down [experts, width, ff]; float32 [R, width].  Every (row, choice)
     reads its expert's matrices itself: the form for a few rows, and the exact
@@ -943,7 +972,7 @@ def moe_experts(x: torch.Tensor, up: torch.Tensor, down: torch.Tensor, ids: torc
     `alpha` and `limit` (`glu_clamped`); "swiglu": the same layout, silu(gate) * up.  `weight_input`: the weight multiplies
     the expert's input instead of its output, sum_k down[e] act(up[e] (wts[r, k]
     x[r])).  `leave_sum`: the grouped form may hand back the experts' rows (`ExpertRows`)
-    in place of their sum."""
+    in place of their sum.  `placed`: from `moe_route`, where it made the places too."""
     R, width = x.shape
     E, ff, _w = up.shape
     gated = activation in ("glu_clamped", "swiglu")
@@ -951,10 +980,10 @@ def moe_experts(x: torch.Tensor, up: torch.Tensor, down: torch.Tensor, ids: torc
         ff //= 2
     top = ids.shape[1]
     in_scale, out_wts = (wts, None) if weight_input else (None, wts)
-    if x.dtype == torch.bfloat16 and MOE_GROUPED and R >= MOE_GROUPED_MIN_ROWS:
+    if moe_grouped(x):
         # captured steps too, as long as the library's grouped product (no wait for the host) is there
         if not torch.cuda.is_current_stream_capturing() or (_GROUPED_MM[0] and width % 8 == 0 and ff % 8 == 0):
-            rows = moe_experts_grouped(x, up, down, ids, wts, activation, weight_input, alpha, limit)
+            rows = moe_experts_grouped(x, up, down, ids, wts, activation, weight_input, alpha, limit, placed)
             return rows if leave_sum else rows.summed()
     act = _new((R * top, ff), x.dtype, x.device)
     st = native.lib().rfx_moe_up(_chk(x, "x"), _chk(up, "up", x.dtype), _chk(ids, "ids", torch.int32),
@@ -976,9 +1005,14 @@ MOE_GROUPED = _env_flag("REFLEX_B200_MOE_GROUPED", True)
 MOE_GROUPED_MIN_ROWS = _env_int("REFLEX_B200_MOE_GROUPED_MIN_ROWS", 2, 1, 1 << 30)
 
 
+def moe_grouped(x: torch.Tensor) -> bool:
+    """Whether `moe_experts` groups these rows expert by expert (where it can)."""
+    return x.dtype == torch.bfloat16 and MOE_GROUPED and x.shape[0] >= MOE_GROUPED_MIN_ROWS
+
+
 def moe_experts_grouped(x: torch.Tensor, up: torch.Tensor, down: torch.Tensor, ids: torch.Tensor,
                         wts: torch.Tensor, activation: str = "relu2", weight_input: bool = False,
-                        alpha: float = 1.0, limit: float = 0.0) -> ExpertRows:
+                        alpha: float = 1.0, limit: float = 0.0, placed=None) -> ExpertRows:
     """The same for many bfloat16 rows (prefill), up to the sum: the (row, choice) pairs are
     placed expert by expert on the device, each expert's block of rows goes
     through its two matrices as library products (where the dense layers use
@@ -1005,10 +1039,13 @@ def moe_experts_grouped(x: torch.Tensor, up: torch.Tensor, down: torch.Tensor, i
                                             MOE_ACTIVATIONS[activation], _stream()), "moe_activation")
         return a
 
-    offsets = _new((E + 1,), torch.int32, x.device)
-    place = _new((n,), torch.int32, x.device)
-    native.check(lib.rfx_moe_group(_chk(ids, "ids", torch.int32), n, E, offsets.data_ptr(), place.data_ptr(),
-                                   _stream()), "moe_group")
+    if placed is not None:
+        offsets, place = placed
+    else:
+        offsets = _new((E + 1,), torch.int32, x.device)
+        place = _new((n,), torch.int32, x.device)
+        native.check(lib.rfx_moe_group(_chk(ids, "ids", torch.int32), n, E, offsets.data_ptr(), place.data_ptr(),
+                                       _stream()), "moe_group")
     xg = _new((n, width), x.dtype, x.device)
     native.check(lib.rfx_moe_gather(_chk(x, "x"), place.data_ptr(), _chk(in_scale, "wts", torch.float32),
                                     xg.data_ptr(), dt_code(x.dtype), n, top, width, _stream()), "moe_gather")
@@ -1829,6 +1866,19 @@ def latent_rot_post(proj: torch.Tensor, kv_weight: torch.Tensor, eps: float, rot
     return out
 
 
+def rotate_tails_(x: torch.Tensor, heads: int, rot_dim: int, rotation, row_pos) -> torch.Tensor:
+    """x [R, heads * n]: the last `rot_dim` elements of every head rotated (half-split
+    pairs) in place; rot_dim a multiple of 4, n even."""
+    R, n = x.shape[0], x.shape[1] // heads
+    denom, rot = _plain_rotation(rotation, "rotate_tails")
+    if rot != rot_dim or x.shape[1] != heads * n:
+        raise InvalidInput("rotate_tails: the rotation covers the whole rotated part of every head")
+    st = native.lib().rfx_rotate_tails(_chk(x, "x"), dt_code(x.dtype), _chk(denom, "denominators", torch.float32),
+                                       _chk(row_pos, "row_pos", torch.int32), R, heads, n, rot_dim, _stream())
+    native.check(st, f"rotate_tails (heads={heads}, n={n}, rot={rot_dim})")
+    return x
+
+
 def latent_low_post(proj: torch.Tensor, q_weight: torch.Tensor, kv_weight: torch.Tensor, eps: float, rotation, row_pos,
                     row_slot, pages, page_table, page_size: int, q_rank: int, rank: int, rot_dim: int, width: int,
                     writes_cache: bool, out_dtype: torch.dtype) -> torch.Tensor:
@@ -1915,10 +1965,12 @@ def latent_gather(pages: torch.Tensor, page_table, page_size: int, batch, width:
 
 
 def attention_prefill_tc_rows(q: torch.Tensor, kv: torch.Tensor, seq_base: torch.Tensor, batch, heads: int, dk: int,
-                              dvp: int, dv: int, window, scale: float, sink: Optional[torch.Tensor] = None) -> torch.Tensor:
+                              dvp: int, dv: int, window, scale: float, sink: Optional[torch.Tensor] = None,
+                              gate=None) -> torch.Tensor:
     """tcgen05 attention of q [R, heads * dk] over keys and values that are the rows of
     `kv` [rows, heads * (dk + dvp)] (all heads' keys, then all heads' values);
-    position p of sequence i is row seq_base[i] + p.  [R, heads * dv]."""
+    position p of sequence i is row seq_base[i] + p.  [R, heads * dv].  `gate` = (rows of
+    a product, first column): out[r, c] is multiplied by sigmoid(rows[r, column + c])."""
     R = q.shape[0]
     if kv.shape[1] != heads * (dk + dvp) or q.shape[1] != heads * dk:
         raise InvalidInput("attention_prefill_tc_rows: q and kv do not match the heads")
@@ -1928,7 +1980,7 @@ def attention_prefill_tc_rows(q: torch.Tensor, kv: torch.Tensor, seq_base: torch
         _chk(batch.seq_slot, "seq_slot", torch.int32), _chk(batch.seq_start, "seq_start", torch.int32),
         _chk(batch.seq_new, "seq_new", torch.int32), _chk(batch.seq_row0, "seq_row0", torch.int32), out.data_ptr(),
         batch.seq_slot.numel(), int(batch.max_new), R, heads, dk, dvp, dv, int(window or 0), float(scale),
-        _chk(sink, "sink", torch.float32), device_error_word(q.device).data_ptr(), _stream())
+        _chk(sink, "sink", torch.float32), *_gate_args(gate, R), device_error_word(q.device).data_ptr(), _stream())
     native.check(st, f"attention_prefill_tc_rows (dk={dk}, dv={dv})")
     return out
 

@@ -21,7 +21,7 @@ c_float = ctypes.c_float
 c_longlong = ctypes.c_longlong
 
 _SIGNATURES = {
-    "rfx_embed": [c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_float, c_void_p, c_void_p, c_void_p],
+    "rfx_embed": [c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_float, c_void_p, c_void_p, c_void_p, c_void_p],
     "rfx_rmsnorm": [c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_float, c_float, c_void_p, c_int,
                     c_void_p, c_int, c_int, c_void_p],
     "rfx_swiglu": [c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_void_p],
@@ -49,14 +49,15 @@ _SIGNATURES = {
                             c_float, c_void_p],
     "rfx_attention_decode_kf": [c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_void_p, c_void_p,
                                 c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_float,
-                                c_void_p, c_void_p, c_float, c_longlong, c_int, c_void_p, c_void_p],
+                                c_void_p, c_void_p, c_float, c_longlong, c_int, c_void_p, c_int, c_int, c_int,
+                                c_void_p, c_void_p],
     "rfx_attention_prefill_kf": [c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_void_p, c_void_p,
                                  c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int,
                                  c_float, c_void_p, c_void_p, c_float, c_void_p],
     "rfx_attention_prefill_tc_kf": [c_void_p, c_void_p, c_void_p, c_longlong, c_void_p, c_int, c_int, c_void_p,
                                     c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int,
                                     c_int, c_int, c_int, c_float, c_void_p, c_void_p, c_float, c_float, c_void_p,
-                                    c_void_p],
+                                    c_int, c_int, c_int, c_void_p, c_void_p],
     "rfx_qkv_post_kv": [c_void_p, c_int, c_int, c_void_p, c_void_p, c_float, c_float, c_void_p, c_int,
                         c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_int, c_int,
                         c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_int, c_void_p],
@@ -91,8 +92,8 @@ _SIGNATURES = {
     "rfx_latent_post": [c_void_p, c_int, c_int, c_void_p, c_void_p, c_float, c_void_p, c_void_p, c_void_p,
                         c_void_p, c_int, c_void_p, c_int, c_int, c_void_p, c_int, c_int, c_int, c_int, c_int,
                         c_void_p],
-    "rfx_heads_linear": [c_void_p, c_int, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_void_p, c_int, c_int,
-                         c_int, c_int, c_void_p],
+    "rfx_heads_linear": [c_void_p, c_int, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_void_p, c_void_p, c_int,
+                         c_int, c_int, c_int, c_int, c_int, c_int, c_void_p],
     "rfx_scale_heads": [c_void_p, c_int, c_void_p, c_longlong, c_int, c_void_p],
     "rfx_mlstm_scan": [c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_float,
                        c_float, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int,
@@ -112,7 +113,7 @@ _SIGNATURES = {
     "rfx_moe_activation": [c_void_p, c_int, c_longlong, c_int, c_void_p],
     "rfx_moe_combine": [c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_void_p],
     "rfx_moe_route_groups": [c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_float,
-                             c_int, c_int, c_void_p],
+                             c_int, c_int, c_void_p, c_void_p, c_void_p],
     "rfx_sandwich_norm": [c_void_p, c_void_p, c_void_p, c_float, c_float, c_float, c_void_p, c_float, c_float,
                           c_void_p, c_int, c_int, c_int, c_int, c_void_p],
     "rfx_group_norm_gate": [c_void_p, c_void_p, c_float, c_void_p, c_int, c_int, c_int, c_int, c_void_p, c_int, c_int,
@@ -137,6 +138,7 @@ _SIGNATURES = {
                           c_void_p],
     "rfx_latent_low_post": [c_void_p, c_int, c_int, c_void_p, c_void_p, c_float, c_void_p, c_void_p, c_void_p, c_void_p,
                             c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p],
+    "rfx_rotate_tails": [c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_void_p],
     "rfx_head_gate_mul": [c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p],
     "rfx_sum_norm": [c_void_p, c_int, c_void_p, c_void_p, c_int, c_void_p, c_float, c_void_p, c_float, c_float,
                      c_void_p, c_int, c_int, c_int, c_void_p],
@@ -145,7 +147,7 @@ _SIGNATURES = {
     "rfx_latent_value_columns": [c_int, c_int],
     "rfx_attention_prefill_tc_rows": [c_void_p, c_void_p, c_longlong, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p,
                                       c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_float,
-                                      c_void_p, c_void_p, c_void_p],
+                                      c_void_p, c_void_p, c_int, c_int, c_int, c_void_p, c_void_p],
     "rfx_latent_rot_post": [c_void_p, c_int, c_int, c_void_p, c_float, c_void_p, c_void_p, c_void_p, c_void_p, c_int,
                             c_void_p, c_int, c_int, c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int,
                             c_int, c_int, c_void_p],

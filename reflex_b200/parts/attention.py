@@ -228,11 +228,10 @@ class GQAttention:
                 values_are_keys=self.values_are_keys, ld=cols)
         ops.prof_mark("norm_rope")
         attn = ops.attention(q, kv.k_pages, kv.v_pages, kv.page_table, kv.page_size, batch, s.num_heads,
-                             s.num_kv_heads, self.pad, s.window, s.scale, keep_first=self.keep_first)
+                             s.num_kv_heads, self.pad, s.window, s.scale, keep_first=self.keep_first,
+                             gate=(proj, gate_col) if self.head_gate else None)
         if self.output_gate:
             ops.sigmoid_gate_mul_(attn, proj, gate_col)
-        elif self.head_gate:
-            ops.sigmoid_gate_mul_(attn, proj, gate_col, heads=s.num_heads)
         ops.prof_mark("attn")
         out = ops.linear(attn, self.o, out_dtype=torch.float32)
         ops.prof_mark("o_proj")

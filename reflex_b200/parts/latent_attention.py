@@ -216,6 +216,7 @@ class LatentAttention:
         ops.prof_mark("qkv_gemm")
         rotation = self._rotation()
         expand = self._expand(batch)
+        gate = (proj, self.gate_col) if self.element_gate else None
         rows, writes = proj, ctx.writes_cache
         if self.q_rank:
             cq = ops.latent_low_post(proj, self.q_norm, self.kv_norm, self.eps, rotation, batch.row_pos, batch.row_slot,
@@ -228,13 +229,17 @@ class LatentAttention:
         post = (rows, self.kv_norm, self.eps, rotation, batch.row_pos, batch.row_slot, kv.k_pages, kv.page_table,
                 kv.page_size, H, d, self.rot_dim, self.kv_rank, self.width, writes, self.dtype)
         if expand:
-            q = ops.latent_rot_post(*post, query_width=self.dk)
+            if self.q_rank and rows.dtype == self.dtype and d + self.rot_dim == self.dk and self.rot_dim % 4 == 0 \
+                    and rotation is not None:
+                q = ops.rotate_tails_(rows, H, self.rot_dim, rotation, batch.row_pos)  # as wide as they are to be
+            else:
+                q = ops.latent_rot_post(*post, query_width=self.dk)
             ops.prof_mark("latent_post")
             rows, base = ops.latent_gather(kv.k_pages, kv.page_table, kv.page_size, batch, self.width)
             both = ops.linear(rows, self.kv_up)
             ops.prof_mark("kv_up")
             vals = ops.attention_prefill_tc_rows(q, both, base, batch, H, self.dk, self.dvp, s.value_dim, s.window,
-                                                 s.scale, sink=self.sink)
+                                                 s.scale, sink=self.sink, gate=gate)
             ops.prof_mark("attn")
         else:
             flat, qa = ops.latent_rot_post(*post)
@@ -244,10 +249,9 @@ class LatentAttention:
             attn = ops.latent_attention(qa, kv.k_pages, kv.page_table, kv.page_size, batch, H, self.width,
                                         self.kv_rank, s.window, s.scale, sink=self.sink)
             ops.prof_mark("attn")
-            vals = ops.heads_linear(attn, self.v_up)  # of each head the latent's elements; the rest is dropped
+            # of each head the latent's elements; the rest is dropped
+            vals = ops.heads_linear(attn, self.v_up, gate=gate)
             ops.prof_mark("v_up")
-        if self.element_gate:
-            ops.sigmoid_gate_mul_(vals, proj, self.gate_col)
         out = ops.linear(vals, self.o, out_dtype=torch.float32)
         ops.prof_mark("o_proj")
         return out

@@ -129,11 +129,13 @@ class MixtureOfExperts:
             logits, col0 = ops.linear(x, self.router, out_dtype=torch.float32), 0  # [rows, experts (+ the shared gate)]
         else:
             logits, col0 = proj
-        ids, wts = ops.moe_route(logits, self.router_bias, self.top, experts=self.experts, scores=self.scores,
-                                 col0=col0, scale=self.score_scale, groups=self.groups)
+        place = ops.moe_grouped(x) and x.shape[0] <= ops.MOE_PLACE_MAX_ROWS
+        ids, wts, *placed = ops.moe_route(logits, self.router_bias, self.top, experts=self.experts, scores=self.scores,
+                                          col0=col0, scale=self.score_scale, groups=self.groups, place=place)
         ops.prof_mark("moe_router")
         out = ops.moe_experts(x, self.up, self.down, ids, wts, self.activation, self.weight_input, self.alpha,
-                              self.limit, leave_sum=leave_sum and self.leaves_sum and onto is None)
+                              self.limit, leave_sum=leave_sum and self.leaves_sum and onto is None,
+                              placed=placed[0] if placed else None)
         ops.prof_mark("moe_experts")
         if self.shared_ff and self.shared_kind == "swiglu":
             # the shared expert as it is: gate and up woven into one product, added to the experts' sum
