@@ -99,8 +99,8 @@ extern "C" int rfx_attention_decode(const void* q, const void* k_pages, const vo
 
 // The same with `keep_first` (the first so many positions of a sequence stay
 // visible beyond the window) and `softcap` (> 0: a score s becomes softcap * tanh(s / softcap)
-// before the softmax; not together with slopes).  `gate_z` (or null): rows of `gate_ld` elements; head
-// h's output of row r is multiplied by sigmoid(gate_z[r, gate_col + h]).
+// before the softmax; not together with slopes).  `gate_z` (or null): rows of `gate_ld` elements;
+// sigmoid(gate_z[r, gate_col + h]) scales what head h of row r gives.
 extern "C" int rfx_attention_decode_kf(const void* q, const void* k_pages, const void* v_pages,
                                        const int* page_table, int max_pages, int page_size,
                                        const int* row_pos, const int* row_slot, void* out,

@@ -656,7 +656,7 @@ extern "C" int rfx_attention_prefill_tc_trace(void* buffer, int ctas) {
 // `keep_first`: with a window, the first so many positions of a sequence stay visible
 // beyond it.  `softcap` > 0: a score s becomes softcap * tanh(s / softcap) (not with slopes);
 // `score_bound` > 0: the caller's word that no |s| is larger.  `gate_z` (or null): rows of
-// `gate_ld` elements; head h's output of row r is multiplied by sigmoid(gate_z[r, gate_col + h]).
+// `gate_ld` elements; sigmoid(gate_z[r, gate_col + h]) scales what head h of row r gives.
 extern "C" int rfx_attention_prefill_tc_kf(const void* q, const void* k_pages, const void* v_pages,
                                            long long n_pages_total, const int* page_table, int max_pages,
                                            int page_size, const int* seq_slot, const int* seq_start,

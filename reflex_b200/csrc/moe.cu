@@ -56,7 +56,7 @@ __device__ __forceinline__ void route_row(const float* __restrict__ logits, int 
         all_sum = warp_sum(s);
     }
     if (keep < groups) {
-        // a group's score is the largest in it; the best `keep` groups stay, ties to the lower index
+        // groups are ranked by their best expert; the first `keep` stay, ties to the lower index
         const int size = E / groups;
         float best[PL];  // group g's best in lane g % 32
 #pragma unroll

@@ -1,8 +1,8 @@
 """Pidodra as data: its typed config turned into a `ModelSpec`.
 
 The design: a token embedding times a scale; layers that norm the sum of a
-multiple of the stream and what a sublayer makes of it, x <- norm1(alpha x +
-mixer(x)), x <- norm2(alpha x + ff(x)); the mixer is a latent attention (queries
+multiple of the stream and what a sublayer makes of it, h = norm1(a h +
+mixer(h)), h = norm2(a h + ff(h)); the mixer is a latent attention (queries
 through a normed latent, one cached latent a position for all heads' keys and
 values, beside it one rotated key part all heads share with neighbouring elements
 as pairs, a sink in the softmax's denominator, a sigmoid gate on every element) or

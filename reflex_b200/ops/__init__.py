@@ -603,8 +603,8 @@ def attention_decode(q, k_pages, v_pages, page_table, page_size, row_pos, row_sl
                      slopes: Optional[torch.Tensor] = None, keep_first: int = 0,
                      softcap: float = 0.0, gate=None) -> torch.Tensor:
     """bfloat16 tensor-core attention for rows that are each one query
-    position (decode), split over the keys.  `gate` = (rows, first column): head h's
-    output is multiplied by sigmoid(rows[r, column + h])."""
+    position (decode), split over the keys.  `gate` = (rows, first column):
+    sigmoid(rows[r, column + h]) scales what head h of row r gives."""
     keep_first = int(keep_first) if window else 0
     R = q.shape[0]
     _chk(q, "q", torch.bfloat16)
@@ -702,8 +702,8 @@ def attention(q, k_pages, v_pages, page_table, page_size, batch, nq, nkv, head_d
     position) is taken off every score.  `keep_first`: with a window, the first
     so many positions of a sequence stay visible beyond it.  `softcap` > 0: a score
     s becomes softcap * tanh(s / softcap) before the softmax; `score_bound` > 0: the
-    caller knows that no |s| is larger.  `gate` = (rows of a product, first column): head
-    h's output is multiplied by sigmoid(rows[r, column + h])."""
+    caller knows that no |s| is larger.  `gate` = (rows of a product, first
+    column): sigmoid(rows[r, column + h]) scales what head h of row r gives."""
     fast = q.dtype == torch.bfloat16 and head_dim % 16 == 0 and head_dim <= 256
     keep_first = int(keep_first) if window else 0
     if fast and batch.is_decode:

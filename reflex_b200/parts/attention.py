@@ -16,8 +16,8 @@ padded alike.
 Options, by the spec's parameters: `values_are_keys` (there is no Wv; a value
 head is its key head as projected, before the norm and the rotation),
 `output_gate` (a further matrix Wg; the concatenated heads are multiplied by
-sigmoid(x Wg^T) before Wo), `head_gate` (Wg has a row a head: head h's output is
-multiplied by the one number sigmoid(x Wg^T)_h), `reads_cache` (the layer has no keys
+sigmoid(x Wg^T) before Wo), `head_gate` (Wg has a row a head, and the one number
+sigmoid(x Wg^T)_h scales all that head h gives), `reads_cache` (the layer has no keys
 and values of its own, and so no Wk, Wv and key norm: its runs read the entry of
 another layer of the same head sizes) and `keep_first` (with a window: the first so many
 positions of a sequence stay visible to every later query, i - j < window or

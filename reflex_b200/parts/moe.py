@@ -20,9 +20,9 @@ is added times sigmoid(w_sg . x), one number a row; its gate's row rides along
 as one more row of the router's matrix.  `scores` "softmax_all": the weights are
 the softmax over all experts' logits, the chosen ones' divided by their sum
 (+ 1e-20); "softmax": the same scores as they are; `score_scale` multiplies the
-weights.  `groups` (count, keep): the experts form `count` equal groups of
-neighbours, a group's score is the largest in it, and only experts of the `keep`
-best groups can be chosen (ties: the lower index).  `activation` "swiglu": an
+weights.  `groups` (count, keep): the choice is limited to `keep` of `count`
+runs of consecutive experts, those whose best expert scores highest (ties: the lower
+index).  `activation` "swiglu": an
 expert is W_down (silu(W_gate x) * (W_up x)).  `shared_kind` "swiglu" (with
 `shared_ff`): the shared expert is that gated silu form and is added as it is,
 with no gate of its own.

@@ -105,12 +105,13 @@ class RotaryYarn(RotaryNeox):
     """The rotation with frequencies scaled by how often a pair turns within the
     original context, and a magnitude.
 
-    With f_i = theta^(-2i/rd), the parameters `factor`, `original`, `fast`, `slow`,
-    and n(t) = rd ln(original / (2 pi t)) / (2 ln theta), the (fractional) index of the
-    pair that turns t times within `original` positions: lo = max(floor(n(fast)), 0),
-    hi = min(ceil(n(slow)), rd - 1), ramp_i = (i - lo) / max(hi - lo, 0.001) within
-    [0, 1], and the frequency is f_i (1 - ramp_i) + f_i / factor * ramp_i.  Cosine and
-    sine are multiplied by 0.1 ln(factor) + 1."""
+    A pair i of plain frequency g_i = theta^(-2i/rd) makes N g_i / (2 pi) turns within
+    N = `original` positions; the pair that makes t of them has the fractional index
+    j(t) = rd / 2 * log_theta(N / (2 pi t)).  Pairs up to a = floor(j(`fast`)) (at
+    least 0) keep g_i, pairs from b = ceil(j(`slow`)) (at most rd - 1) on turn `factor`
+    times slower, and between them the two frequencies are blended with the weight
+    s_i = (i - a) / (b - a) on the slower one (the width b - a taken as 0.001 at least,
+    s_i kept within 0 and 1).  Cosine and sine grow by 1 + ln(factor) / 10."""
 
     def __init__(self, spec: PositionSpec, dtype: torch.dtype, device):
         super().__init__(spec, dtype, device)
@@ -123,11 +124,11 @@ class RotaryYarn(RotaryNeox):
         def index_of(turns: float) -> float:
             return rd * math.log(original / (2.0 * math.pi * turns)) / (2.0 * math.log(base))
 
-        lo, hi = max(math.floor(index_of(fast)), 0), min(math.ceil(index_of(slow)), rd - 1)
+        first, last = max(math.floor(index_of(fast)), 0), min(math.ceil(index_of(slow)), rd - 1)
         denom = []
         for i in range(rd // 2):
-            f = math.pow(base, -2.0 * i / float(rd))
-            ramp = min(max((i - lo) / max(hi - lo, 0.001), 0.0), 1.0)
-            denom.append(1.0 / (f / factor * ramp + f * (1.0 - ramp)))
+            g = math.pow(base, -2.0 * i / float(rd))
+            s = min(max((i - first) / max(last - first, 0.001), 0.0), 1.0)
+            denom.append(1.0 / (g / factor * s + g * (1.0 - s)))
         self.denominators = torch.tensor(denom, dtype=torch.float64).to(torch.float32).to(device)
         self.magnitude = 0.1 * math.log(factor) + 1.0

@@ -5,8 +5,8 @@ precision; it shares no code with `reflex_b200`.  Linear weights are [out, in]
 and applied as y = x W^T.
 
 The design: the token embedding times a scale; layers that norm the sum of a
-multiple of the stream and what a sublayer makes of it, x <- norm1(alpha x +
-mixer(x)), x <- norm2(alpha x + ff(x)); the mixer is a latent attention (queries
+multiple of the stream and what a sublayer makes of it, h = norm1(a h +
+mixer(h)), h = norm2(a h + ff(h)); the mixer is a latent attention (queries
 through a normed latent, keys and values from a cached normed latent, one rotated
 key part all heads share, a sink in the softmax, a gate per element) or a grouped
 attention (normed queries and keys, a YaRN-scaled rotation, a gate per head), which
@@ -80,12 +80,12 @@ def yarn_frequencies(dims: int, base: float, factor: float, original: float, fas
     def index_of(turns: float) -> float:
         return dims * math.log(original / (2.0 * math.pi * turns)) / (2.0 * math.log(base))
 
-    lo = max(math.floor(index_of(fast)), 0)
-    hi = min(math.ceil(index_of(slow)), dims - 1)
+    a = max(math.floor(index_of(fast)), 0)
+    b = min(math.ceil(index_of(slow)), dims - 1)
     out = []
-    for i, f in enumerate(inverse_frequencies(dims, base)):
-        ramp = min(max((i - lo) / max(hi - lo, 0.001), 0.0), 1.0)
-        out.append(f / factor * ramp + f * (1.0 - ramp))
+    for i, g in enumerate(inverse_frequencies(dims, base)):
+        slower = min(max((i - a) / max(b - a, 0.001), 0.0), 1.0)  # the share of the divided frequency
+        out.append((g / factor) * slower + g * (1.0 - slower))
     return out
 
 
